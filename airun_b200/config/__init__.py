@@ -6,6 +6,7 @@ from .vedizen import VedizenConfig
 from .pogarax import PogaraxConfig
 from .gamanex import GamanexConfig
 from .tagulix import TagulixConfig
+from .losalorn import LosalornConfig
 
 
 def _register_builtin() -> None:
@@ -15,6 +16,7 @@ def _register_builtin() -> None:
     register_architecture("Pogarax", PogaraxConfig, build_decoder)
     register_architecture("Gamanex", GamanexConfig, build_decoder)
     register_architecture("Tagulix", TagulixConfig, build_decoder)
+    register_architecture("Losalorn", LosalornConfig, build_decoder)
 
 
 _register_builtin()

@@ -47,11 +47,13 @@ class LayerCall:
     own, or the index of an earlier entry of the order whose cache it reads
     instead of writing one.  ``add_row`` names a row of the configuration's ``order_table()`` (a
     [rows, hidden] tensor of the model) that is added to every token of the residual stream right before
-    this entry runs: the offset of a pass over layers that run several times.
+    this entry runs: the offset of a pass over layers that run several times.  ``reinject``: the model's
+    ``residual_input()`` part mixes the stream with the embedding right before this entry runs.
     """
     layer: int
     cache_from: Optional[int] = None
     add_row: Optional[int] = None     # row of the model's order table added to the residual stream before this entry
+    reinject: bool = False            # the residual stream is mixed with the embedding before this entry
 
 
 class ModelConfig:
@@ -79,6 +81,11 @@ class ModelConfig:
     def head(self) -> Tuple[str, dict]:
         """(registered name, constructor arguments) of the output head, e.g. ("lm_head", {"soft_cap": 30.0})."""
         return "lm_head", {}
+
+    def residual_input(self) -> Optional[Tuple[str, str, dict]]:
+        """(registered name, tensor prefix, constructor arguments) of the part that mixes the residual stream with the
+        embedding ahead of the entries of the execution order marked ``reinject``; None: there is none."""
+        return None
 
     def residual_streams(self) -> int:
         """Copies of the residual a token carries through the layers (arrangements that declare ``multi_stream`` read

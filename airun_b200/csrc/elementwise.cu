@@ -602,6 +602,148 @@ AIRUN_EXPORT int airun_postnorm_add(float* x, const float* y, const float* w, vo
     return airun_launch_status();
 }
 
+// What lies between two sub-layers whose inputs AND outputs are normed, in one pass over the residual row:
+//     v = x[src] + y[src] / rms(y[src]) * w_post                 the result of the sub-layer before (without y: v = x[src])
+//     x[src] = v                                                 when `write_back` is set
+//     out[r]  by `mode`:  SANDWICH_NORM   v / rms(v) * w_pre     the input of the sub-layer after, in TOut
+//                         SANDWICH_COPY   v                      float32
+//                         SANDWICH_SPLIT  [hi | lo], 2n bfloat16 numbers with hi + lo = v to 16 bits of mantissa: a product
+//                                         over them reads v without rounding it to bfloat16
+// src = rows ? rows[r] : r.  One block per row; up to KEEP vectors a thread stay in registers between the passes, and
+// the weights, which no kernel writes, are read before the kernel in front has finished.
+#define SANDWICH_NORM 0
+#define SANDWICH_COPY 1
+#define SANDWICH_SPLIT 2
+template <typename TOut>
+__device__ __forceinline__ void sandwich_put(TOut* __restrict__ out, int i, int n, int mode, float v, float inv, float w) {
+    if (mode == SANDWICH_NORM) {
+        out[i] = from_f32<TOut>(v * inv * w);
+    } else if (mode == SANDWICH_COPY) {
+        out[i] = from_f32<TOut>(v);
+    } else {
+        const TOut hi = from_f32<TOut>(v);
+        out[i] = hi;
+        out[n + i] = from_f32<TOut>(v - to_f32<TOut>(hi));
+    }
+}
+
+template <typename TOut, int VEC>
+__global__ __launch_bounds__(512) void sandwich_norm_kernel(float* __restrict__ x, const float* __restrict__ y, const float* __restrict__ w_post,
+                                     const float* __restrict__ w_pre, TOut* __restrict__ out, const int32_t* __restrict__ rows,
+                                     int n, float eps_post, float eps_pre, int write_back, int mode) {
+    pdl_trigger();
+    __shared__ float red[33];
+    const int nv = n / VEC;
+    float v[KEEP][VEC], yk[KEEP][VEC], wa[KEEP][VEC], wb[KEEP][VEC];
+    auto load = [&](const float* __restrict__ p, float (&d)[VEC], int i, float none) {
+        if (!p || i >= nv) {
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) d[e] = none;
+        } else if (VEC == 4) {
+            const float4 f = reinterpret_cast<const float4*>(p)[i];
+            d[0] = f.x; d[1 % VEC] = f.y; d[2 % VEC] = f.z; d[3 % VEC] = f.w;
+        } else {
+            d[0] = p[i];
+        }
+    };
+#pragma unroll
+    for (int k = 0; k < KEEP; ++k) {
+        load(y ? w_post : nullptr, wa[k], threadIdx.x + k * blockDim.x, 0.0f);
+        load(mode == SANDWICH_NORM ? w_pre : nullptr, wb[k], threadIdx.x + k * blockDim.x, 1.0f);
+    }
+    pdl_wait();
+    const int r = blockIdx.x, src = rows ? rows[r] : r;
+    float* xr = x + (size_t)src * n;
+    const float* yr = y ? y + (size_t)src * n : nullptr;
+    TOut* outr = out ? out + (size_t)r * (mode == SANDWICH_SPLIT ? 2 * n : n) : nullptr;
+    const int tail0 = (threadIdx.x + KEEP * blockDim.x) * VEC, tstep = blockDim.x * VEC;       // a row longer than the registers hold
+    float ss = 0.0f;
+#pragma unroll
+    for (int k = 0; k < KEEP; ++k) {
+        load(xr, v[k], threadIdx.x + k * blockDim.x, 0.0f);
+        load(yr, yk[k], threadIdx.x + k * blockDim.x, 0.0f);
+    }
+    float inv_y = 0.0f;
+    if (yr) {
+#pragma unroll
+        for (int k = 0; k < KEEP; ++k)
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) ss = fmaf(yk[k][e], yk[k][e], ss);
+        for (int i = tail0; i < n; i += tstep)
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) ss = fmaf(yr[i + e], yr[i + e], ss);
+        inv_y = 1.0f / sqrtf(block_sum(ss, red) / (float)n + eps_post);
+    }
+    ss = 0.0f;
+#pragma unroll
+    for (int k = 0; k < KEEP; ++k) {
+        const int i = threadIdx.x + k * blockDim.x;
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) {
+            v[k][e] += yk[k][e] * inv_y * wa[k][e];
+            ss = fmaf(v[k][e], v[k][e], ss);
+        }
+        if (yr && write_back && i < nv) {
+            if (VEC == 4) reinterpret_cast<float4*>(xr)[i] = make_float4(v[k][0], v[k][1 % VEC], v[k][2 % VEC], v[k][3 % VEC]);
+            else xr[i] = v[k][0];
+        }
+    }
+    for (int i = tail0; i < n; i += tstep)
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) {
+            const float u = xr[i + e] + (yr ? yr[i + e] * inv_y * w_post[i + e] : 0.0f);
+            if (yr && write_back) xr[i + e] = u;
+            ss = fmaf(u, u, ss);
+        }
+    if (!outr) return;
+    const float inv = mode == SANDWICH_NORM ? 1.0f / sqrtf(block_sum(ss, red) / (float)n + eps_pre) : 1.0f;
+#pragma unroll
+    for (int k = 0; k < KEEP; ++k) {
+        const int i = threadIdx.x + k * blockDim.x;
+        if (i >= nv) continue;
+        if (VEC == 4 && sizeof(TOut) == 2 && mode == SANDWICH_NORM) {
+            __nv_bfloat162 lo = __floats2bfloat162_rn(v[k][0] * inv * wb[k][0], v[k][1 % VEC] * inv * wb[k][1 % VEC]);
+            __nv_bfloat162 hi = __floats2bfloat162_rn(v[k][2 % VEC] * inv * wb[k][2 % VEC], v[k][3 % VEC] * inv * wb[k][3 % VEC]);
+            reinterpret_cast<uint2*>(outr)[i] = make_uint2(*reinterpret_cast<uint32_t*>(&lo), *reinterpret_cast<uint32_t*>(&hi));
+        } else if (VEC == 4 && sizeof(TOut) == 4 && mode == SANDWICH_NORM) {
+            reinterpret_cast<float4*>(outr)[i] = make_float4(v[k][0] * inv * wb[k][0], v[k][1 % VEC] * inv * wb[k][1 % VEC],
+                                                             v[k][2 % VEC] * inv * wb[k][2 % VEC], v[k][3 % VEC] * inv * wb[k][3 % VEC]);
+        } else {
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) sandwich_put<TOut>(outr, i * VEC + e, n, mode, v[k][e], inv, wb[k][e]);
+        }
+    }
+    for (int i = tail0; i < n; i += tstep)
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) {
+            const float u = xr[i + e] + (yr && !write_back ? yr[i + e] * inv_y * w_post[i + e] : 0.0f);
+            sandwich_put<TOut>(outr, i + e, n, mode, u, inv, mode == SANDWICH_NORM ? w_pre[i + e] : 1.0f);
+        }
+}
+
+AIRUN_EXPORT int airun_sandwich_norm(float* x, const float* y, const float* w_post, const float* w_pre, void* out, int out_dtype,
+                                     const int32_t* rows, int n_rows, int n, float eps_post, float eps_pre, int write_back,
+                                     int mode, cudaStream_t stream) {
+    if (n_rows < 0 || n <= 0 || !x || (y && !w_post) || (!y && !out) || mode < 0 || mode > 2 || (mode == SANDWICH_NORM && out && !w_pre) ||
+        (rows && write_back) || (mode == SANDWICH_SPLIT && out_dtype != AIRUN_DT_BF16) || (mode == SANDWICH_COPY && out_dtype != AIRUN_DT_F32))
+        return AIRUN_ERR_ARG;
+    if (n_rows == 0) return AIRUN_OK;
+    const bool vec = n % 4 == 0 && (((uintptr_t)x | (uintptr_t)y | (uintptr_t)w_post | (uintptr_t)w_pre | (uintptr_t)out) & 15) == 0;
+    const int nv = vec ? n / 4 : n;
+    // many rows: as few threads as hold the row in registers; few rows: more of them, with fewer loads each
+    int threads = ((n_rows > 64 ? (nv + KEEP - 1) / KEEP : (nv + 1) / 2) + 31) / 32 * 32;
+    if (threads > 512) threads = 512;
+    if (threads < 32) threads = 32;
+#define SW_LAUNCH(TOut, VEC) \
+    airun_launch(sandwich_norm_kernel<TOut, VEC>, dim3(n_rows), dim3(threads), 0, stream, x, y, w_post, w_pre, (TOut*)out, rows, n, \
+                 eps_post, eps_pre, write_back, mode)
+    if (out_dtype == AIRUN_DT_F32) { if (vec) SW_LAUNCH(float, 4); else SW_LAUNCH(float, 1); }
+    else if (out_dtype == AIRUN_DT_BF16) { if (vec) SW_LAUNCH(__nv_bfloat16, 4); else SW_LAUNCH(__nv_bfloat16, 1); }
+    else return AIRUN_ERR_UNSUPPORTED;
+#undef SW_LAUNCH
+    return airun_launch_status();
+}
+
 // out = in in another type (float32 -> bfloat16 or a plain copy), n elements.
 template <typename TOut>
 __global__ void cast_kernel(const float* __restrict__ in, TOut* __restrict__ out, long long n) {

@@ -5,6 +5,7 @@
 //     u[j]     = beta_t * (v_t[j] - sum_d S[d][j] * k_t[d])
 //     S[d][j] <- S[d][j] + k_t[d] * u[j]
 //     o_t[j]   = sum_d S[d][j] * q_t[d]                      (the read-out sees the token's own write)
+// The same with ONE decay per head, worked out here from its projection a_t, g_t = exp(-exp(A_log) * softplus(a_t + dt_bias)).
 // Time mix with a bonus for the current token (value channels j < D as well):
 //     o_t[j]   = sum_d r_t[d] * (S[d][j] + u[d] * k_t[d] * v_t[j])
 //     S[d][j] <- w_t[d] * S[d][j] + k_t[d] * v_t[j]
@@ -130,11 +131,13 @@ AIRUN_EXPORT int airun_token_shift(const float* x, const float* mu, int n_mix, c
 #define RS_TT 16
 #define RS_DELTA 0
 #define RS_WKV 1
+#define RS_DELTA_HEAD 2
 
 struct RecurrentArgs {
     const float* q; const float* k; const float* v; const float* g;     // delta: q, k, v, decay; time mix: r, k, v, decay
     long long q_stride, k_stride, v_stride, g_stride;                    // row strides in elements
     const float* beta; long long beta_stride;                            // delta: [T][heads], before its sigmoid
+    const float* a_log; const float* dt_bias;                            // delta with one decay per head: [heads] each, and g is a_t [T][heads]
     const float* bonus;                                                  // time mix: [heads][D]
     float* state; long long slot_stride; int max_slots;
     const int32_t* cu_tokens; const int32_t* state_slots;
@@ -160,8 +163,10 @@ __global__ __launch_bounds__(128) void recurrent_state_kernel(RecurrentArgs a) {
     constexpr int COLS = 128 / DG;               // value columns of a block: 32 / DG a warp
     constexpr int TT = DP >= 256 ? 4 : DP >= 128 ? 8 : RS_TT;     // tokens of a stage (static shared memory stays under 48 KB)
     // two stages: the next tokens arrive by asynchronous copies while these are used
-    __shared__ __align__(16) float s_q[2][TT][DP], s_k[2][TT][DP], s_g[2][TT][DP], s_v[2][TT][COLS];
-    __shared__ float s_b[2][TT];
+    constexpr bool DELTA = MODE != RS_WKV, HEAD = MODE == RS_DELTA_HEAD;
+    constexpr int GW = HEAD ? 1 : DP;            // decays of a token: one number, or one a key channel
+    __shared__ __align__(16) float s_q[2][TT][DP], s_k[2][TT][DP], s_g[2][TT][GW], s_v[2][TT][COLS];
+    __shared__ float s_b[2][TT], s_kq[HEAD ? TT : 1];
     const int r = blockIdx.x, head = blockIdx.y, col0 = blockIdx.z * COLS;
     const int t0 = a.cu_tokens[r], n = a.cu_tokens[r + 1] - t0;
     if (n <= 0) return;
@@ -178,16 +183,17 @@ __global__ __launch_bounds__(128) void recurrent_state_kernel(RecurrentArgs a) {
     const int ncol = min(COLS, Dv - col0);
     // the padding beyond D and Dv is zero in both stages and is never copied into (nothing to do when there is none)
     if (D < DP || ncol < COLS) {
-        for (int e = threadIdx.x; e < 2 * TT * DP; e += 128) { (&s_q[0][0][0])[e] = 0.0f; (&s_k[0][0][0])[e] = 0.0f; (&s_g[0][0][0])[e] = 0.0f; }
+        for (int e = threadIdx.x; e < 2 * TT * DP; e += 128) { (&s_q[0][0][0])[e] = 0.0f; (&s_k[0][0][0])[e] = 0.0f; }
+        for (int e = threadIdx.x; e < 2 * TT * GW; e += 128) (&s_g[0][0][0])[e] = 0.0f;
         for (int e = threadIdx.x; e < 2 * TT * COLS; e += 128) (&s_v[0][0][0])[e] = 0.0f;
         __syncthreads();
     }
     const float* qh = a.q + (size_t)qk_head * D;
     const float* kh = a.k + (size_t)qk_head * D;
-    const float* gh = a.g + (size_t)head * D;
+    const float* gh = a.g + (size_t)head * (HEAD ? 1 : D);
     const float* vh = a.v + (size_t)head * Dv + col0;
-    const bool vec = (D % 4 == 0) && ((a.q_stride | a.k_stride | a.g_stride) % 4 == 0) &&
-                     ((((uintptr_t)qh | (uintptr_t)kh | (uintptr_t)gh) & 15) == 0);
+    const bool vec = (D % 4 == 0) && ((a.q_stride | a.k_stride | (HEAD ? 0 : a.g_stride)) % 4 == 0) &&
+                     ((((uintptr_t)qh | (uintptr_t)kh | (HEAD ? 0 : (uintptr_t)gh)) & 15) == 0);
     const bool vvec = (ncol % 4 == 0) && (a.v_stride % 4 == 0) && (((uintptr_t)vh & 15) == 0);
     auto stage = [&](int base, int buf) {
         const int nt = min(TT, n - base);
@@ -198,7 +204,7 @@ __global__ __launch_bounds__(128) void recurrent_state_kernel(RecurrentArgs a) {
                 const size_t row = (size_t)(t0 + base + tt);
                 rs_cp16(&s_q[buf][tt][d], qh + row * a.q_stride + d);
                 rs_cp16(&s_k[buf][tt][d], kh + row * a.k_stride + d);
-                rs_cp16(&s_g[buf][tt][d], gh + row * a.g_stride + d);
+                if (!HEAD) rs_cp16(&s_g[buf][tt][HEAD ? 0 : d], gh + row * a.g_stride + d);
             }
         } else {
             for (int e = threadIdx.x; e < nt * D; e += 128) {
@@ -206,7 +212,7 @@ __global__ __launch_bounds__(128) void recurrent_state_kernel(RecurrentArgs a) {
                 const size_t row = (size_t)(t0 + base + tt);
                 rs_cp4(&s_q[buf][tt][d], qh + row * a.q_stride + d);
                 rs_cp4(&s_k[buf][tt][d], kh + row * a.k_stride + d);
-                rs_cp4(&s_g[buf][tt][d], gh + row * a.g_stride + d);
+                if (!HEAD) rs_cp4(&s_g[buf][tt][HEAD ? 0 : d], gh + row * a.g_stride + d);
             }
         }
         if (vvec) {
@@ -221,8 +227,9 @@ __global__ __launch_bounds__(128) void recurrent_state_kernel(RecurrentArgs a) {
                 rs_cp4(&s_v[buf][tt][c], vh + (size_t)(t0 + base + tt) * a.v_stride + c);
             }
         }
-        if (MODE == RS_DELTA && threadIdx.x < nt)
+        if (DELTA && threadIdx.x < nt)
             rs_cp4(&s_b[buf][threadIdx.x], a.beta + (size_t)(t0 + base + threadIdx.x) * a.beta_stride + head);
+        if (HEAD && threadIdx.x < nt) rs_cp4(&s_g[buf][threadIdx.x][0], gh + (size_t)(t0 + base + threadIdx.x) * a.g_stride);
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
     stage(0, 0);
@@ -236,6 +243,7 @@ __global__ __launch_bounds__(128) void recurrent_state_kernel(RecurrentArgs a) {
         if (MODE == RS_WKV) bonus[i] = d < D ? a.bonus[(size_t)head * D + d] : 0.0f;
     }
     float* orow = a.out + (size_t)t0 * ((size_t)a.heads * Dv) + (size_t)head * Dv + col;
+    const float rate = HEAD ? expf(a.a_log[head]) : 0.0f, dt = HEAD ? a.dt_bias[head] : 0.0f;
     int it = 0;
     for (int base = 0; base < n; base += TT, ++it) {
         const int buf = it & 1, nt = min(TT, n - base);
@@ -246,18 +254,62 @@ __global__ __launch_bounds__(128) void recurrent_state_kernel(RecurrentArgs a) {
             asm volatile("cp.async.wait_group 0;" ::: "memory");
         }
         __syncthreads();
+        if (HEAD) {
+            // what belongs to a token and not to a column, once for the stage: its beta, its decay and k . q
+            constexpr int TPT = 128 / TT;       // neighbouring threads that share a token
+            const int tt = threadIdx.x / TPT, e0 = threadIdx.x % TPT;
+            float kq = 0.0f;
+#pragma unroll
+            for (int d = e0; d < DP; d += TPT) kq = fmaf(s_k[buf][tt][d], s_q[buf][tt][d], kq);
+#pragma unroll
+            for (int off = 1; off < TPT; off <<= 1) kq += __shfl_xor_sync(0xffffffffu, kq, off);
+            if (e0 == 0 && tt < nt) {
+                const float z = s_g[buf][tt][0] + dt;
+                s_g[buf][tt][0] = expf(-rate * (fmaxf(z, 0.0f) + log1pf(expf(-fabsf(z)))));
+                s_b[buf][tt] = 1.0f / (1.0f + expf(-s_b[buf][tt]));
+                s_kq[tt] = kq;
+            }
+            __syncthreads();
+        }
 #pragma unroll 2
         for (int tt = 0; tt < nt; ++tt) {
             const float vj = s_v[buf][tt][cl];
             float o;
-            if (MODE == RS_DELTA) {
+            if (HEAD) {
+                // the decay is one number, so it is applied to the sums over the old state and in the update
+                const float gt = s_g[buf][tt][0], beta = s_b[buf][tt];
+                float pred[2] = {0.0f, 0.0f}, oq[2] = {0.0f, 0.0f}, kr[NS];
+#pragma unroll
+                for (int i4 = 0; i4 < NS / 4; ++i4) {
+                    const int d = (i4 * DG + dg) * 4;
+                    const float4 k4 = *reinterpret_cast<const float4*>(&s_k[buf][tt][d]);
+                    const float4 q4 = *reinterpret_cast<const float4*>(&s_q[buf][tt][d]);
+                    const float kk[4] = {k4.x, k4.y, k4.z, k4.w}, qq[4] = {q4.x, q4.y, q4.z, q4.w};
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) {
+                        kr[4 * i4 + e] = kk[e];
+                        pred[e & 1] = fmaf(S[4 * i4 + e], kk[e], pred[e & 1]);
+                        oq[e & 1] = fmaf(S[4 * i4 + e], qq[e], oq[e & 1]);
+                    }
+                }
+                float p = pred[0] + pred[1], oqs = oq[0] + oq[1];
+#pragma unroll
+                for (int off = 1; off < DG; off <<= 1) {
+                    p += __shfl_xor_sync(0xffffffffu, p, off);
+                    oqs += __shfl_xor_sync(0xffffffffu, oqs, off);
+                }
+                const float u = beta * fmaf(-gt, p, vj);
+#pragma unroll
+                for (int i = 0; i < NS; ++i) S[i] = fmaf(kr[i], u, gt * S[i]);
+                o = fmaf(u, s_kq[tt], gt * oqs);
+            } else if (MODE == RS_DELTA) {
                 // beta arrives as the projection's output: the gate is its sigmoid
                 const float beta = 1.0f / (1.0f + expf(-s_b[buf][tt]));
                 float pred[2] = {0.0f, 0.0f}, oq[2] = {0.0f, 0.0f}, kq[2] = {0.0f, 0.0f};
 #pragma unroll
                 for (int i4 = 0; i4 < NS / 4; ++i4) {
                     const int d = (i4 * DG + dg) * 4;
-                    const float4 g4 = *reinterpret_cast<const float4*>(&s_g[buf][tt][d]);
+                    const float4 g4 = *reinterpret_cast<const float4*>(&s_g[buf][tt][HEAD ? 0 : d]);
                     const float4 k4 = *reinterpret_cast<const float4*>(&s_k[buf][tt][d]);
                     const float4 q4 = *reinterpret_cast<const float4*>(&s_q[buf][tt][d]);
                     const float gg[4] = {g4.x, g4.y, g4.z, g4.w}, kk[4] = {k4.x, k4.y, k4.z, k4.w}, qq[4] = {q4.x, q4.y, q4.z, q4.w};
@@ -292,7 +344,7 @@ __global__ __launch_bounds__(128) void recurrent_state_kernel(RecurrentArgs a) {
 #pragma unroll
                 for (int i4 = 0; i4 < NS / 4; ++i4) {
                     const int d = (i4 * DG + dg) * 4;
-                    const float4 g4 = *reinterpret_cast<const float4*>(&s_g[buf][tt][d]);
+                    const float4 g4 = *reinterpret_cast<const float4*>(&s_g[buf][tt][HEAD ? 0 : d]);
                     const float4 k4 = *reinterpret_cast<const float4*>(&s_k[buf][tt][d]);
                     const float4 q4 = *reinterpret_cast<const float4*>(&s_q[buf][tt][d]);
                     const float gg[4] = {g4.x, g4.y, g4.z, g4.w}, kk[4] = {k4.x, k4.y, k4.z, k4.w}, qq[4] = {q4.x, q4.y, q4.z, q4.w};
@@ -338,7 +390,8 @@ __global__ __launch_bounds__(128) void recurrent_state_kernel(RecurrentArgs a) {
 
 AIRUN_EXPORT int airun_recurrent_state(int mode, const float* q, const float* k, const float* v, const float* g,
                                        long long q_stride, long long k_stride, long long v_stride, long long g_stride,
-                                       const float* beta, long long beta_stride, const float* bonus, float* state,
+                                       const float* beta, long long beta_stride, const float* a_log, const float* dt_bias,
+                                       const float* bonus, float* state,
                                        long long slot_stride, int max_slots, const int32_t* cu_tokens, const int32_t* state_slots,
                                        int num_reqs, float* out, int heads, int kv_rep, int D, int Dv, const float* tail_src,
                                        long long tail_src_stride, long long tail_off, int tail_rows, int tail_width,
@@ -346,7 +399,8 @@ AIRUN_EXPORT int airun_recurrent_state(int mode, const float* q, const float* k,
     if (num_reqs < 0 || heads <= 0 || heads > 65535 || kv_rep <= 0 || heads % kv_rep || D <= 0 || D > 256 || Dv <= 0 || !state ||
         !cu_tokens || !state_slots || !err || !q || !k || !v || !g || !out || slot_stride < (long long)heads * D * Dv)
         return AIRUN_ERR_ARG;
-    if (mode == RS_DELTA ? !beta : !bonus) return AIRUN_ERR_ARG;
+    if (mode < RS_DELTA || mode > RS_DELTA_HEAD || (mode == RS_WKV ? !bonus : !beta) || (mode == RS_DELTA_HEAD && (!a_log || !dt_bias)))
+        return AIRUN_ERR_ARG;
     if (tail_rows < 0 || (tail_rows > 0 && (!tail_src || tail_width <= 0))) return AIRUN_ERR_ARG;
     if (num_reqs == 0) return AIRUN_OK;
     // lanes that share a value column: 8 where requests bring many tokens (the chain of a prompt's tokens bounds the
@@ -355,12 +409,13 @@ AIRUN_EXPORT int airun_recurrent_state(int mode, const float* q, const float* k,
     const int dg = (D <= 32 || !long_chains) ? 4 : 8;
     const int tiles = ceil_div_i(Dv, 128 / dg);
     if (tiles > 65535) return AIRUN_ERR_ARG;
-    RecurrentArgs a = {q, k, v, g, q_stride, k_stride, v_stride, g_stride, beta, beta_stride, bonus, state, slot_stride, max_slots,
+    RecurrentArgs a = {q, k, v, g, q_stride, k_stride, v_stride, g_stride, beta, beta_stride, a_log, dt_bias, bonus, state, slot_stride, max_slots,
                        cu_tokens, state_slots, out, heads, kv_rep, D, Dv, tail_src, tail_src_stride, tail_off, tail_rows,
                        tail_width, err};
     dim3 grid(num_reqs, heads, tiles);
 #define RS_LAUNCH(NS, DG) \
     do { if (mode == RS_DELTA) airun_launch(recurrent_state_kernel<RS_DELTA, NS, DG>, grid, dim3(128), 0, stream, a); \
+         else if (mode == RS_DELTA_HEAD) airun_launch(recurrent_state_kernel<RS_DELTA_HEAD, NS, DG>, grid, dim3(128), 0, stream, a); \
          else airun_launch(recurrent_state_kernel<RS_WKV, NS, DG>, grid, dim3(128), 0, stream, a); } while (0)
     if (D <= 16) RS_LAUNCH(4, 4);
     else if (D <= 32) RS_LAUNCH(8, 4);

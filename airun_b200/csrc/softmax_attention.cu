@@ -14,6 +14,11 @@
 // temperature, scores, the softmax and the sum over keys are float32; q, keys and values are stored in the type of
 // the cache.  A page holds, for `page_size` tokens, the keys of all KV heads ([kv_heads][page_size][D]) followed by
 // the values ([kv_heads][page_size][Dv]).
+//
+// `one_row`: the values are the keys before their rotation (v = k as projected, Dv = D, no value columns in proj).
+// Rotation changes the first r dimensions only, so ONE cached row of D + r elements serves as both:
+//     [ rotated 0..r-1 | unrotated r..D-1 | unrotated 0..r-1 ]      key = elements 0..D-1, value = elements r..D+r-1
+// (a page is [kv_heads][page_size][D + r]).  A value, and so an output, holds its dimensions in the order r..D-1, 0..r-1.
 #include "common.cuh"
 
 #define XA_MAX_PER_LANE 8     // D <= 256 and Dv <= 256
@@ -39,7 +44,7 @@ __global__ __launch_bounds__(32 * XA_PREP_WARPS) void qkv_prepare_kernel(
     const int32_t* __restrict__ rope_positions, float temp_coef, int temp_every, T* __restrict__ q_out, T* __restrict__ pool,
     const int32_t* __restrict__ block_table, int max_blocks, const int32_t* __restrict__ positions,
     const int32_t* __restrict__ req_of_token, int num_reqs, int num_pages, int page_size, int nh, int nkv, int D, int Dv,
-    int store, int* __restrict__ err) {
+    int store, int one_row, int* __restrict__ err) {
     pdl_trigger();
     pdl_wait();
     __shared__ float s_x[XA_PREP_WARPS][32 * XA_MAX_PER_LANE];
@@ -61,11 +66,12 @@ __global__ __launch_bounds__(32 * XA_PREP_WARPS) void qkv_prepare_kernel(
             if (threadIdx.x == 0) atomicOr(err, AIRUN_DEV_BAD_PAGE);
             store = 0;
         } else {
-            pk = pool + (size_t)page * nkv * page_size * (D + Dv);
+            pk = pool + (size_t)page * nkv * page_size * (one_row ? D + rdim : D + Dv);
             pv = pk + (size_t)nkv * page_size * D;
         }
     }
     const float* row = proj + (size_t)t * proj_stride;
+    const int krow = one_row ? D + rdim : D;              // elements from one token's key to the next
     const float rpos = (float)(rope_positions ? rope_positions[t] : pos);
     // the angles are the same for every head of the token: one sine and cosine per rotated pair, worked out once
     __shared__ float s_cos[16 * XA_MAX_PER_LANE], s_sin[16 * XA_MAX_PER_LANE];
@@ -77,8 +83,12 @@ __global__ __launch_bounds__(32 * XA_PREP_WARPS) void qkv_prepare_kernel(
     float* sx = s_x[warp];
     // Head sizes in multiples of four on 16-byte boundaries: a lane takes four neighbouring dimensions (eight for heads
     // above 128) with one load each, so both dimensions of a rotated pair (2i, 2i + 1) lie in the lane that turns them.
+    // Pairs (i, i + r/2) with r in multiples of eight and heads up to 128: the other halves come from the lane r/8 away.
+    const int half4 = rdim >> 3;                          // lanes between the two halves of a pair
+    const bool neox4 = rope_kind == XA_ROPE_NEOX && (rdim & 7) == 0 && D <= 128;
     const bool vec4 = (D & 3) == 0 && (proj_stride & 3) == 0 && ((uintptr_t)proj & 15) == 0 && (!bias || ((uintptr_t)bias & 15) == 0) &&
-                      ((uintptr_t)q_out & 15) == 0 && (!store || ((uintptr_t)pool & 15) == 0) && rope_kind != XA_ROPE_NEOX &&
+                      ((uintptr_t)q_out & 15) == 0 && (!store || ((uintptr_t)pool & 15) == 0) && (rope_kind != XA_ROPE_NEOX || neox4) &&
+                      (!one_row || (rdim & 3) == 0) &&
                       (!q_w || ((uintptr_t)q_w & 15) == 0) && (!k_w || ((uintptr_t)k_w & 15) == 0);
     if (vec4) {
         for (int u = warp; u < units; u += XA_PREP_WARPS) {
@@ -111,6 +121,25 @@ __global__ __launch_bounds__(32 * XA_PREP_WARPS) void qkv_prepare_kernel(
                     }
                 }
             }
+            if (one_row && !is_q && 4 * lane < rdim)       // the rotated dimensions once more, as they are (lane and lane + 32)
+                xa_store4(pk + ((size_t)(u - nh) * page_size + slot) * krow + D + 4 * lane, x[0]);
+            if (one_row && !is_q && 4 * lane + 128 < rdim)
+                xa_store4(pk + ((size_t)(u - nh) * page_size + slot) * krow + D + 4 * lane + 128, x[1]);
+            if (neox4) {
+                const bool first = lane < half4;
+                const int other = first ? lane + half4 : lane - half4;
+                float4 o;
+                o.x = __shfl_sync(0xffffffffu, x[0].x, other & 31); o.y = __shfl_sync(0xffffffffu, x[0].y, other & 31);
+                o.z = __shfl_sync(0xffffffffu, x[0].z, other & 31); o.w = __shfl_sync(0xffffffffu, x[0].w, other & 31);
+                if (4 * lane < rdim) {
+                    const int pair = 4 * (first ? lane : lane - half4);
+                    const float sg = first ? -1.0f : 1.0f;
+                    x[0].x = x[0].x * s_cos[pair] + sg * o.x * s_sin[pair];
+                    x[0].y = x[0].y * s_cos[pair + 1] + sg * o.y * s_sin[pair + 1];
+                    x[0].z = x[0].z * s_cos[pair + 2] + sg * o.z * s_sin[pair + 2];
+                    x[0].w = x[0].w * s_cos[pair + 3] + sg * o.w * s_sin[pair + 3];
+                }
+            }
             if (rope_kind == XA_ROPE_INTERLEAVED) {
 #pragma unroll
                 for (int i = 0; i < 2; ++i) {
@@ -138,14 +167,14 @@ __global__ __launch_bounds__(32 * XA_PREP_WARPS) void qkv_prepare_kernel(
 #pragma unroll
                 for (int i = 0; i < 2; ++i) { x[i].x *= inv; x[i].y *= inv; x[i].z *= inv; x[i].w *= inv; }
             }
-            T* dst = is_q ? q_out + ((size_t)t * nh + u) * D : pk + ((size_t)(u - nh) * page_size + slot) * D;
+            T* dst = is_q ? q_out + ((size_t)t * nh + u) * D : pk + ((size_t)(u - nh) * page_size + slot) * krow;
 #pragma unroll
             for (int i = 0; i < 2; ++i) {
                 const int d = 4 * lane + 128 * i;
                 if (d < D) xa_store4(dst + d, make_float4(x[i].x * mulv, x[i].y * mulv, x[i].z * mulv, x[i].w * mulv));
             }
         }
-        if (!store) return;
+        if (!store || one_row) return;
         const int vcol = (nh + nkv) * D;
         if ((Dv & 3) == 0) {
             for (int c = threadIdx.x; c < (nkv * Dv) >> 2; c += blockDim.x) {
@@ -185,6 +214,14 @@ __global__ __launch_bounds__(32 * XA_PREP_WARPS) void qkv_prepare_kernel(
                 if (d < D) x[i] = x[i] * inv * w[d];
             }
         }
+        if (one_row && !is_q) {
+            T* dst = pk + ((size_t)(u - nh) * page_size + slot) * krow + D;
+#pragma unroll
+            for (int i = 0; i < XA_MAX_PER_LANE; ++i) {
+                const int d = lane + 32 * i;
+                if (d < rdim) dst[d] = from_f32<T>(x[i]);
+            }
+        }
         if (rope_kind != XA_ROPE_NONE && rdim > 0) {
             __syncwarp();
 #pragma unroll
@@ -220,7 +257,7 @@ __global__ __launch_bounds__(32 * XA_PREP_WARPS) void qkv_prepare_kernel(
                 if (d < D) dst[d] = from_f32<T>(x[i] * temp);
             }
         } else {
-            T* dst = pk + ((size_t)(u - nh) * page_size + slot) * D;
+            T* dst = pk + ((size_t)(u - nh) * page_size + slot) * krow;
 #pragma unroll
             for (int i = 0; i < XA_MAX_PER_LANE; ++i) {
                 const int d = lane + 32 * i;
@@ -228,7 +265,7 @@ __global__ __launch_bounds__(32 * XA_PREP_WARPS) void qkv_prepare_kernel(
             }
         }
     }
-    if (!store) return;
+    if (!store || one_row) return;
     const int vcol0 = (nh + nkv) * D;
     for (int c = threadIdx.x; c < nkv * Dv; c += blockDim.x) {
         const int g = c / Dv, e = c - g * Dv;
@@ -241,16 +278,17 @@ AIRUN_EXPORT int airun_qkv_prepare(const float* proj, long long proj_stride, con
                                    const int32_t* rope_positions, float temp_coef, int temp_every, void* q_out, void* pool,
                                    int dtype, const int32_t* block_table, int max_blocks, const int32_t* positions,
                                    const int32_t* req_of_token, int T, int num_reqs, int num_pages, int page_size, int nh,
-                                   int nkv, int D, int Dv, int store, int* err, cudaStream_t stream) {
+                                   int nkv, int D, int Dv, int store, int one_row, int* err, cudaStream_t stream) {
     if (T < 0 || nh <= 0 || nkv <= 0 || D <= 0 || D > 32 * XA_MAX_PER_LANE || Dv <= 0 || temp_every < 0 || !err || !positions ||
         !req_of_token || !proj || !q_out || rdim < 0 || rdim > D || (rdim & 1) ||
         (rope_kind != XA_ROPE_NONE && rdim > 0 && !inv_freq) || rope_kind < 0 || rope_kind > 2 ||
+        (one_row && (Dv != D || k_w || unit_norm || (rope_kind == XA_ROPE_NONE && rdim > 0))) ||
         (store && (!pool || !block_table || page_size <= 0 || num_pages <= 0 || max_blocks <= 0)))
         return AIRUN_ERR_ARG;
     if (T == 0) return AIRUN_OK;
 #define XP_LAUNCH(TT) airun_launch(qkv_prepare_kernel<TT>, dim3(T), dim3(32 * XA_PREP_WARPS), 0, stream, proj, proj_stride, bias, q_w, \
         k_w, unit_norm, eps, rope_kind, rdim, inv_freq, rope_positions, temp_coef, temp_every, (TT*)q_out, (TT*)pool, block_table, \
-        max_blocks, positions, req_of_token, num_reqs, num_pages, page_size, nh, nkv, D, Dv, store, err)
+        max_blocks, positions, req_of_token, num_reqs, num_pages, page_size, nh, nkv, D, Dv, store, one_row, err)
     if (dtype == AIRUN_DT_F32) XP_LAUNCH(float);
     else if (dtype == AIRUN_DT_BF16) XP_LAUNCH(__nv_bfloat16);
     else return AIRUN_ERR_UNSUPPORTED;
@@ -267,7 +305,7 @@ __global__ __launch_bounds__(32 * XA_WARPS) void softmax_attention_kernel(
     const int32_t* __restrict__ block_table, int max_blocks, const int32_t* __restrict__ positions,
     const int32_t* __restrict__ req_of_token, int num_reqs, int num_pages, int page_size, int nh, int nkv, int D, int Dv,
     float scale, const float* __restrict__ table, int table_len, const float* __restrict__ sink, int window, float out_scale,
-    int* __restrict__ err) {
+    int tail, int* __restrict__ err) {
     pdl_trigger();
     pdl_wait();
     extern __shared__ float s_acc[];           // [XA_WARPS][Dv], then [XA_WARPS] maxima and [XA_WARPS] sums
@@ -295,15 +333,18 @@ __global__ __launch_bounds__(32 * XA_WARPS) void softmax_attention_kernel(
     const int32_t* bt = block_table + (size_t)req * max_blocks;
     const int begin = window > 0 ? max(0, pos - window + 1) : 0;
     bool bad = false;
-    const size_t page_elems = (size_t)nkv * page_size * (D + Dv);
+    // one row for key and value (`tail` >= 0): rows of D + tail elements, the value begins `tail` elements into its row
+    const int krow = tail >= 0 ? D + tail : D, vrow = tail >= 0 ? D + tail : Dv;
+    const size_t page_elems = (size_t)nkv * page_size * (tail >= 0 ? D + tail : D + Dv);
+    const size_t v_off = tail >= 0 ? (size_t)tail : (size_t)nkv * page_size * D;
     float m = -INFINITY, l = 0.0f;
     for (int j = begin + warp; j <= pos; j += XA_WARPS) {
         const int blk = j / page_size;
         const int page = blk < max_blocks ? bt[blk] : -1;
         if (page < 0 || page >= num_pages) { bad = true; continue; }
         const T* pk = pool + (size_t)page * page_elems;
-        const T* kj = pk + ((size_t)kvh * page_size + (j - blk * page_size)) * D;
-        const T* vj = pk + (size_t)nkv * page_size * D + ((size_t)kvh * page_size + (j - blk * page_size)) * Dv;
+        const T* kj = pk + ((size_t)kvh * page_size + (j - blk * page_size)) * krow;
+        const T* vj = pk + v_off + ((size_t)kvh * page_size + (j - blk * page_size)) * vrow;
         float dot = 0.0f;
 #pragma unroll
         for (int i = 0; i < XA_MAX_PER_LANE; ++i) {
@@ -353,17 +394,17 @@ AIRUN_EXPORT int airun_softmax_attention(const void* q, void* out, long long out
                                          const int32_t* block_table, int max_blocks, const int32_t* positions,
                                          const int32_t* req_of_token, int T, int num_reqs, int num_pages, int page_size,
                                          int nh, int nkv, int D, int Dv, float scale, const float* table, int table_len,
-                                         const float* sink, int window, float out_scale, int* err, cudaStream_t stream) {
+                                         const float* sink, int window, float out_scale, int tail, int* err, cudaStream_t stream) {
     if (T < 0 || nh <= 0 || nkv <= 0 || nh % nkv != 0 || D <= 0 || D > 32 * XA_MAX_PER_LANE || Dv <= 0 ||
         Dv > 32 * XA_MAX_PER_LANE || page_size <= 0 || num_pages <= 0 || max_blocks <= 0 || window < 0 || !err || nh > 65535 ||
-        out_stride < (long long)nh * Dv || (table && table_len <= 0))
+        out_stride < (long long)nh * Dv || (table && table_len <= 0) || tail > D || (tail >= 0 && Dv != D))
         return AIRUN_ERR_ARG;
     if (T == 0) return AIRUN_OK;
     dim3 grid(T, nh);
     const size_t smem = ((size_t)XA_WARPS * Dv + 2 * XA_WARPS) * sizeof(float);
 #define XA_LAUNCH(TT) airun_launch(softmax_attention_kernel<TT>, grid, dim3(32 * XA_WARPS), smem, stream, (const TT*)q, (TT*)out, \
         out_stride, (const TT*)pool, block_table, max_blocks, positions, req_of_token, num_reqs, num_pages, page_size, nh, nkv, D, Dv, \
-        scale, table, table_len, sink, window, out_scale, err)
+        scale, table, table_len, sink, window, out_scale, tail, err)
     if (dtype == AIRUN_DT_F32) XA_LAUNCH(float);
     else if (dtype == AIRUN_DT_BF16) XA_LAUNCH(__nv_bfloat16);
     else return AIRUN_ERR_UNSUPPORTED;

@@ -12,6 +12,11 @@
 // head, and the distance i - j of an element depends on (row - column) alone: the 127 table entries a key tile can
 // need are copied once, by one thread each, into shared memory.
 //
+// Keys that serve as values (`tail` >= 0, see softmax_attention.cu: one cached row of D + tail elements, the value being
+// its elements tail .. tail + D - 1) are copied ONCE: the instances with ONE keep rows of up to 2 DP elements in the key
+// stage and read the values out of them, `tail` elements further on.  (That takes D and tail in multiples of 8; other
+// sizes copy the two halves element by element, the values behind the padded key.)
+//
 // D and Dv are padded to the template sizes DP and DVP with zeros in shared memory, so any D, Dv up to 128 run.  A
 // token's result does not depend on the other rows of its tile or on the batch: its keys are walked in tiles that
 // begin at the first key its TILE can see, so the same token in another portion meets other tile borders, which moves
@@ -99,6 +104,7 @@ struct XamParams {
     const float* sink;            // [nh]: exp(sink) joins the denominator; null: no sink
     float out_scale;
     int window;
+    int tail;                     // one row for key and value: elements before the value begins; -1: rows of their own
     int skip_single;              // requests that bring ONE token are left to the kernel for single tokens
     float* partial;               // [splits][T][nh * (Dv + 2)] float32 (sums, then maximum and denominator per head), when the keys of a single token are cut over CTAs
     int splits, T;
@@ -109,7 +115,7 @@ struct XamParams {
 // are asynchronous 16-byte pieces; when those pieces divide the CTA's 128 threads evenly and pages are a power of
 // two, a thread owns one piece (where it lies in the page and in shared memory) for every key it copies, so that a
 // copy costs a page lookup and little else.  Rows beyond the last key keep what they held: their weights are zero.
-template <int KS, int VS>
+template <int KS, int VS, bool ONE>
 struct XamLoader {
     const XamParams& p;
     const int32_t* bt;
@@ -119,10 +125,10 @@ struct XamLoader {
     size_t page_elems, src;
     __device__ XamLoader(const XamParams& p_, const int32_t* bt_, int kvh_) : p(p_), bt(bt_), kvh(kvh_), tid(threadIdx.x), bad(false) {
         const int D = p.D, Dv = p.Dv;
-        vec = (D % 8 == 0) && (Dv % 8 == 0);
-        page_elems = (size_t)p.nkv * p.page_size * (D + Dv);
+        vec = (D % 8 == 0) && (Dv % 8 == 0) && (!ONE || p.tail % 8 == 0);
+        page_elems = (size_t)p.nkv * p.page_size * (ONE ? D + p.tail : D + Dv);
         const int lp = max(1, D / 8 + Dv / 8);
-        regular = vec && lp <= 128 && 128 % lp == 0 && (p.page_size & (p.page_size - 1)) == 0;
+        regular = !ONE && vec && lp <= 128 && 128 % lp == 0 && (p.page_size & (p.page_size - 1)) == 0;
         ps_shift = __ffs(p.page_size) - 1;
         const int u = tid % lp;
         key0 = tid / lp; step = 128 / lp;
@@ -153,9 +159,9 @@ struct XamLoader {
             const int j = kbase + key, blk = j / p.page_size;
             const int page = blk < p.max_blocks ? bt[blk] : -1;
             if (page < 0 || page >= p.num_pages) { bad = true; continue; }
-            const __nv_bfloat16* pk = p.pool + (size_t)page * page_elems + ((size_t)kvh * p.page_size + (j - blk * p.page_size)) * D;
-            const __nv_bfloat16* pv = p.pool + (size_t)page * page_elems + (size_t)p.nkv * p.page_size * D +
-                                      ((size_t)kvh * p.page_size + (j - blk * p.page_size)) * Dv;
+            const size_t at = (size_t)kvh * p.page_size + (j - blk * p.page_size);
+            const __nv_bfloat16* pk = p.pool + (size_t)page * page_elems + at * (ONE ? D + p.tail : D);
+            const __nv_bfloat16* pv = ONE ? pk + p.tail : p.pool + (size_t)page * page_elems + (size_t)p.nkv * p.page_size * D + at * Dv;
             if (vec) {
                 if (u < perk) xam_cp16(Ks + key * KS + u * 8, pk + u * 8);
                 else xam_cp16(Vs + key * VS + (u - perk) * 8, pv + (u - perk) * 8);
@@ -178,16 +184,18 @@ struct XamLoader {
 // stage's mbarrier, on which every thread arrives with the bytes it has asked for, completes when all of them have
 // landed.  (Sixteen-byte cp.async pieces, sixteen a thread and tile, held all four warps up for as long as the copy
 // took to be accepted: copies and products ran one after the other.)  Other head sizes are copied element by element.
-template <int DP, int DVP>
+template <int DP, int DVP, bool ONE>
 __global__ __launch_bounds__(128) void softmax_attention_mma_kernel(const XamParams p) {
     pdl_trigger();
     pdl_wait();
-    constexpr int QS = DP + XAM_PAD, VS = DVP + XAM_PAD;
+    constexpr int QS = DP + XAM_PAD, KS = ONE ? 2 * DP + XAM_PAD : QS, VS = ONE ? KS : DVP + XAM_PAD;
+    constexpr int STAGES = 2 * XAM_KEYS * (ONE ? KS : KS + VS);                // elements of both stages
     extern __shared__ __align__(16) unsigned char xam_smem[];
     __nv_bfloat16* Qs = reinterpret_cast<__nv_bfloat16*>(xam_smem);            // [64][QS]
-    __nv_bfloat16* Ks0 = Qs + XAM_ROWS * QS;                                   // [2][64][QS]
-    __nv_bfloat16* Vs0 = Ks0 + 2 * XAM_KEYS * QS;                              // [2][64][VS]
-    float* tab = reinterpret_cast<float*>(Vs0 + 2 * XAM_KEYS * VS);            // [128]: log2(e) * table[d] by row - column + 63
+    __nv_bfloat16* Ks0 = Qs + XAM_ROWS * QS;                                   // [2][64][KS]
+    // [2][64][VS]; in ONE the values lie in the key stage: `tail` elements on, or behind the padded key when copied apart
+    __nv_bfloat16* Vs0 = ONE ? Ks0 + (p.D % 8 == 0 && p.tail % 8 == 0 ? p.tail : DP) : Ks0 + 2 * XAM_KEYS * KS;
+    float* tab = reinterpret_cast<float*>(Ks0 + STAGES);                       // [128]: log2(e) * table[d] by row - column + 63
     const uint32_t bar0 = xam_u32(tab + 128);                                  // two mbarriers, one a stage
     // ---- which tile (tiles later in a request see more keys: the grid is walked from its end so that they start first)
     int b = gridDim.y - 1 - blockIdx.y, req = -1, first = 0, n = 0, p0 = 0;
@@ -206,10 +214,10 @@ __global__ __launch_bounds__(128) void softmax_attention_mma_kernel(const XamPar
     const int head = blockIdx.x, kvh = head / (p.nh / p.nkv);
     const int D = p.D, Dv = p.Dv;
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3;
-    XamLoader<QS, VS> ld(p, p.block_table + (size_t)req * p.max_blocks, kvh);
+    XamLoader<KS, VS, ONE> ld(p, p.block_table + (size_t)req * p.max_blocks, kvh);
     // ---- shared memory starts as zeros (the padding beyond D and Dv stays so), then the Q tile
     {
-        constexpr int WORDS16 = (3 * XAM_ROWS * QS + 2 * XAM_KEYS * VS) / 8 + 128 * 4 / 16;
+        constexpr int WORDS16 = (XAM_ROWS * QS + STAGES) / 8 + 128 * 4 / 16;
         uint4* z = reinterpret_cast<uint4*>(xam_smem);
         for (int e = tid; e < WORDS16; e += 128) z[e] = make_uint4(0u, 0u, 0u, 0u);
     }
@@ -254,30 +262,31 @@ __global__ __launch_bounds__(128) void softmax_attention_mma_kernel(const XamPar
     const float* table = has_dist ? p.table + (size_t)head * p.table_len : nullptr;
     const float mul = p.scale * XAM_LOG2E;                 // scores are kept as log2 of the weights
     float m_run[2] = {-INFINITY, -INFINITY}, l_run[2] = {0.0f, 0.0f};      // running maximum and this thread's part of the sum, per row
-    // this thread's row of a tile: K of key tid (threads 0-63) or V of key tid - 64
+    // this thread's row of a tile: K of key tid (threads 0-63) or V of key tid - 64 (nothing when the key's row is the value's too)
     const bool row_k = tid < XAM_KEYS;
     const int row_key = tid & (XAM_KEYS - 1);
-    const uint32_t row_bytes = (uint32_t)(row_k ? D : Dv) * 2u;
-    const size_t row_off = row_k ? (size_t)kvh * p.page_size * D : (size_t)p.nkv * p.page_size * D + (size_t)kvh * p.page_size * Dv;
-    const size_t page_elems = (size_t)p.nkv * p.page_size * (D + Dv);
+    const int row_elems = ONE ? D + p.tail : row_k ? D : Dv;
+    const uint32_t row_bytes = (uint32_t)row_elems * 2u;
+    const size_t row_off = row_k ? (size_t)kvh * p.page_size * row_elems : (size_t)p.nkv * p.page_size * D + (size_t)kvh * p.page_size * Dv;
+    const size_t page_elems = (size_t)p.nkv * p.page_size * (ONE ? row_elems : D + Dv);
     const int32_t* bt = p.block_table + (size_t)req * p.max_blocks;
     bool bad_page = false, gave_up = false;
     auto fill = [&](int kbase, int stage) {                // asks for the tile that begins at key kbase
         if (!bulk) {
-            ld.load(kbase, hi, Ks0 + stage * XAM_KEYS * QS, Vs0 + stage * XAM_KEYS * VS);
+            ld.load(kbase, hi, Ks0 + stage * XAM_KEYS * KS, Vs0 + stage * XAM_KEYS * VS);
             return;
         }
         const int j = kbase + row_key, blk = j / p.page_size;
         const int page = (j <= hi && blk < p.max_blocks) ? bt[blk] : -1;
-        if (j > hi) {
+        if (j > hi || (ONE && !row_k)) {
             xam_mbar_arrive(bar0 + 8 * stage);
         } else if (page < 0 || page >= p.num_pages) {
             bad_page = true;
             xam_mbar_arrive(bar0 + 8 * stage);
         } else {
             xam_mbar_arrive_tx(bar0 + 8 * stage, row_bytes);
-            __nv_bfloat16* dst = row_k ? Ks0 + (stage * XAM_KEYS + row_key) * QS : Vs0 + (stage * XAM_KEYS + row_key) * VS;
-            xam_bulk_row(dst, p.pool + (size_t)page * page_elems + row_off + (size_t)(j - blk * p.page_size) * (row_k ? D : Dv),
+            __nv_bfloat16* dst = row_k ? Ks0 + (stage * XAM_KEYS + row_key) * KS : Vs0 + (stage * XAM_KEYS + row_key) * VS;
+            xam_bulk_row(dst, p.pool + (size_t)page * page_elems + row_off + (size_t)(j - blk * p.page_size) * row_elems,
                          row_bytes, bar0 + 8 * stage);
         }
     };
@@ -285,7 +294,7 @@ __global__ __launch_bounds__(128) void softmax_attention_mma_kernel(const XamPar
     int it = 0;
     for (int kbase = lo; kbase <= hi; kbase += XAM_KEYS, ++it) {
         const int buf = it & 1;
-        const __nv_bfloat16* Ks = Ks0 + buf * XAM_KEYS * QS;
+        const __nv_bfloat16* Ks = Ks0 + buf * XAM_KEYS * KS;
         const __nv_bfloat16* Vs = Vs0 + buf * XAM_KEYS * VS;
         if (kbase + XAM_KEYS <= hi) fill(kbase + XAM_KEYS, buf ^ 1);
         bool landed = true;
@@ -318,7 +327,7 @@ __global__ __launch_bounds__(128) void softmax_attention_mma_kernel(const XamPar
                 a[3] = *reinterpret_cast<const uint32_t*>(qa + 8 * QS + 8);
 #pragma unroll
                 for (int nt = 0; nt < XAM_KEYS / 8; ++nt) {
-                    const __nv_bfloat16* kb = Ks + (nt * 8 + g) * QS + ks * 16 + 2 * t;
+                    const __nv_bfloat16* kb = Ks + (nt * 8 + g) * KS + ks * 16 + 2 * t;
                     xam_mma(S[nt], a, *reinterpret_cast<const uint32_t*>(kb), *reinterpret_cast<const uint32_t*>(kb + 8));
                 }
             }
@@ -420,31 +429,32 @@ __global__ __launch_bounds__(128) void softmax_attention_mma_kernel(const XamPar
 // their common maximum and added through shared memory in warp order.  With one slice the result (with the sink, the
 // division and the factor) goes to `out`; with several each slice writes its float32 sums, its maximum and its
 // denominator to `partial` ([splits][T][nh * (Dv + 2)]) and xam_reduce_kernel merges them in slice order.
-template <int DP, int DVP>
+template <int DP, int DVP, bool ONE>
 __global__ __launch_bounds__(128) void softmax_attention_group_kernel(const XamParams p) {
     pdl_trigger();
     pdl_wait();
-    constexpr int QS = DP + XAM_PAD, VS = DVP + XAM_PAD;
+    constexpr int QS = DP + XAM_PAD, KS = ONE ? 2 * DP + XAM_PAD : QS, VS = ONE ? KS : DVP + XAM_PAD;
+    constexpr int STAGES = 2 * XAM_KEYS * (ONE ? KS : KS + VS);
     constexpr int PER = DVP / 8 * 4 + 1;                   // floats a thread hands to the merge (odd: no bank conflicts)
     extern __shared__ __align__(16) unsigned char xam_smem[];
     __nv_bfloat16* Qs = reinterpret_cast<__nv_bfloat16*>(xam_smem);            // [16][QS]
-    __nv_bfloat16* Ks0 = Qs + 16 * QS;                                         // [2][64][QS]
-    __nv_bfloat16* Vs0 = Ks0 + 2 * XAM_KEYS * QS;                              // [2][64][VS]
+    __nv_bfloat16* Ks0 = Qs + 16 * QS;                                         // [2][64][KS]
+    __nv_bfloat16* Vs0 = ONE ? Ks0 + (p.D % 8 == 0 && p.tail % 8 == 0 ? p.tail : DP) : Ks0 + 2 * XAM_KEYS * KS;      // [2][64][VS]
     const int r = blockIdx.y, kvh = blockIdx.x, slice = blockIdx.z;
     const int tok = p.cu_tokens[r];
     if (p.cu_tokens[r + 1] - tok != 1) return;
     const int pos = p.context_lens[r] - 1;                 // the token's position: the last key it sees
     const int D = p.D, Dv = p.Dv, G = p.nh / p.nkv;
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3;
-    XamLoader<QS, VS> ld(p, p.block_table + (size_t)r * p.max_blocks, kvh);
+    XamLoader<KS, VS, ONE> ld(p, p.block_table + (size_t)r * p.max_blocks, kvh);
     {
-        constexpr int WORDS16 = ((16 + 2 * XAM_KEYS) * QS + 2 * XAM_KEYS * VS) / 8;
+        constexpr int WORDS16 = (16 * QS + STAGES) / 8;
         uint4* z = reinterpret_cast<uint4*>(xam_smem);
         for (int e = tid; e < WORDS16; e += 128) z[e] = make_uint4(0u, 0u, 0u, 0u);
     }
     // the stages are filled by bulk copies, a row a thread, as in the tile kernel (head sizes in multiples of 8)
     const bool bulk = ld.vec;
-    const uint32_t bar0 = xam_u32(Vs0 + 2 * XAM_KEYS * VS);                    // two mbarriers behind the stages
+    const uint32_t bar0 = xam_u32(Ks0 + STAGES);                               // two mbarriers behind the stages
     if (bulk) {
         if (tid == 0) {
             xam_mbar_init(bar0, 128);
@@ -488,27 +498,28 @@ __global__ __launch_bounds__(128) void softmax_attention_group_kernel(const XamP
         for (int j = 0; j < 4; ++j) O[i][j] = 0.0f;
     const bool row_k = tid < XAM_KEYS;
     const int row_key = tid & (XAM_KEYS - 1);
-    const uint32_t row_bytes = (uint32_t)(row_k ? D : Dv) * 2u;
-    const size_t row_off = row_k ? (size_t)kvh * p.page_size * D : (size_t)p.nkv * p.page_size * D + (size_t)kvh * p.page_size * Dv;
-    const size_t page_elems = (size_t)p.nkv * p.page_size * (D + Dv);
+    const int row_elems = ONE ? D + p.tail : row_k ? D : Dv;
+    const uint32_t row_bytes = (uint32_t)row_elems * 2u;
+    const size_t row_off = row_k ? (size_t)kvh * p.page_size * row_elems : (size_t)p.nkv * p.page_size * D + (size_t)kvh * p.page_size * Dv;
+    const size_t page_elems = (size_t)p.nkv * p.page_size * (ONE ? row_elems : D + Dv);
     const int32_t* bt = p.block_table + (size_t)r * p.max_blocks;
     bool bad_page = false, gave_up = false;
     auto fill = [&](int kbase, int stage) {
         if (!bulk) {
-            ld.load(kbase, hi, Ks0 + stage * XAM_KEYS * QS, Vs0 + stage * XAM_KEYS * VS);
+            ld.load(kbase, hi, Ks0 + stage * XAM_KEYS * KS, Vs0 + stage * XAM_KEYS * VS);
             return;
         }
         const int j = kbase + row_key, blk = j / p.page_size;
         const int page = (j <= hi && blk < p.max_blocks) ? bt[blk] : -1;
-        if (j > hi) {
+        if (j > hi || (ONE && !row_k)) {
             xam_mbar_arrive(bar0 + 8 * stage);
         } else if (page < 0 || page >= p.num_pages) {
             bad_page = true;
             xam_mbar_arrive(bar0 + 8 * stage);
         } else {
             xam_mbar_arrive_tx(bar0 + 8 * stage, row_bytes);
-            __nv_bfloat16* dst = row_k ? Ks0 + (stage * XAM_KEYS + row_key) * QS : Vs0 + (stage * XAM_KEYS + row_key) * VS;
-            xam_bulk_row(dst, p.pool + (size_t)page * page_elems + row_off + (size_t)(j - blk * p.page_size) * (row_k ? D : Dv),
+            __nv_bfloat16* dst = row_k ? Ks0 + (stage * XAM_KEYS + row_key) * KS : Vs0 + (stage * XAM_KEYS + row_key) * VS;
+            xam_bulk_row(dst, p.pool + (size_t)page * page_elems + row_off + (size_t)(j - blk * p.page_size) * row_elems,
                          row_bytes, bar0 + 8 * stage);
         }
     };
@@ -519,7 +530,7 @@ __global__ __launch_bounds__(128) void softmax_attention_group_kernel(const XamP
     int it = 0;
     for (int kbase = lo; kbase <= hi; kbase += XAM_KEYS, ++it) {
         const int buf = it & 1;
-        const __nv_bfloat16* Ks = Ks0 + buf * XAM_KEYS * QS;
+        const __nv_bfloat16* Ks = Ks0 + buf * XAM_KEYS * KS;
         const __nv_bfloat16* Vs = Vs0 + buf * XAM_KEYS * VS;
         if (kbase + XAM_KEYS <= hi) fill(kbase + XAM_KEYS, buf ^ 1);
         bool landed = true;
@@ -548,7 +559,7 @@ __global__ __launch_bounds__(128) void softmax_attention_group_kernel(const XamP
                 a[3] = *reinterpret_cast<const uint32_t*>(qa + 8 * QS + 8);
 #pragma unroll
                 for (int nt = 0; nt < 2; ++nt) {
-                    const __nv_bfloat16* kb = Ks + (16 * warp + nt * 8 + g) * QS + ks * 16 + 2 * t;
+                    const __nv_bfloat16* kb = Ks + (16 * warp + nt * 8 + g) * KS + ks * 16 + 2 * t;
                     xam_mma(S[nt], a, *reinterpret_cast<const uint32_t*>(kb), *reinterpret_cast<const uint32_t*>(kb + 8));
                 }
             }
@@ -716,40 +727,43 @@ __global__ __launch_bounds__(256) void xam_reduce_kernel(const XamParams p) {
     }
 }
 
-template <int DP, int DVP>
+template <int DP, int DVP, bool ONE>
 static int xag_launch(const XamParams& p, cudaStream_t stream) {
-    const size_t tiles = (size_t)((16 + 2 * XAM_KEYS) * (DP + XAM_PAD) + 2 * XAM_KEYS * (DVP + XAM_PAD)) * sizeof(__nv_bfloat16) + 16;
+    const size_t stages = 2 * XAM_KEYS * (ONE ? 2 * DP + XAM_PAD : DP + DVP + 2 * XAM_PAD);
+    const size_t tiles = (16 * (DP + XAM_PAD) + stages) * sizeof(__nv_bfloat16) + 16;
     const size_t merge = (size_t)128 * (DVP / 8 * 4 + 1) * sizeof(float) + 128 * sizeof(float);
     const size_t smem = tiles > merge ? tiles : merge;
     static unsigned long long configured = 0;
     if (smem > 48 * 1024 && first_on_device(configured)) {
-        cudaError_t e = cudaFuncSetAttribute(softmax_attention_group_kernel<DP, DVP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        cudaError_t e = cudaFuncSetAttribute(softmax_attention_group_kernel<DP, DVP, ONE>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) return (int)e;
     }
-    airun_launch(softmax_attention_group_kernel<DP, DVP>, dim3(p.nkv, p.num_reqs, p.splits), dim3(128), smem, stream, p);
+    airun_launch(softmax_attention_group_kernel<DP, DVP, ONE>, dim3(p.nkv, p.num_reqs, p.splits), dim3(128), smem, stream, p);
     int rc = airun_launch_status();
     if (rc != AIRUN_OK || p.splits <= 1) return rc;
     airun_launch(xam_reduce_kernel, dim3(p.num_reqs), dim3(256), 0, stream, p);
     return airun_launch_status();
 }
 
-template <int DP, int DVP>
+template <int DP, int DVP, bool ONE>
 static int xam_launch(const XamParams& p, int max_tiles, cudaStream_t stream) {
-    const size_t smem = (size_t)(3 * XAM_ROWS * (DP + XAM_PAD) + 2 * XAM_KEYS * (DVP + XAM_PAD)) * sizeof(__nv_bfloat16) + 128 * sizeof(float) + 16;
+    const size_t stages = 2 * XAM_KEYS * (ONE ? 2 * DP + XAM_PAD : DP + DVP + 2 * XAM_PAD);
+    const size_t smem = (XAM_ROWS * (DP + XAM_PAD) + stages) * sizeof(__nv_bfloat16) + 128 * sizeof(float) + 16;
     static unsigned long long configured = 0;
     if (smem > 48 * 1024 && first_on_device(configured)) {
-        cudaError_t e = cudaFuncSetAttribute(softmax_attention_mma_kernel<DP, DVP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        cudaError_t e = cudaFuncSetAttribute(softmax_attention_mma_kernel<DP, DVP, ONE>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) return (int)e;
     }
     if (max_tiles > 65535) return AIRUN_ERR_ARG;
-    airun_launch(softmax_attention_mma_kernel<DP, DVP>, dim3(p.nh, max_tiles), dim3(128), smem, stream, p);
+    airun_launch(softmax_attention_mma_kernel<DP, DVP, ONE>, dim3(p.nh, max_tiles), dim3(128), smem, stream, p);
     return airun_launch_status();
 }
 
 static bool xam_fill(XamParams& p, const void* q, void* out, long long out_stride, const void* pool, const int32_t* block_table,
                      int max_blocks, const int32_t* cu_tokens, const int32_t* context_lens, int num_reqs, int num_pages,
                      int page_size, int nh, int nkv, int D, int Dv, float scale, const float* table, int table_len,
-                     const float* sink, int window, float out_scale, int* err) {
+                     const float* sink, int window, float out_scale, int tail, int* err) {
+    if (tail > D || (tail >= 0 && Dv != D)) return false;
     if (num_reqs < 0 || nh <= 0 || nkv <= 0 || nh % nkv != 0 || D <= 0 || D > 128 || Dv <= 0 || Dv > 128 || page_size <= 0 ||
         num_pages <= 0 || max_blocks <= 0 || window < 0 || !err || nh > 65535 || out_stride < (long long)nh * Dv || !cu_tokens ||
         !context_lens || (table && table_len <= 0))
@@ -758,22 +772,27 @@ static bool xam_fill(XamParams& p, const void* q, void* out, long long out_strid
     p.pool = (const __nv_bfloat16*)pool; p.block_table = block_table; p.max_blocks = max_blocks;
     p.cu_tokens = cu_tokens; p.context_lens = context_lens; p.num_reqs = num_reqs; p.num_pages = num_pages;
     p.page_size = page_size; p.nh = nh; p.nkv = nkv; p.D = D; p.Dv = Dv; p.scale = scale;
-    p.table = table; p.table_len = table_len; p.sink = sink; p.out_scale = out_scale; p.window = window; p.skip_single = 0;
+    p.table = table; p.table_len = table_len; p.sink = sink; p.out_scale = out_scale; p.window = window; p.tail = tail; p.skip_single = 0;
     p.partial = nullptr; p.splits = 1; p.T = 0; p.err = err;
     return true;
 }
 
 #define XAM_CASES(CALL)                                                              \
+    if (tail >= 0) {                                                                 \
+        if (D <= 32) return CALL(32, 32, true);                                      \
+        if (D <= 64) return CALL(64, 64, true);                                      \
+        return CALL(128, 128, true);                                                 \
+    }                                                                                \
     const int dp = D <= 32 ? 32 : D <= 64 ? 64 : 128, dvp = Dv <= 32 ? 32 : Dv <= 64 ? 64 : 128; \
-    if (dp == 32 && dvp == 32) return CALL(32, 32);                                  \
-    if (dp == 32 && dvp == 64) return CALL(32, 64);                                  \
-    if (dp == 32 && dvp == 128) return CALL(32, 128);                                \
-    if (dp == 64 && dvp == 32) return CALL(64, 32);                                  \
-    if (dp == 64 && dvp == 64) return CALL(64, 64);                                  \
-    if (dp == 64 && dvp == 128) return CALL(64, 128);                                \
-    if (dp == 128 && dvp == 32) return CALL(128, 32);                                \
-    if (dp == 128 && dvp == 64) return CALL(128, 64);                                \
-    if (dp == 128 && dvp == 128) return CALL(128, 128);                              \
+    if (dp == 32 && dvp == 32) return CALL(32, 32, false);                                  \
+    if (dp == 32 && dvp == 64) return CALL(32, 64, false);                                  \
+    if (dp == 32 && dvp == 128) return CALL(32, 128, false);                                \
+    if (dp == 64 && dvp == 32) return CALL(64, 32, false);                                  \
+    if (dp == 64 && dvp == 64) return CALL(64, 64, false);                                  \
+    if (dp == 64 && dvp == 128) return CALL(64, 128, false);                                \
+    if (dp == 128 && dvp == 32) return CALL(128, 32, false);                                \
+    if (dp == 128 && dvp == 64) return CALL(128, 64, false);                                \
+    if (dp == 128 && dvp == 128) return CALL(128, 128, false);                              \
     return AIRUN_ERR_UNSUPPORTED
 
 // Prompt portions (and, with skip_single == 0, single tokens too).  max_tiles: an upper bound of the number of 64-token
@@ -782,15 +801,15 @@ AIRUN_EXPORT int airun_softmax_attention_mma(const void* q, void* out, long long
                                              const int32_t* block_table, int max_blocks, const int32_t* cu_tokens,
                                              const int32_t* context_lens, int num_reqs, int max_tiles, int num_pages,
                                              int page_size, int nh, int nkv, int D, int Dv, float scale, const float* table,
-                                             int table_len, const float* sink, int window, float out_scale, int skip_single,
-                                             int* err, cudaStream_t stream) {
+                                             int table_len, const float* sink, int window, float out_scale, int tail,
+                                             int skip_single, int* err, cudaStream_t stream) {
     XamParams p;
     if (max_tiles < 0 || !xam_fill(p, q, out, out_stride, pool, block_table, max_blocks, cu_tokens, context_lens, num_reqs, num_pages,
-                                   page_size, nh, nkv, D, Dv, scale, table, table_len, sink, window, out_scale, err))
+                                   page_size, nh, nkv, D, Dv, scale, table, table_len, sink, window, out_scale, tail, err))
         return AIRUN_ERR_ARG;
     if (num_reqs == 0 || max_tiles == 0) return AIRUN_OK;
     p.skip_single = skip_single;
-#define XAM_TILE(A, B) xam_launch<A, B>(p, max_tiles, stream)
+#define XAM_TILE(A, B, ONE) xam_launch<A, B, ONE>(p, max_tiles, stream)
     XAM_CASES(XAM_TILE);
 #undef XAM_TILE
 }
@@ -801,16 +820,16 @@ AIRUN_EXPORT int airun_softmax_attention_group(const void* q, void* out, long lo
                                                const int32_t* block_table, int max_blocks, const int32_t* cu_tokens,
                                                const int32_t* context_lens, int num_reqs, int num_pages, int page_size,
                                                int nh, int nkv, int D, int Dv, float scale, const float* table, int table_len,
-                                               const float* sink, int window, float out_scale, int splits, float* partial,
-                                               int T, int* err, cudaStream_t stream) {
+                                               const float* sink, int window, float out_scale, int tail, int splits,
+                                               float* partial, int T, int* err, cudaStream_t stream) {
     XamParams p;
     if (!xam_fill(p, q, out, out_stride, pool, block_table, max_blocks, cu_tokens, context_lens, num_reqs, num_pages, page_size,
-                  nh, nkv, D, Dv, scale, table, table_len, sink, window, out_scale, err) ||
+                  nh, nkv, D, Dv, scale, table, table_len, sink, window, out_scale, tail, err) ||
         nh / nkv > 16 || num_reqs > 65535 || splits < 1 || splits > 65535 || (splits > 1 && (!partial || T <= 0)))
         return AIRUN_ERR_ARG;
     if (num_reqs == 0) return AIRUN_OK;
     p.splits = splits; p.partial = partial; p.T = T;
-#define XAM_GROUP(A, B) xag_launch<A, B>(p, stream)
+#define XAM_GROUP(A, B, ONE) xag_launch<A, B, ONE>(p, stream)
     XAM_CASES(XAM_GROUP);
 #undef XAM_GROUP
 }

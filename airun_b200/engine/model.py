@@ -18,7 +18,7 @@ from typing import Dict, List, Optional, Tuple
 import torch
 
 from ..config.base import LayerCall, ModelConfig
-from ..parts.base import CastActivations, StreamWrite, make_part, part_factory
+from ..parts.base import CastActivations, PostNormWrite, StreamWrite, make_part, part_factory
 from ..parts import embedding as _embedding_parts      # noqa: F401  (registers the embedding and head parts)
 from ..weights.loader import (DictSource, TensorSource, WeightSpec, load_tensors, random_tensors)
 
@@ -59,8 +59,12 @@ class DecoderModel:
             mixer = make_part("mixer", spec.mixer, prefix=f"{p}.{names['mixer']}", **spec.mixer_args, **common)
             ffn = make_part("feed_forward", spec.feed_forward, prefix=f"{p}.{names['ffn']}", **spec.ffn_args, **common) \
                 if spec.feed_forward else None
+            more = dict(getattr(spec, "arrangement_args", {}))
+            if getattr(factory, "post_norms", False):       # an arrangement that norms its sub-layers' results as well
+                for which, has in (("norm1_post", True), ("norm2_post", two_norms)):
+                    more[which] = make_part("norm", spec.norm, prefix=f"{p}.{names[which]}", **spec.norm_args, **common) if has else None
             self.layers.append(make_part("arrangement", spec.arrangement, norm1=norm1, mixer=mixer,
-                                         norm2=norm2, ffn=ffn, dtype=dtype, **getattr(spec, "arrangement_args", {})))
+                                         norm2=norm2, ffn=ffn, dtype=dtype, **more))
         # a residual of several streams: every layer's arrangement must read and write all of them
         self.multi_stream = bool(self.layers) and all(getattr(l, "multi_stream", False) for l in self.layers)
         if not self.multi_stream and any(getattr(l, "multi_stream", False) for l in self.layers):
@@ -78,6 +82,11 @@ class DecoderModel:
         for c in self.order:
             if getattr(c, "add_row", None) is not None and not (0 <= c.add_row < self.order_table_rows):
                 raise ValueError(f"the execution order adds row {c.add_row} of a table of {self.order_table_rows} rows")
+        # the part that mixes the residual stream with the embedding before entries of the order that ask for it
+        ri = config.residual_input() if hasattr(config, "residual_input") else None
+        self.residual_input = make_part("residual_input", ri[0], prefix=ri[1], dtype=dtype, device=self.device, **ri[2]) if ri else None
+        if any(getattr(c, "reinject", False) for c in self.order) and (self.residual_input is None or self.multi_stream):
+            raise ValueError("the execution order mixes the residual with the embedding: that takes a residual_input part and one stream")
         self.layer_hook = None      # debugging and tests: called as hook(entry, residual [T, H]) after every entry
         fn_name, fn_args = config.final_norm() if hasattr(config, "final_norm") else \
             ("rmsnorm", dict(size=H, eps=config.rms_norm_eps))
@@ -91,7 +100,8 @@ class DecoderModel:
 
     # ---- weights ----
     def parts(self):
-        return [self.embedding] + self.layers + [self.final_norm, self.head]
+        mix = [self.residual_input] if self.residual_input is not None else []
+        return [self.embedding] + mix + self.layers + [self.final_norm, self.head]
 
     def weight_specs(self) -> List[WeightSpec]:
         specs = [s for p in self.parts() for s in p.weight_specs()]
@@ -208,13 +218,18 @@ class DecoderModel:
 
     # ---- one pass over the given tokens ----
     def forward(self, ctx, want_rows: Optional[torch.Tensor], n_want: int) -> Optional[torch.Tensor]:
+        from ..kernels import ops
         T = ctx.num_tokens
         ctx.ws_main.reset()
         x = ctx.ws_main.alloc((T, self.H), torch.float32)
         self.embedding.forward(ctx, ctx.token_ids[:T], x)
         if self.multi_stream:
             return self._forward_streams(ctx, x, want_rows, n_want)
-        delta = None
+        delta = kept = None
+        if self.residual_input is not None:
+            ctx.ws = ctx.ws_pair[0]
+            ctx.ws.reset()
+            kept = self.residual_input.begin(ctx, x)
         trace = TRACE_LAYERS and not torch.cuda.is_current_stream_capturing()
         for ci, call in enumerate(self.order):
             ctx.ws = ctx.ws_pair[ci % 2]
@@ -222,24 +237,25 @@ class DecoderModel:
             nxt = self.layers[self.order[ci + 1].layer] if ci + 1 < len(self.order) else None
             next_norm = nxt.norm1 if (nxt is not None and getattr(nxt, "accepts_normed", lambda: False)()) else None
             layer, extra = self.layers[call.layer], {}
+            if getattr(call, "reinject", False):
+                delta = self.residual_input.forward(ctx, x, delta, kept)
             if getattr(call, "add_row", None) is not None:
                 vec = self.order_table[call.add_row]
                 if getattr(layer, "accepts_add_vec", False):
                     extra["add_vec"] = vec
                 else:                                   # x += what is pending + the row, by a kernel of its own
-                    from ..kernels import ops
                     ops.add_rows(x[:T], delta=delta if isinstance(delta, torch.Tensor) else None, vec=vec)
                     delta = None if isinstance(delta, torch.Tensor) else delta
             if next_norm is not None:
                 extra["next_norm"] = next_norm
             delta = layer.forward(ctx, x, delta, ctx.caches[ci], **extra)
             if self.layer_hook is not None and not torch.cuda.is_current_stream_capturing():
-                if isinstance(delta, torch.Tensor):
-                    self.layer_hook(ci, x[:T] + delta[:T])
-                elif delta is None or isinstance(delta, CastActivations):       # nothing pending: x is the stream
-                    self.layer_hook(ci, x[:T])
+                now = self._stream_after(x, delta, T)
+                if now is not None:
+                    self.layer_hook(ci, now)
             if trace:           # synchronises after every block: a debugging aid, as the reference's AIRUN_TRACE_LAYERS
-                r = x[:ctx.num_tokens] if not isinstance(delta, torch.Tensor) else (x[:ctx.num_tokens] + delta[:ctx.num_tokens])
+                r = self._stream_after(x, delta, T)
+                r = x[:T] if r is None else r
                 print(f"[airun_b200] entry {ci} layer {call.layer}: rms {float(r.pow(2).mean().sqrt()):.6f} "
                       f"mean {float(r.mean()):+.6f}", file=sys.stderr)
         if n_want == 0:
@@ -249,11 +265,29 @@ class DecoderModel:
         hsel = ctx.ws.alloc((n_want, self.H), self.dtype)
         if isinstance(delta, CastActivations):
             delta = None
-        self.final_norm.forward(ctx, x, hsel, delta=delta, rows=want_rows[:n_want])
+        if isinstance(delta, PostNormWrite):            # the last result joins the stream on the final norm's way
+            if hasattr(self.final_norm, "fusable"):
+                w, eps = self.final_norm.fusable()
+                ops.sandwich_norm(x, hsel, y=delta.y, w_post=delta.weight, eps_post=delta.eps, w_pre=w, eps_pre=eps, rows=want_rows[:n_want])
+                delta = hsel
+            else:
+                ops.sandwich_norm(x, None, y=delta.y, w_post=delta.weight, eps_post=delta.eps)
+                delta = None
+        if delta is not hsel:
+            self.final_norm.forward(ctx, x, hsel, delta=delta, rows=want_rows[:n_want])
         logits = ctx.ws_main.alloc((n_want, self.V), torch.float32)
         self.head.forward(ctx, hsel, logits)
         return logits
 
+    @staticmethod
+    def _stream_after(x: torch.Tensor, pending, T: int) -> Optional[torch.Tensor]:
+        """The residual stream after a block, for hooks and traces: x with what the block left pending (None: not known)."""
+        if isinstance(pending, torch.Tensor):
+            return x[:T] + pending[:T]
+        if isinstance(pending, PostNormWrite):
+            y = pending.y[:T]
+            return x[:T] + y / torch.sqrt((y * y).mean(dim=-1, keepdim=True) + pending.eps) * pending.weight
+        return x[:T] if pending is None or isinstance(pending, CastActivations) else None
 
     def _forward_streams(self, ctx, x: torch.Tensor, want_rows: Optional[torch.Tensor], n_want: int) -> Optional[torch.Tensor]:
         """The pass over the layers with a residual of ``streams`` copies, [T, S, H]: every copy starts as the embedding,

@@ -777,7 +777,9 @@ def softmax_attention_bf16(ctx, q, out, cache, part) -> bool:
     _need(tuple(out.shape) == (T, nh * Dv) and out.stride(1) == 1 and out.dtype == torch.bfloat16,
           "out must be row-major bfloat16 [T, heads*Dv]")
     pool, bt = cache.pool, cache.block_table
-    _need(pool.is_contiguous() and pool[0].numel() == nkv * cache.page_size * (D + Dv), "the cache pages do not fit the head sizes")
+    tail = int(getattr(part, "tail", -1))              # >= 0: one cached row of D + tail elements is key and value
+    _need(pool.is_contiguous() and pool[0].numel() == nkv * cache.page_size * (D + tail if tail >= 0 else D + Dv),
+          "the cache pages do not fit the head sizes")
     _need(ctx.cu_tokens.numel() >= ctx.num_reqs + 1 and ctx.context_lens.numel() >= ctx.num_reqs,
           "the batch's layout arrays are shorter than its number of requests")
     table_len = 0
@@ -790,9 +792,9 @@ def softmax_attention_bf16(ctx, q, out, cache, part) -> bool:
     common = [_p(q), _p(out), out.stride(0) if T > 1 else max(out.shape[1], out.stride(0)), _p(pool), _p(bt), bt.stride(0),
               _p(ctx.cu_tokens), _p(ctx.context_lens), int(ctx.num_reqs)]
     consts = [pool.shape[0], int(cache.page_size), nh, nkv, D, Dv, float(part.scale), _p(part.table), int(table_len), _p(part.sink),
-              int(part.window), float(part.out_scale)]
+              int(part.window), float(part.out_scale), tail]
     sig = [c_void_p, c_void_p, c_longlong, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int]
-    csig = [c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_void_p, c_int, c_void_p, c_int, c_float]
+    csig = [c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_void_p, c_int, c_void_p, c_int, c_float, c_int]
     # requests that bring ONE token go to the kernel whose product rows are the query heads of a KV head (groups of up
     # to 16), which finds them on the device; the tile kernel then skips them
     single = "softmax_group" not in DISABLED and nh // nkv <= 16

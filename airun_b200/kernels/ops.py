@@ -258,6 +258,36 @@ def postnorm_add(x: torch.Tensor, y: torch.Tensor, weight: torch.Tensor, eps: fl
              _stream()), "postnorm_add")
 
 
+SANDWICH_NORM, SANDWICH_COPY, SANDWICH_SPLIT = 0, 1, 2
+
+
+def sandwich_norm(x: torch.Tensor, out: Optional[torch.Tensor], y: Optional[torch.Tensor] = None,
+                  w_post: Optional[torch.Tensor] = None, eps_post: float = 0.0, w_pre: Optional[torch.Tensor] = None,
+                  eps_pre: float = 0.0, rows: Optional[torch.Tensor] = None, mode: int = SANDWICH_NORM,
+                  write_back: bool = True) -> None:
+    """v = x [+ y / rms(y) * w_post] and, in the same pass, ``out`` by ``mode``: v / rms(v) * w_pre (SANDWICH_NORM), v in
+    float32 (SANDWICH_COPY) or v as two bfloat16 halves side by side, [T, 2n], whose sum is v to 16 bits (SANDWICH_SPLIT).
+    v becomes x unless ``rows`` picks the rows (out[0..len(rows))) or ``write_back`` is False."""
+    _cuda(x, out, y, w_post, w_pre, rows)
+    _need(x.dtype == torch.float32 and x.dim() == 2 and x.is_contiguous(), "x must be contiguous float32 [T, n]")
+    T, n = x.shape
+    if y is not None:
+        _need(y.dtype == torch.float32 and y.shape == x.shape and y.is_contiguous(), "y must match x")
+    for w in (w_post, w_pre):
+        _need(w is None or (w.dtype == torch.float32 and tuple(w.shape) == (n,) and w.is_contiguous()), "norm weights must be float32 [n]")
+    n_rows = T
+    if rows is not None:
+        _need(rows.dtype == torch.int32 and rows.dim() == 1 and rows.is_contiguous(), "rows must be int32 [R]")
+        n_rows = rows.shape[0]
+    if out is not None:
+        _need(out.dim() == 2 and out.shape[0] >= n_rows and out.shape[1] == (2 * n if mode == SANDWICH_SPLIT else n) and out.is_contiguous(),
+              "out must be contiguous [rows, n] ([rows, 2n] for a split)")
+    f = _fn("elementwise", "airun_sandwich_norm",
+            [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_float, c_float, c_int, c_int, c_void_p])
+    _check(f(_p(x), _p(y), _p(w_post), _p(w_pre), _p(out), _dt(out) if out is not None else DT_F32, _p(rows), n_rows, n,
+             float(eps_post), float(eps_pre), 1 if write_back and rows is None else 0, int(mode), _stream()), "sandwich_norm")
+
+
 def cast_f32(src: torch.Tensor, out: torch.Tensor) -> None:
     """out = src (float32) in out's type."""
     _cuda(src, out)
@@ -662,15 +692,19 @@ def stream_step(xs: torch.Tensor, y: Optional[torch.Tensor] = None, carry: Optio
 def qkv_prepare(proj: torch.Tensor, bias: Optional[torch.Tensor], q_w: Optional[torch.Tensor], k_w: Optional[torch.Tensor],
                 unit_norm: bool, eps: float, rope_kind: int, rotary_dim: int, inv_freq: Optional[torch.Tensor],
                 temp_coef: float, temp_every: int, q_out: torch.Tensor, cache, ctx, nh: int, nkv: int, D: int, Dv: int,
-                store: bool = True, rope_positions: Optional[torch.Tensor] = None) -> None:
+                store: bool = True, rope_positions: Optional[torch.Tensor] = None, one_row: bool = False) -> None:
     """What lies between the q/k/v product and the attention (csrc/softmax_attention.cu: qkv_prepare_kernel): biases,
     a weighted root-mean-square norm per head before the rotation (``q_w`` / ``k_w`` float32 [D]), the rotation, an
     unweighted norm per head after it (``unit_norm``), the query temperature; q out, k and v into the token's page.
-    ``proj`` float32 rows [q heads | k heads | v heads] (q heads only without ``store``)."""
+    ``proj`` float32 rows [q heads | k heads | v heads] (q heads only without ``store``).  ``one_row``: the values are
+    the keys before the rotation, so proj has no value columns and a cached row is [key | its first ``rotary_dim``
+    dimensions unrotated], D + rotary_dim elements."""
     _cuda(proj, bias, q_w, k_w, inv_freq, q_out, cache.pool, cache.block_table, ctx.positions, ctx.req_of_token, ctx.err, rope_positions)
     _rows_f32(proj, "proj")
     T = proj.shape[0]
-    width = nh * D + (nkv * (D + Dv) if store else 0)
+    row = D + rotary_dim if one_row else D + Dv
+    width = nh * D + (nkv * (D if one_row else row) if store else 0)
+    _need(not one_row or (Dv == D and k_w is None and not unit_norm), "keys that serve as values have no norm of their own")
     _need(proj.shape[1] >= width, f"proj must have at least {width} columns")
     _need(q_out.is_contiguous() and tuple(q_out.shape) == (T, nh * D), "q_out must be contiguous [T, heads*D]")
     if bias is not None:
@@ -680,31 +714,33 @@ def qkv_prepare(proj: torch.Tensor, bias: Optional[torch.Tensor], q_w: Optional[
     _need(D <= 256, "head sizes above 256 are beyond the kernel")
     pool, bt = cache.pool, cache.block_table
     if store:
-        _need(pool.dtype == q_out.dtype and pool.is_contiguous() and pool[0].numel() == nkv * cache.page_size * (D + Dv),
+        _need(pool.dtype == q_out.dtype and pool.is_contiguous() and pool[0].numel() == nkv * cache.page_size * row,
               "the cache pages do not fit the head sizes or the type of q")
     f = _fn("softmax_attention", "airun_qkv_prepare",
             [c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_int, c_float, c_int, c_int, c_void_p, c_void_p, c_float, c_int,
              c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
-             c_int, c_void_p, c_void_p])
+             c_int, c_int, c_void_p, c_void_p])
     _check(f(_p(proj), _row_stride(proj), _p(bias), _p(q_w), _p(k_w), 1 if unit_norm else 0, float(eps), int(rope_kind),
              int(rotary_dim), _p(inv_freq), _p(rope_positions), float(temp_coef), int(temp_every), _p(q_out), _p(pool), _dt(q_out),
              _p(bt), bt.stride(0), _p(ctx.positions), _p(ctx.req_of_token), T, int(ctx.num_reqs), pool.shape[0],
-             int(cache.page_size), nh, nkv, D, Dv, 1 if store else 0, _p(ctx.err), _stream()), "qkv_prepare")
+             int(cache.page_size), nh, nkv, D, Dv, 1 if store else 0, 1 if one_row else 0, _p(ctx.err), _stream()), "qkv_prepare")
 
 
 def softmax_attention(q: torch.Tensor, out: torch.Tensor, cache, ctx, nh: int, nkv: int, D: int, Dv: int, scale: float,
                       table: Optional[torch.Tensor] = None, sink: Optional[torch.Tensor] = None, window: int = 0,
-                      out_scale: float = 1.0) -> None:
+                      out_scale: float = 1.0, tail: int = -1) -> None:
     """Softmax attention over cache pages in float32 arithmetic (csrc/softmax_attention.cu: softmax_attention_kernel):
     ``table`` float32 [heads, n] adds table[h, min(i - j, n - 1)] to the scaled score, ``sink`` float32 [heads] adds
     exp(sink_h) to the denominator, ``window`` > 0 hides keys with i - j >= window; the result is times ``out_scale``.
-    ``out`` may be a column slice of a wider buffer."""
+    ``out`` may be a column slice of a wider buffer.  ``tail`` >= 0: a cached row of D + tail elements is key (its first D)
+    and value (its last D) at once."""
     _cuda(q, out, cache.pool, cache.block_table, ctx.positions, ctx.req_of_token, ctx.err, table, sink)
     T = q.shape[0]
     _need(q.is_contiguous() and tuple(q.shape) == (T, nh * D), "q must be contiguous [T, heads*D]")
     _need(tuple(out.shape) == (T, nh * Dv) and out.stride(1) == 1 and out.dtype == q.dtype, "out must be row-major [T, heads*Dv] of q's type")
     pool, bt = cache.pool, cache.block_table
-    _need(pool.dtype == q.dtype and pool.is_contiguous() and pool[0].numel() == nkv * cache.page_size * (D + Dv),
+    _need(pool.dtype == q.dtype and pool.is_contiguous()
+          and pool[0].numel() == nkv * cache.page_size * (D + tail if tail >= 0 else D + Dv),
           "the cache pages do not fit the head sizes or the type of q")
     table_len = 0
     if table is not None:
@@ -715,10 +751,10 @@ def softmax_attention(q: torch.Tensor, out: torch.Tensor, cache, ctx, nh: int, n
         _need(sink.dtype == torch.float32 and sink.numel() == nh and sink.is_contiguous(), "the sinks must be float32 [heads]")
     f = _fn("softmax_attention", "airun_softmax_attention",
             [c_void_p, c_void_p, c_longlong, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int,
-             c_int, c_int, c_int, c_float, c_void_p, c_int, c_void_p, c_int, c_float, c_void_p, c_void_p])
+             c_int, c_int, c_int, c_float, c_void_p, c_int, c_void_p, c_int, c_float, c_int, c_void_p, c_void_p])
     _check(f(_p(q), _p(out), _row_stride(out), _p(pool), _dt(q), _p(bt), bt.stride(0), _p(ctx.positions), _p(ctx.req_of_token), T,
              int(ctx.num_reqs), pool.shape[0], int(cache.page_size), nh, nkv, D, Dv, float(scale), _p(table), int(table_len),
-             _p(sink), int(window), float(out_scale), _p(ctx.err), _stream()), "softmax_attention")
+             _p(sink), int(window), float(out_scale), int(tail), _p(ctx.err), _stream()), "softmax_attention")
 
 
 # ---------------------------------------------------------------- products
@@ -817,24 +853,29 @@ def token_shift(x: torch.Tensor, mu: torch.Tensor, state: torch.Tensor, prev_off
              _p(ctx.state_slots), int(ctx.num_reqs), _p(out), _dt(out), T, W, _p(ctx.err), _stream()), "token_shift")
 
 
-RECURRENCE_DELTA, RECURRENCE_WKV = 0, 1
+RECURRENCE_DELTA, RECURRENCE_WKV, RECURRENCE_DELTA_HEAD = 0, 1, 2
 
 
 def recurrent_state(mode: int, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, g: torch.Tensor, state: torch.Tensor, ctx,
                     out: torch.Tensor, heads: int, kv_rep: int, D: int, Dv: int, beta: Optional[torch.Tensor] = None,
                     bonus: Optional[torch.Tensor] = None, tail_src: Optional[torch.Tensor] = None, tail_off: int = 0,
-                    tail_rows: int = 0) -> None:
+                    tail_rows: int = 0, a_log: Optional[torch.Tensor] = None, dt_bias: Optional[torch.Tensor] = None) -> None:
     """The delta rule (RECURRENCE_DELTA: q, k [T, heads/kv_rep * D], v [T, heads*Dv], decay g [T, heads*D], beta
-    [T, heads] BEFORE its sigmoid) or the time mix with a bonus (RECURRENCE_WKV: r, k, v, decay [T, heads*D], bonus [heads, D]) over the
+    [T, heads] BEFORE its sigmoid), the same with one decay per head (RECURRENCE_DELTA_HEAD: g [T, heads] is its
+    projection, the decay exp(-exp(a_log) * softplus(g + dt_bias)) with a_log, dt_bias [heads]) or the time mix with a bonus (RECURRENCE_WKV: r, k, v, decay [T, heads*D], bonus [heads, D]) over the
     rows of every request in order, on state[slot, : heads*D*Dv] viewed as [heads, D, Dv]; out float32 [T, heads*Dv].
     With ``tail_rows`` the last rows of (state[slot, tail_off:] as [tail_rows, C], then this step's rows of
     ``tail_src`` [T, C]) are kept there for the next step."""
-    _cuda(q, k, v, g, state, out, beta, bonus, tail_src)
+    _cuda(q, k, v, g, state, out, beta, bonus, tail_src, a_log, dt_bias)
+    head_decay = mode == RECURRENCE_DELTA_HEAD
     for t_, name in ((q, "q"), (k, "k"), (v, "v"), (g, "g")):
         _rows_f32(t_, name)
     T = q.shape[0]
-    _need(q.shape[1] == heads // kv_rep * D and k.shape[1] == q.shape[1] and v.shape[1] == heads * Dv and g.shape[1] == heads * D,
-          "q, k, v or the decay has the wrong width")
+    _need(q.shape[1] == heads // kv_rep * D and k.shape[1] == q.shape[1] and v.shape[1] == heads * Dv
+          and g.shape[1] == heads * (1 if head_decay else D), "q, k, v or the decay has the wrong width")
+    for t_ in (a_log, dt_bias):
+        _need((t_ is not None) == head_decay and (t_ is None or (t_.dtype == torch.float32 and t_.numel() == heads and t_.is_contiguous())),
+              "a_log and dt_bias, float32 [heads], belong to the mode with one decay per head")
     _need(state.dtype == torch.float32 and state.dim() == 2 and state.stride(1) == 1 and state.shape[1] >= heads * D * Dv,
           "state must be float32 [slots, >= heads*D*Dv]")
     _need(out.dtype == torch.float32 and tuple(out.shape) == (T, heads * Dv) and out.is_contiguous(), "out must be float32 [T, heads*Dv]")
@@ -852,11 +893,11 @@ def recurrent_state(mode: int, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor
         _need(tail_off + tail_rows * tw <= state.shape[1], "the tail does not fit the state")
     f = _fn("recurrent_state", "airun_recurrent_state",
             [c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_longlong, c_longlong, c_longlong, c_longlong, c_void_p, c_longlong,
-             c_void_p, c_void_p, c_longlong, c_int, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_void_p,
+             c_void_p, c_void_p, c_void_p, c_void_p, c_longlong, c_int, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_void_p,
              c_longlong, c_longlong, c_int, c_int, c_int, c_void_p, c_void_p])
     long_chains = 1 if T > 2 * int(ctx.num_reqs) else 0          # requests bring many tokens each, not one
     _check(f(int(mode), _p(q), _p(k), _p(v), _p(g), _row_stride(q), _row_stride(k), _row_stride(v), _row_stride(g), _p(beta), bs,
-             _p(bonus), _p(state), state.stride(0), state.shape[0], _p(ctx.cu_tokens), _p(ctx.state_slots), int(ctx.num_reqs),
+             _p(a_log), _p(dt_bias), _p(bonus), _p(state), state.stride(0), state.shape[0], _p(ctx.cu_tokens), _p(ctx.state_slots), int(ctx.num_reqs),
              _p(out), heads, kv_rep, D, Dv, _p(tail_src), ts, int(tail_off), int(tail_rows), tw, long_chains, _p(ctx.err),
              _stream()), "recurrent_state")
 

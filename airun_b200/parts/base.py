@@ -20,6 +20,8 @@ PositionEncoding fused() -> (kind, rotary_dim, inv_freq) the attention prologue
                 rotation_positions(ctx) -> int32 [T] or None (None: the cache positions)
 Embedding       forward(ctx, token_ids, out float32 [T, hidden]); .table for a tied head
 Head            forward(ctx, h [rows, hidden], out float32 [rows, vocab])
+ResidualInput   begin(ctx, x0) -> kept; forward(ctx, x, pending, kept) -> pending: the residual stream mixed
+                  with the embedding ahead of a pass over layers that run several times
 Mixer           cache_spec() -> PagedKVSpec | StateSpec | None
                 forward(ctx, h, cache) -> float32 [T, hidden] (the residual delta)
 FeedForward     forward(ctx, h) -> float32 [T, hidden]
@@ -105,6 +107,16 @@ class CastActivations:
 
 
 @dataclass
+class PostNormWrite:
+    """What a block whose sub-layers' results are normed on their way out leaves pending: the result ``y`` [T, H] of its
+    last sub-layer and that norm's weight and eps, x += y / rms(y) * weight; the pass that next reads the residual (the
+    next block's first norm, a mix of the residual with the embedding, the final norm) carries it out on its way."""
+    y: torch.Tensor
+    weight: torch.Tensor
+    eps: float
+
+
+@dataclass
 class StreamWrite:
     """What a block over a residual of several streams leaves pending: the result ``y`` [T, H] of its last sub-layer
     and the numbers that write it into the streams, x_t <- sum_s carry[s, t] x_s + mult * write[t] * (y + y_bias); the
@@ -173,6 +185,22 @@ class Head(Part):
         raise NotImplementedError
 
 
+class ResidualInput(Part):
+    """What mixes the residual stream with the embedding in front of entries of the execution order that ask for it
+    (``LayerCall.reinject``).
+
+    begin(ctx, x0): called once a step with the embedding's output x0 float32 [T, H], before any layer; returns
+                    whatever forward needs of it (kept in ``ctx.ws_main``).
+    forward(ctx, x, pending, kept) -> pending: makes x [T, H] the mixed stream, having carried out what the block
+                    before left pending, and returns what is still to be added to x by the block that follows."""
+
+    def begin(self, ctx, x0: torch.Tensor):
+        raise NotImplementedError
+
+    def forward(self, ctx, x: torch.Tensor, pending, kept):
+        raise NotImplementedError
+
+
 class Mixer(Part):
     def cache_spec(self):
         return None
@@ -187,7 +215,8 @@ class FeedForward(Part):
 
 
 _REGISTRIES: Dict[str, Dict[str, Callable]] = {
-    "mixer": {}, "feed_forward": {}, "norm": {}, "position": {}, "arrangement": {}, "embedding": {}, "head": {}}
+    "mixer": {}, "feed_forward": {}, "norm": {}, "position": {}, "arrangement": {}, "embedding": {}, "head": {},
+    "residual_input": {}}
 
 
 def register_part(kind: str, name: str, factory: Callable) -> None:

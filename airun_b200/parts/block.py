@@ -18,7 +18,7 @@ from typing import Dict, List, Optional
 import torch
 
 from ..weights.loader import WeightSpec
-from .base import CastActivations, FeedForward, Mixer, Norm, NormedActivations, Part, ResidualSink, StreamWrite, register_part
+from .base import CastActivations, FeedForward, Mixer, Norm, NormedActivations, Part, PostNormWrite, ResidualSink, StreamWrite, register_part
 
 
 class PreNormBlock(Part):
@@ -447,3 +447,65 @@ class HyperConnectionBlock(Part):
 
 
 register_part("arrangement", "hyper_connections", HyperConnectionBlock)
+
+
+class SandwichBlock(Part):
+    """A norm before and a norm after each sub-layer: x += norm1b(mixer(norm1(x))), then x += norm2b(ffn(norm2(x))).  The
+    feed-forward may be absent, and then so are norm2 and norm2b.  The norm and the add on a sub-layer's result and the
+    norm in front of the next sub-layer are ONE pass over the residual (csrc/elementwise.cu: sandwich_norm_kernel), also
+    from block to block: the last result is left pending (``PostNormWrite``) for whoever reads the residual next.  The
+    norms must offer ``fusable()`` (weight, eps) of a root-mean-square norm."""
+    norm2_belongs_to_ffn = True
+    post_norms = True
+
+    def __init__(self, norm1: Norm, mixer: Mixer, norm2: Optional[Norm], ffn: Optional[FeedForward], dtype: torch.dtype,
+                 norm1_post: Norm, norm2_post: Optional[Norm]):
+        self.norm1, self.mixer, self.norm2, self.ffn, self.dtype = norm1, mixer, norm2, ffn, dtype
+        self.norm1_post, self.norm2_post = norm1_post, norm2_post
+        for n in (norm1, norm1_post, norm2, norm2_post):
+            if n is not None and not hasattr(n, "fusable"):
+                raise ValueError("a block with norms on both sides needs root-mean-square norms (parts with fusable())")
+
+    def parts(self):
+        return tuple(p for p in (self.norm1, self.mixer, self.norm1_post, self.norm2, self.ffn, self.norm2_post) if p is not None)
+
+    def weight_specs(self) -> List[WeightSpec]:
+        return [s for p in self.parts() for s in p.weight_specs()]
+
+    def load_weights(self, tensors: Dict[str, torch.Tensor]) -> None:
+        for p in self.parts():
+            p.load_weights(tensors)
+
+    def cache_spec(self):
+        return self.mixer.cache_spec()
+
+    def device_driven(self) -> bool:
+        return all(getattr(p, "device_driven", False) for p in self.parts())
+
+    def graph_safe(self) -> bool:
+        return all(getattr(p, "graph_safe", True) for p in self.parts())
+
+    def accepts_normed(self) -> bool:
+        return False
+
+    def _read(self, ctx, x: torch.Tensor, pending, norm: Norm) -> torch.Tensor:
+        """The next sub-layer's input: norm(x) once what is pending (a PostNormWrite, or a plain delta) is in x."""
+        from ..kernels import ops
+        h = ctx.ws.alloc(tuple(x.shape), self.dtype)
+        w, eps = norm.fusable()
+        if isinstance(pending, PostNormWrite):
+            ops.sandwich_norm(x, h, y=pending.y, w_post=pending.weight, eps_post=pending.eps, w_pre=w, eps_pre=eps)
+        else:
+            ops.rmsnorm(x, w, eps, h, delta=pending if isinstance(pending, torch.Tensor) else None)
+        return h
+
+    def forward(self, ctx, x: torch.Tensor, pending, cache, next_norm: Optional[Norm] = None):
+        y = self.mixer.forward(ctx, self._read(ctx, x, pending, self.norm1), cache)
+        pending = PostNormWrite(y, *self.norm1_post.fusable())
+        if self.ffn is not None:
+            y = self.ffn.forward(ctx, self._read(ctx, x, pending, self.norm2))
+            pending = PostNormWrite(y, *self.norm2_post.fusable())
+        return pending
+
+
+register_part("arrangement", "sandwich", SandwichBlock)

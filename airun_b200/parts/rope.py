@@ -90,3 +90,38 @@ class RotaryScaledInterleaved(RotaryInterleaved):
 
 
 register_part("position", "rotary_scaled_interleaved", RotaryScaledInterleaved)
+
+
+class RotaryNeoxByWavelength(RotaryNeox):
+    """Pairs (i, i + dims/2) with frequencies stretched by their wavelength: with ``scaling`` = {factor, low, high,
+    original} a pair of frequency f and wavelength l = 2 pi / f
+
+        l < original / high     keeps f
+        l > original / low      turns at f / factor
+        between                 at (1 - s) f / factor + s f,   s = (original / l - low) / (high - low).
+
+    Without ``scaling`` it is RotaryNeox.  Everything is computed once in double precision and rounded to float32."""
+
+    def __init__(self, prefix: str = "", rotary_dim: int = 0, theta: float = 10000.0, scaling: Optional[dict] = None,
+                 dtype=None, device=None):
+        import math
+        super().__init__(prefix, rotary_dim, theta, dtype, device)
+        if not scaling:
+            return
+        factor, original, low, high = (float(scaling[k]) for k in ("factor", "original", "low", "high"))
+        if not (factor > 0 and original > 0 and low > 0 and high >= low):
+            raise ValueError("factor, original and low of a rotary scaling must be positive, high at least low")
+        freqs = []
+        for i in range(rotary_dim // 2):
+            f = self.theta ** (-2.0 * i / rotary_dim)
+            wavelength = 2.0 * math.pi / f
+            if wavelength > original / low:
+                f /= factor
+            elif wavelength >= original / high and high > low:
+                s = (original / wavelength - low) / (high - low)
+                f = (1.0 - s) * f / factor + s * f
+            freqs.append(f)
+        self.inv_freq = torch.tensor(freqs, dtype=torch.float64).to(torch.float32).to(device)
+
+
+register_part("position", "rotary_neox_by_wavelength", RotaryNeoxByWavelength)

@@ -12,8 +12,13 @@ With h the mixer's input, H query heads and G key/value heads (query head h read
                                                          bucket(n) = n for n < B/2, else
                                                          min(B - 1, B/2 + floor(ln(n / (B/2)) / ln(far / (B/2)) * (B - B/2)))
     p_ij = exp(s_ij) / (sum_j' exp(s_ij') + exp(sink_h)) with ``sink``: one more term of the denominator per head, which
-                                                         has no key and no value
+                                                         has no key and no value; ``sink="one"``: the term is 1 for every
+                                                         head (sink_h = 0) and no tensor holds it
     o_i = sum_j p_ij v_j over j <= i (and i - j < window when ``window`` > 0),   out = out_scale * Wo concat_heads(o)
+
+``values="keys"``: v = k as projected, ahead of the rotation; there is no Wv.  Key and value of a token then share one
+cached row (csrc/softmax_attention.cu: ``one_row``) of key_dim + rotated dims elements, in which a value's dimensions
+come in another order; the columns of Wo are put into that order when the weights are loaded.
 
 The bucket of every distance is worked out once, in double precision on the host, into a table per head that the kernels
 index by min(i - j, far).  The three input projections run as one product.  The part has the split form
@@ -51,7 +56,7 @@ class SoftmaxAttention(Mixer):
     def __init__(self, prefix: str, hidden_size: int, num_heads: int, num_kv_heads: int, key_dim: int, value_dim: int,
                  scale: float, norm_eps: float = 1e-6, bias: bool = False, qk_norm: str = "none",
                  position: str = "none", position_args: Optional[dict] = None, temp_coef: float = 0.0, temp_every: int = 0,
-                 distance_rows: int = 0, distance_far: int = 0, sink: bool = False, window: int = 0, out_scale: float = 1.0,
+                 distance_rows: int = 0, distance_far: int = 0, sink=False, values: str = "own", window: int = 0, out_scale: float = 1.0,
                  dtype: torch.dtype = torch.bfloat16, device=None, names: Optional[Dict[str, str]] = None):
         self.prefix, self.H = prefix, int(hidden_size)
         self.nh, self.nkv, self.D, self.Dv = int(num_heads), int(num_kv_heads), int(key_dim), int(value_dim)
@@ -68,10 +73,16 @@ class SoftmaxAttention(Mixer):
         self.distance_rows, self.distance_far = int(distance_rows or 0), int(distance_far or 0)
         if self.distance_rows and self.distance_far <= self.distance_rows // 2:
             raise ValueError("the farthest distance of the table must lie beyond half its rows")
-        self.has_sink, self.window, self.out_scale = bool(sink), int(window or 0), float(out_scale)
+        self.has_sink, self.sink_is_one = bool(sink), sink == "one"
+        self.window, self.out_scale = int(window or 0), float(out_scale)
         self.dtype, self.device = dtype, device
         self.pos = make_part("position", position, prefix=prefix, dtype=dtype, device=device, **(position_args or {}))
         kind, rdim, _ = self.pos.fused()
+        if values not in ("own", "keys"):
+            raise ValueError("values is 'own' (a projection Wv) or 'keys' (the keys before their rotation)")
+        if values == "keys" and (self.Dv != self.D or qk_norm != "none"):
+            raise ValueError("keys that serve as values have the keys' size and no norm")
+        self.tail = rdim if values == "keys" else -1        # >= 0: elements a cached row has beyond the key
         if rdim > self.D:
             raise ValueError(f"{rdim} rotated dimensions do not fit a head of {self.D}")
         n = dict(q="q", k="k", v="v", o="o", q_bias="q.b", k_bias="k.b", v_bias="v.b", o_bias="o.b", q_norm="q.norm",
@@ -85,26 +96,33 @@ class SoftmaxAttention(Mixer):
     # ---- weights ----
     def weight_specs(self) -> List[WeightSpec]:
         nm, H, qw, kw, vw = self.names, self.H, self.nh * self.D, self.nkv * self.D, self.nkv * self.Dv
-        specs = [WeightSpec(nm["q"], (qw, H)), WeightSpec(nm["k"], (kw, H)), WeightSpec(nm["v"], (vw, H)),
-                 WeightSpec(nm["o"], (H, self.nh * self.Dv))]
+        specs = [WeightSpec(nm["q"], (qw, H)), WeightSpec(nm["k"], (kw, H)), WeightSpec(nm["o"], (H, self.nh * self.Dv))]
+        if self.tail < 0:
+            specs.append(WeightSpec(nm["v"], (vw, H)))
         if self.bias:
             specs += [WeightSpec(nm["q_bias"], (qw,), storage="float32"), WeightSpec(nm["k_bias"], (kw,), storage="float32"),
-                      WeightSpec(nm["v_bias"], (vw,), storage="float32"), WeightSpec(nm["o_bias"], (H,), storage="float32")]
+                      WeightSpec(nm["o_bias"], (H,), storage="float32")]
+            if self.tail < 0:
+                specs.append(WeightSpec(nm["v_bias"], (vw,), storage="float32"))
         if self.qk_norm == "weight":
             specs += [WeightSpec(nm["q_norm"], (self.D,), storage="float32", init="norm"),
                       WeightSpec(nm["k_norm"], (self.D,), storage="float32", init="norm")]
         if self.distance_rows:
             specs.append(WeightSpec(nm["rel"], (self.distance_rows, self.nh), storage="float32"))
-        if self.has_sink:
+        if self.has_sink and not self.sink_is_one:
             specs.append(WeightSpec(nm["sink"], (self.nh,), storage="float32"))
         return specs + self.pos.weight_specs()
 
     def load_weights(self, tensors: Dict[str, torch.Tensor]) -> None:
         nm = self.names
-        self.w_in = torch.cat([tensors.pop(nm["q"]), tensors.pop(nm["k"]), tensors.pop(nm["v"])], dim=0).contiguous()
+        which = ("q", "k", "v") if self.tail < 0 else ("q", "k")
+        self.w_in = torch.cat([tensors.pop(nm[k]) for k in which], dim=0).contiguous()
         self.w_out = tensors.pop(nm["o"])
+        if self.tail > 0:       # values, and so the heads' results, hold dimensions tail .. D-1, then 0 .. tail-1
+            w = self.w_out.view(self.H, self.nh, self.Dv)
+            self.w_out = torch.cat([w[:, :, self.tail:], w[:, :, :self.tail]], dim=2).reshape(self.H, -1).contiguous()
         if self.bias:
-            self.in_bias = torch.cat([tensors[nm["q_bias"]], tensors[nm["k_bias"]], tensors[nm["v_bias"]]]).contiguous()
+            self.in_bias = torch.cat([tensors[nm[k + "_bias"]] for k in which]).contiguous()
             self.output_bias = tensors[nm["o_bias"]]
         if self.qk_norm == "weight":
             self.q_norm_w, self.k_norm_w = tensors[nm["q_norm"]], tensors[nm["k_norm"]]
@@ -112,7 +130,9 @@ class SoftmaxAttention(Mixer):
             rel = tensors[nm["rel"]]
             idx = torch.tensor(distance_buckets(self.distance_rows, self.distance_far), dtype=torch.long, device=rel.device)
             self.table = rel[idx].t().contiguous()                 # [heads, distances]
-        if self.has_sink:
+        if self.sink_is_one:
+            self.sink = torch.zeros(self.nh, dtype=torch.float32, device=self.w_in.device)
+        elif self.has_sink:
             self.sink = tensors[nm["sink"]]
         self.pos.load_weights(tensors)
 
@@ -121,6 +141,8 @@ class SoftmaxAttention(Mixer):
 
     # ---- cache ----
     def cache_spec(self):
+        if self.tail >= 0:
+            return PagedKVSpec(self.nkv, self.D + self.tail, self.window, values=False)
         return PagedKVSpec(self.nkv, self.D, self.window, value_dim=self.Dv if self.Dv != self.D else 0)
 
     # ---- compute ----
@@ -137,7 +159,7 @@ class SoftmaxAttention(Mixer):
         kind, rdim, inv_freq = self.pos.fused()
         ops.qkv_prepare(proj, self.in_bias, self.q_norm_w, self.k_norm_w, self.qk_norm == "unit", self.eps, kind, rdim, inv_freq,
                         self.temp_coef, self.temp_every, q, cache, ctx, self.nh, self.nkv, self.D, self.Dv, store=True,
-                        rope_positions=self.pos.rotation_positions(ctx))
+                        rope_positions=self.pos.rotation_positions(ctx), one_row=self.tail >= 0)
         self.attend(ctx, q, act, cache)
 
     def attend(self, ctx, q: torch.Tensor, out: torch.Tensor, cache) -> None:
@@ -146,7 +168,7 @@ class SoftmaxAttention(Mixer):
             if fast.softmax_attention_bf16(ctx, q, out, cache, self):
                 return
         ops.softmax_attention(q, out, cache, ctx, self.nh, self.nkv, self.D, self.Dv, self.scale, self.table, self.sink,
-                              self.window, self.out_scale)
+                              self.window, self.out_scale, tail=self.tail)
 
     def forward(self, ctx, h, cache, sink=None, add_bias: bool = True):
         """The residual delta.  With ``add_bias`` False the output bias (``output_bias``, times nothing) is left to the
