@@ -705,6 +705,89 @@ def workload_vedizen(a) -> int:
 
 
 
+def measure_design(eng, kinds, T: int, ctx_len: int, steps: int, warmup: int, pk: dict) -> dict:
+    """Prefill of one T-token prompt and decode at batch 8 and 64 (context ``ctx_len``) through the step function and its
+    CUDA graphs, and how long each kind of kernel runs inside the prefill step and the batch-64 decode step: CUDA events
+    around every call of the kind, the step launched kernel by kernel, the fastest of four.  ``kinds``: name -> (module,
+    function, work at t tokens of one prompt, bytes at a batch of b single tokens, what bounds the prompt's: "hbm" (work in
+    bytes), "fp32" or a tensor product (FLOPs))."""
+    import torch
+    from airun_b200 import StepEntry
+    fp32_peak = 148 * 128 * 2 * 1.965e9          # FMA lanes x 2 x the highest SM clock: nominal, no measured figure
+    res = {}
+    pre_ms = time_prefill(eng, T, runs=5)
+    b64 = time_decode_onward(eng, 64, ctx_len, steps, warmup, "v")
+    b8 = time_decode_onward(eng, 8, ctx_len, steps, warmup, "w")
+    res["prefill"] = {"ms": round(pre_ms, 3), "tokens_per_s": round(T / pre_ms * 1e3, 1)}
+    res["decode_b8"] = {"ms_per_step": round(b8, 4), "tokens_per_s": round(8 / b8 * 1e3, 1)}
+    res["decode_b64"] = {"ms_per_step": round(b64, 4), "tokens_per_s": round(64 / b64 * 1e3, 1)}
+    spans = {k: [] for k in kinds}
+    real = {k: getattr(v[0], v[1]) for k, v in kinds.items()}
+
+    def timed(kind):
+        def call(*x, **kw):
+            e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+            e0.record()
+            out = real[kind](*x, **kw)
+            e1.record()
+            spans[kind].append((e0, e1))
+            return out
+        return call
+
+    def step_times(run):
+        best = {}
+        for _ in range(4):
+            for k in spans:
+                spans[k].clear()
+            run()
+            torch.cuda.synchronize()
+            for k, evs in spans.items():
+                us = sum(e0.elapsed_time(e1) for e0, e1 in evs) * 1e3
+                best[k] = min(best.get(k, us), us)
+        return best
+
+    toks = torch.randint(0, eng.config.vocab_size, (T,), generator=torch.Generator().manual_seed(3)).tolist()
+    rids = [f"k{i}" for i in range(64)]
+    count = [0]
+
+    def run_prefill():
+        count[0] += 1
+        eng.manager.add_request(f"kp{count[0]}")
+        eng.runner.step([StepEntry(f"kp{count[0]}", toks, (T - 1,))])
+        eng.manager.free_request(f"kp{count[0]}")
+
+    def run_decode():
+        eng.runner.step([StepEntry(r, [toks[j]], (0,)) for j, r in enumerate(rids)])
+
+    graphs, eng.runner.use_graphs = eng.runner.use_graphs, False
+    for k, v in kinds.items():
+        setattr(v[0], v[1], timed(k))
+    try:
+        pre_t = step_times(run_prefill)
+        fill_contexts(eng, rids, ctx_len)
+        fill_states(eng)
+        dec_t = step_times(run_decode)
+    finally:
+        for k, v in kinds.items():
+            setattr(v[0], v[1], real[k])
+        eng.runner.use_graphs = graphs
+    for r in rids:
+        eng.manager.free_request(r)
+    res["kernels"] = {}
+    for kind, (_, _, work_p, work_d, bound) in kinds.items():
+        pre_us, dec_us = max(pre_t[kind], 1e-3), max(dec_t[kind], 1e-3)
+        row = {"prefill_us": round(pre_us, 1), "decode_b64_us": round(dec_us, 1)}
+        if bound == "hbm":
+            row["prefill_frac_of_hbm"] = round(work_p(T) / pre_us / 1e3 / pk["hbm_gbs"], 4)
+        elif bound == "fp32":
+            row["prefill_frac_of_nominal_fp32"] = round(work_p(T) / pre_us * 1e6 / fp32_peak, 4)
+        else:
+            row["prefill_frac_of_bf16_peak"] = round(work_p(T) / pre_us * 1e6 / (pk["bf16_tflops"] * 1e12), 4)
+        row["decode_b64_frac_of_hbm"] = round(work_d(64) / dec_us / 1e3 / pk["hbm_gbs"], 4)
+        res["kernels"][kind] = row
+    return res
+
+
 # ---------------------------------------------------------------------------------------------------------
 # The Pogarax design beside the Vedizen design at equal size (--workload pogarax)
 def pogarax_pair(size: dict):
@@ -729,6 +812,39 @@ def pogarax_pair(size: dict):
     return pog, vedizen_pair(size)[0]
 
 
+def pogarax_kinds(size: dict, ctx_len: int) -> dict:
+    """Kind -> (module, function, work at t tokens of one prompt, work at a batch of b single tokens, bound)."""
+    from airun_b200.kernels import fast, ops
+    from airun_b200.parts import latent_attention as latent_part
+    W, F, H = size["width"], size["ff"], size["heads"]
+    win = lambda t: sum(min(i + 1, 2048) for i in range(t))      # keys all tokens of a t-token prompt see together
+    R, rd, D, Dv, qr, Fe, E, top, Hw = 512, 64, 128, 128, W // 2, F // 2, 16, 2, W // 64
+    return {
+        "norm on the output + add (rms)": (ops, "postnorm_add", lambda t: 12 * t * W * 14.0, lambda b: 12 * b * W * 14.0, "hbm"),
+        "latent: norms, rotation, cache write": (ops, "latent_prepare", lambda t: 2 * t * ((qr + R + rd) * 4.0 + qr * 2 + (R + rd)),
+                                                 lambda b: 2 * b * ((qr + R + rd) * 4.0 + qr * 2 + (R + rd)), "hbm"),
+        "latent: query parts and rotation": (ops, "latent_query", lambda t: 2 * t * H * ((D + rd) * 4.0 + (D + rd) * 2),
+                                             lambda b: 2 * b * H * ((D + rd) * 4.0 + (D + rd) * 2), "hbm"),
+        "latent attention": (fast, "latent_attention_bf16", lambda t: 2 * H * 2.0 * (2 * R + rd) * win(t),
+                             lambda b: 2 * b * min(ctx_len, 2048) * (R + rd) * 2.0, "mixed"),
+        "products per head (Wuk, Wuv)": (latent_part, "head_linear", lambda t: 2 * t * H * 2.0 * (D * R + R * Dv),
+                                         lambda b: 2 * H * (D * R + R * Dv) * 2.0, "tensor"),
+        "delta rule: convolution": (ops, "short_conv", lambda t: 3 * t * (H * 64 + H * 128) * 8.0, lambda b: 3 * b * (H * 64 + H * 128) * 8.0, "hbm"),
+        "low-rank second halves (decays, gate)": (ops, "lowrank_act", lambda t: t * (3 * (H * 64 + H * 128) + W) * 4.0,
+                                                  lambda b: b * (3 * (H * 64 + H * 128) + W) * 4.0, "hbm"),
+        "recurrence (delta rule, time mix)": (ops, "recurrent_state", lambda t: t * (3 * H * 64 * 128 * 9.0 + Hw * 64 * 64 * 6.0),
+                                              lambda b: b * (3 * H * 64 * 128 + Hw * 64 * 64) * 8.0, "fp32"),
+        "norm and gate of the heads": (ops, "gla_out_gate", lambda t: t * (3 * H * 128 + W) * 10.0, lambda b: b * (3 * H * 128 + W) * 10.0, "hbm"),
+        "token shift": (ops, "token_shift", lambda t: t * W * 14.0, lambda b: b * W * 14.0, "hbm"),
+        "gate/up product + gated unit (dense)": (fast, "linear_swiglu_bf16", lambda t: 3 * 2.0 * t * W * 2 * F, lambda b: 3 * W * 2 * F * 2.0, "tensor"),
+        "expert products (gate/up + unit, down)": (fast, "grouped_linear_bf16", lambda t: 3 * t * top * 6.0 * W * Fe,
+                                                   lambda b: 3 * min(E, b * top) * 3 * W * Fe * 2.0, "tensor"),
+        "router": (ops, "moe_route", lambda t: 3 * t * W * 2.0, lambda b: 3 * (b * W + E * W) * 2.0, "hbm"),
+        "rows to experts and back": (ops, "moe_scatter", lambda t: 3 * t * (W * 2 + top * W * 2.0), lambda b: 3 * b * (W * 2 + top * W * 2.0), "hbm"),
+        "sum of a token's experts": (ops, "moe_combine", lambda t: 3 * t * (top + 1) * W * 4.0, lambda b: 3 * b * (top + 1) * W * 4.0, "hbm"),
+    }
+
+
 def workload_pogarax(a) -> int:
     """Prefill (one 2,048-token prompt) and decode (batch 8 and 64 at a context of 1,024) of the Pogarax design and of
     the Vedizen design at equal size, through the step function and its CUDA graphs, and how long each kind of kernel
@@ -736,12 +852,10 @@ def workload_pogarax(a) -> int:
     launched kernel by kernel), with the fraction of the measured peak its bytes or FLOPs over that time come to.  One
     JSON line per size."""
     import torch
-    from airun_b200 import Engine, EngineOptions, StepEntry
+    from airun_b200 import Engine, EngineOptions
     from airun_b200.kernels import fast, ops
-    from airun_b200.parts import latent_attention as latent_part
     pk = peaks()
     T, ctx_len, steps = 2048, 1024, max(8, min(a.steps, 32))
-    fp32_peak = 148 * 128 * 2 * 1.965e9          # FMA lanes x 2 x the highest SM clock: nominal, no measured figure
     for name in (a.sizes.split(",") if a.sizes else list(VEDIZEN_SIZES)):
         size = VEDIZEN_SIZES[name]
         W, F, H, G = size["width"], size["ff"], size["heads"], size["kv_heads"]
@@ -751,34 +865,9 @@ def workload_pogarax(a) -> int:
             eng = Engine.from_config(cfg, seed=0, options=EngineOptions(
                 dtype="bfloat16", page_size=16, cache_tokens=64 * (ctx_len + 4 * steps + 64) + 4096, max_batch_tokens=T,
                 max_requests=64, max_context=max(T, ctx_len + 4 * steps + 64)))
-            win = lambda t: sum(min(i + 1, 2048) for i in range(t))      # keys all tokens of a t-token prompt see together
-            # kind -> (module, function, work at t tokens of one prompt or None, work at a batch of b single tokens, bound)
+            # kind -> (module, function, work at t tokens of one prompt, work at a batch of b single tokens, bound)
             if model == "pogarax":
-                R, rd, D, Dv, qr, Fe, E, top, Hw = 512, 64, 128, 128, W // 2, F // 2, 16, 2, W // 64
-                kinds = {
-                    "norm on the output + add (rms)": (ops, "postnorm_add", lambda t: 12 * t * W * 14.0, lambda b: 12 * b * W * 14.0, "hbm"),
-                    "latent: norms, rotation, cache write": (ops, "latent_prepare", lambda t: 2 * t * ((qr + R + rd) * 4.0 + qr * 2 + (R + rd)),
-                                                             lambda b: 2 * b * ((qr + R + rd) * 4.0 + qr * 2 + (R + rd)), "hbm"),
-                    "latent: query parts and rotation": (ops, "latent_query", lambda t: 2 * t * H * ((D + rd) * 4.0 + (D + rd) * 2),
-                                                         lambda b: 2 * b * H * ((D + rd) * 4.0 + (D + rd) * 2), "hbm"),
-                    "latent attention": (fast, "latent_attention_bf16", lambda t: 2 * H * 2.0 * (2 * R + rd) * win(t),
-                                         lambda b: 2 * b * min(ctx_len, 2048) * (R + rd) * 2.0, "mixed"),
-                    "products per head (Wuk, Wuv)": (latent_part, "head_linear", lambda t: 2 * t * H * 2.0 * (D * R + R * Dv),
-                                                     lambda b: 2 * H * (D * R + R * Dv) * 2.0, "tensor"),
-                    "delta rule: convolution": (ops, "short_conv", lambda t: 3 * t * (H * 64 + H * 128) * 8.0, lambda b: 3 * b * (H * 64 + H * 128) * 8.0, "hbm"),
-                    "low-rank second halves (decays, gate)": (ops, "lowrank_act", lambda t: t * (3 * (H * 64 + H * 128) + W) * 4.0,
-                                                              lambda b: b * (3 * (H * 64 + H * 128) + W) * 4.0, "hbm"),
-                    "recurrence (delta rule, time mix)": (ops, "recurrent_state", lambda t: t * (3 * H * 64 * 128 * 9.0 + Hw * 64 * 64 * 6.0),
-                                                          lambda b: b * (3 * H * 64 * 128 + Hw * 64 * 64) * 8.0, "fp32"),
-                    "norm and gate of the heads": (ops, "gla_out_gate", lambda t: t * (3 * H * 128 + W) * 10.0, lambda b: b * (3 * H * 128 + W) * 10.0, "hbm"),
-                    "token shift": (ops, "token_shift", lambda t: t * W * 14.0, lambda b: b * W * 14.0, "hbm"),
-                    "gate/up product + gated unit (dense)": (fast, "linear_swiglu_bf16", lambda t: 3 * 2.0 * t * W * 2 * F, lambda b: 3 * W * 2 * F * 2.0, "tensor"),
-                    "expert products (gate/up + unit, down)": (fast, "grouped_linear_bf16", lambda t: 3 * t * top * 6.0 * W * Fe,
-                                                               lambda b: 3 * min(E, b * top) * 3 * W * Fe * 2.0, "tensor"),
-                    "router": (ops, "moe_route", lambda t: 3 * t * W * 2.0, lambda b: 3 * (b * W + E * W) * 2.0, "hbm"),
-                    "rows to experts and back": (ops, "moe_scatter", lambda t: 3 * t * (W * 2 + top * W * 2.0), lambda b: 3 * b * (W * 2 + top * W * 2.0), "hbm"),
-                    "sum of a token's experts": (ops, "moe_combine", lambda t: 3 * t * (top + 1) * W * 4.0, lambda b: 3 * b * (top + 1) * W * 4.0, "hbm"),
-                }
+                kinds = pogarax_kinds(size, ctx_len)
             else:
                 n_att, n_gla = 3, 3
                 kinds = {
@@ -793,78 +882,7 @@ def workload_pogarax(a) -> int:
                     "linear attention: norm and gate": (ops, "gla_out_gate", lambda t: n_gla * t * H * 128 * 10.0, lambda b: n_gla * b * H * 128 * 10.0, "hbm"),
                     "gate/up product + gated unit": (fast, "linear_glu_clamped_bf16", lambda t: 6 * 2.0 * t * W * 2 * F, lambda b: 6 * W * 2 * F * 2.0, "tensor"),
                 }
-            res = {}
-            pre_ms = time_prefill(eng, T, runs=5)
-            b64 = time_decode_onward(eng, 64, ctx_len, steps, a.warmup, "v")
-            b8 = time_decode_onward(eng, 8, ctx_len, steps, a.warmup, "w")
-            res["prefill"] = {"ms": round(pre_ms, 3), "tokens_per_s": round(T / pre_ms * 1e3, 1)}
-            res["decode_b8"] = {"ms_per_step": round(b8, 4), "tokens_per_s": round(8 / b8 * 1e3, 1)}
-            res["decode_b64"] = {"ms_per_step": round(b64, 4), "tokens_per_s": round(64 / b64 * 1e3, 1)}
-            spans = {k: [] for k in kinds}
-            real = {k: getattr(v[0], v[1]) for k, v in kinds.items()}
-
-            def timed(kind):
-                def call(*x, **kw):
-                    e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
-                    e0.record()
-                    out = real[kind](*x, **kw)
-                    e1.record()
-                    spans[kind].append((e0, e1))
-                    return out
-                return call
-
-            def step_times(run):
-                best = {}
-                for _ in range(4):
-                    for k in spans:
-                        spans[k].clear()
-                    run()
-                    torch.cuda.synchronize()
-                    for k, evs in spans.items():
-                        us = sum(e0.elapsed_time(e1) for e0, e1 in evs) * 1e3
-                        best[k] = min(best.get(k, us), us)
-                return best
-
-            toks = torch.randint(0, eng.config.vocab_size, (T,), generator=torch.Generator().manual_seed(3)).tolist()
-            rids = [f"k{i}" for i in range(64)]
-            count = [0]
-
-            def run_prefill():
-                count[0] += 1
-                eng.manager.add_request(f"kp{count[0]}")
-                eng.runner.step([StepEntry(f"kp{count[0]}", toks, (T - 1,))])
-                eng.manager.free_request(f"kp{count[0]}")
-
-            def run_decode():
-                eng.runner.step([StepEntry(r, [toks[j]], (0,)) for j, r in enumerate(rids)])
-
-            graphs, eng.runner.use_graphs = eng.runner.use_graphs, False
-            for k, v in kinds.items():
-                setattr(v[0], v[1], timed(k))
-            try:
-                pre_t = step_times(run_prefill)
-                fill_contexts(eng, rids, ctx_len)
-                fill_states(eng)
-                dec_t = step_times(run_decode)
-            finally:
-                for k, v in kinds.items():
-                    setattr(v[0], v[1], real[k])
-                eng.runner.use_graphs = graphs
-            for r in rids:
-                eng.manager.free_request(r)
-            res["kernels"] = {}
-            for kind, (_, _, work_p, work_d, bound) in kinds.items():
-                pre_us, dec_us = max(pre_t[kind], 1e-3), max(dec_t[kind], 1e-3)
-                row = {"prefill_us": round(pre_us, 1), "decode_b64_us": round(dec_us, 1)}
-                if bound == "hbm":
-                    row["prefill_frac_of_hbm"] = round(work_p(T) / pre_us / 1e3 / pk["hbm_gbs"], 4)
-                elif bound == "fp32":
-                    row["prefill_frac_of_nominal_fp32"] = round(work_p(T) / pre_us * 1e6 / fp32_peak, 4)
-                else:
-                    row["prefill_frac_of_bf16_peak"] = round(work_p(T) / pre_us * 1e6 / (pk["bf16_tflops"] * 1e12), 4)
-                row["decode_b64_frac_of_hbm"] = round(work_d(64) / dec_us / 1e3 / pk["hbm_gbs"], 4)
-                res["kernels"][kind] = row
-            line["models"][model] = res
+            line["models"][model] = measure_design(eng, kinds, T, ctx_len, steps, a.warmup, pk)
             del eng
             torch.cuda.empty_cache()
         print(json.dumps(line), flush=True)
@@ -900,7 +918,7 @@ def workload_gamanex(a) -> int:
     launched kernel by kernel), with the fraction of the measured peak its bytes or FLOPs over that time come to.  One
     JSON line per size."""
     import torch
-    from airun_b200 import Engine, EngineOptions, StepEntry
+    from airun_b200 import Engine, EngineOptions
     from airun_b200.kernels import fast, ops
     pk = peaks()
     T, ctx_len, steps = 2048, 1024, max(8, min(a.steps, 32))
@@ -940,75 +958,7 @@ def workload_gamanex(a) -> int:
                     "gate/up product + gated unit": (fast, "linear_swiglu_bf16", lambda t: 6 * 2.0 * t * W * 2 * F, lambda b: 6 * W * 2 * F * 2.0, "tensor"),
                 }
             kinds = {k: v for k, v in kinds.items() if hasattr(v[0], v[1])}
-            res = {}
-            pre_ms = time_prefill(eng, T, runs=5)
-            b64 = time_decode_onward(eng, 64, ctx_len, steps, a.warmup, "v")
-            b8 = time_decode_onward(eng, 8, ctx_len, steps, a.warmup, "w")
-            res["prefill"] = {"ms": round(pre_ms, 3), "tokens_per_s": round(T / pre_ms * 1e3, 1)}
-            res["decode_b8"] = {"ms_per_step": round(b8, 4), "tokens_per_s": round(8 / b8 * 1e3, 1)}
-            res["decode_b64"] = {"ms_per_step": round(b64, 4), "tokens_per_s": round(64 / b64 * 1e3, 1)}
-            spans = {k: [] for k in kinds}
-            real = {k: getattr(v[0], v[1]) for k, v in kinds.items()}
-
-            def timed(kind):
-                def call(*x, **kw):
-                    e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
-                    e0.record()
-                    out = real[kind](*x, **kw)
-                    e1.record()
-                    spans[kind].append((e0, e1))
-                    return out
-                return call
-
-            def step_times(run):
-                best = {}
-                for _ in range(4):
-                    for k in spans:
-                        spans[k].clear()
-                    run()
-                    torch.cuda.synchronize()
-                    for k, evs in spans.items():
-                        us = sum(e0.elapsed_time(e1) for e0, e1 in evs) * 1e3
-                        best[k] = min(best.get(k, us), us)
-                return best
-
-            toks = torch.randint(0, eng.config.vocab_size, (T,), generator=torch.Generator().manual_seed(3)).tolist()
-            rids = [f"k{i}" for i in range(64)]
-            count = [0]
-
-            def run_prefill():
-                count[0] += 1
-                eng.manager.add_request(f"kp{count[0]}")
-                eng.runner.step([StepEntry(f"kp{count[0]}", toks, (T - 1,))])
-                eng.manager.free_request(f"kp{count[0]}")
-
-            def run_decode():
-                eng.runner.step([StepEntry(r, [toks[j]], (0,)) for j, r in enumerate(rids)])
-
-            graphs, eng.runner.use_graphs = eng.runner.use_graphs, False
-            for k, v in kinds.items():
-                setattr(v[0], v[1], timed(k))
-            try:
-                pre_t = step_times(run_prefill)
-                fill_contexts(eng, rids, ctx_len)
-                dec_t = step_times(run_decode)
-            finally:
-                for k, v in kinds.items():
-                    setattr(v[0], v[1], real[k])
-                eng.runner.use_graphs = graphs
-            for r in rids:
-                eng.manager.free_request(r)
-            res["kernels"] = {}
-            for kind, (_, _, work_p, work_d, bound) in kinds.items():
-                pre_us, dec_us = max(pre_t[kind], 1e-3), max(dec_t[kind], 1e-3)
-                row = {"prefill_us": round(pre_us, 1), "decode_b64_us": round(dec_us, 1)}
-                if bound == "hbm":
-                    row["prefill_frac_of_hbm"] = round(work_p(T) / pre_us / 1e3 / pk["hbm_gbs"], 4)
-                else:
-                    row["prefill_frac_of_bf16_peak"] = round(work_p(T) / pre_us * 1e6 / (pk["bf16_tflops"] * 1e12), 4)
-                row["decode_b64_frac_of_hbm"] = round(work_d(64) / dec_us / 1e3 / pk["hbm_gbs"], 4)
-                res["kernels"][kind] = row
-            line["models"][model] = res
+            line["models"][model] = measure_design(eng, kinds, T, ctx_len, steps, a.warmup, pk)
             del eng
             torch.cuda.empty_cache()
         print(json.dumps(line), flush=True)
@@ -1039,6 +989,32 @@ def tagulix_pair(size: dict):
     return tag, vedizen_pair(size)[1]
 
 
+def tagulix_kinds(size: dict, ctx_len: int) -> dict:
+    """Kind -> (module, function, work at t tokens of one prompt, work at a batch of b single tokens, bound)."""
+    from airun_b200.kernels import fast, ops
+    W, F, H, G = size["width"], size["ff"], size["heads"], size["kv_heads"]
+    tri = lambda t: t * (t + 1) / 2                                   # keys all tokens of a t-token prompt see together
+    win = lambda t: tri(min(t, 1024)) + max(0, t - 1024) * 1024.0     # the same under a window of 1,024
+    S, Fe, E, top, Hl = 4, F // 4, 16, 4, H // 2
+    lin_in, lin_out = Hl * (64 * 2 + 128 * 2) * 4.0, Hl * 128 * 4.0
+    return {
+        "streams: write, read and norm in one pass": (ops, "stream_step", lambda t: 13 * t * W * (8.0 * S + 6), lambda b: 13 * b * W * (8.0 * S + 6), "hbm"),
+        "q/k norm, rotation, temperature, cache write": (ops, "qkv_prepare", lambda t: 6 * t * (H + 2 * G) * 128 * 6.0,
+                                                         lambda b: 6 * b * (H + 2 * G) * 128 * 6.0, "hbm"),
+        "softmax attention (window; table and sink)": (fast, "softmax_attention_bf16", lambda t: 3 * H * 4.0 * 128 * (tri(t) + win(t)),
+                                                       lambda b: 6 * b * ctx_len * G * 256 * 2.0, "mixed"),
+        "decayed linear attention: recurrence": (ops, "decay_recurrent", lambda t: 3 * t * (lin_in - Hl * 128 * 4.0 + lin_out),
+                                                 lambda b: 3 * b * (Hl * 64 * 128 * 8.0), "hbm"),
+        "norm over all heads and gate": (ops, "rownorm_gate", lambda t: 3 * t * Hl * 128 * 10.0, lambda b: 3 * b * Hl * 128 * 10.0, "hbm"),
+        # a random router sends top * E / (E + 4) of a token's choices to experts with matrices
+        "expert products (up + GELU, down)": (fast, "grouped_linear_bf16", lambda t: 6 * t * (top * E / (E + 4.0)) * 4.0 * W * Fe,
+                                              lambda b: 6 * min(E, b * top) * 2 * W * Fe * 2.0, "tensor"),
+        "router with groups": (ops, "moe_route_grouped", lambda t: 6 * t * (E + 4 + 3 * top) * 4.0, lambda b: 6 * b * (E + 4 + 3 * top) * 4.0, "hbm"),
+        "rows to experts and back": (ops, "moe_scatter", lambda t: 6 * t * (W * 2 + top * W * 2.0), lambda b: 6 * b * (W * 2 + top * W * 2.0), "hbm"),
+        "sum of a token's experts": (ops, "moe_combine", lambda t: 6 * t * (top + 1) * W * 4.0, lambda b: 6 * b * (top + 1) * W * 4.0, "hbm"),
+    }
+
+
 def workload_tagulix(a) -> int:
     """Prefill (one 2,048-token prompt) and decode (batch 8 and 64 at a context of 1,024) of the Tagulix design and of
     the Qwen3 decoder at equal size, through the step function and its CUDA graphs, and how long each kind of kernel
@@ -1046,7 +1022,7 @@ def workload_tagulix(a) -> int:
     launched kernel by kernel), with the fraction of the measured peak its bytes or FLOPs over that time come to.  One
     JSON line per size."""
     import torch
-    from airun_b200 import Engine, EngineOptions, StepEntry
+    from airun_b200 import Engine, EngineOptions
     from airun_b200.kernels import fast, ops
     pk = peaks()
     T, ctx_len, steps = 2048, 1024, max(8, min(a.steps, 32))
@@ -1060,27 +1036,9 @@ def workload_tagulix(a) -> int:
                 dtype="bfloat16", page_size=16, cache_tokens=64 * (ctx_len + 4 * steps + 64) + 4096, max_batch_tokens=T,
                 max_requests=64, max_context=max(T, ctx_len + 4 * steps + 64)))
             tri = lambda t: t * (t + 1) / 2                                   # keys all tokens of a t-token prompt see together
-            win = lambda t: tri(min(t, 1024)) + max(0, t - 1024) * 1024.0     # the same under a window of 1,024
             # kind -> (module, function, work at t tokens of one prompt, work at a batch of b single tokens, bound)
             if model == "tagulix":
-                S, Fe, E, top, Hl = 4, F // 4, 16, 4, H // 2
-                lin_in, lin_out = Hl * (64 * 2 + 128 * 2) * 4.0, Hl * 128 * 4.0
-                kinds = {
-                    "streams: write, read and norm in one pass": (ops, "stream_step", lambda t: 13 * t * W * (8.0 * S + 6), lambda b: 13 * b * W * (8.0 * S + 6), "hbm"),
-                    "q/k norm, rotation, temperature, cache write": (ops, "qkv_prepare", lambda t: 6 * t * (H + 2 * G) * 128 * 6.0,
-                                                                     lambda b: 6 * b * (H + 2 * G) * 128 * 6.0, "hbm"),
-                    "softmax attention (window; table and sink)": (fast, "softmax_attention_bf16", lambda t: 3 * H * 4.0 * 128 * (tri(t) + win(t)),
-                                                                   lambda b: 6 * b * ctx_len * G * 256 * 2.0, "mixed"),
-                    "decayed linear attention: recurrence": (ops, "decay_recurrent", lambda t: 3 * t * (lin_in - Hl * 128 * 4.0 + lin_out),
-                                                             lambda b: 3 * b * (Hl * 64 * 128 * 8.0), "hbm"),
-                    "norm over all heads and gate": (ops, "rownorm_gate", lambda t: 3 * t * Hl * 128 * 10.0, lambda b: 3 * b * Hl * 128 * 10.0, "hbm"),
-                    # a random router sends top * E / (E + 4) of a token's choices to experts with matrices
-                    "expert products (up + GELU, down)": (fast, "grouped_linear_bf16", lambda t: 6 * t * (top * E / (E + 4.0)) * 4.0 * W * Fe,
-                                                          lambda b: 6 * min(E, b * top) * 2 * W * Fe * 2.0, "tensor"),
-                    "router with groups": (ops, "moe_route_grouped", lambda t: 6 * t * (E + 4 + 3 * top) * 4.0, lambda b: 6 * b * (E + 4 + 3 * top) * 4.0, "hbm"),
-                    "rows to experts and back": (ops, "moe_scatter", lambda t: 6 * t * (W * 2 + top * W * 2.0), lambda b: 6 * b * (W * 2 + top * W * 2.0), "hbm"),
-                    "sum of a token's experts": (ops, "moe_combine", lambda t: 6 * t * (top + 1) * W * 4.0, lambda b: 6 * b * (top + 1) * W * 4.0, "hbm"),
-                }
+                kinds = tagulix_kinds(size, ctx_len)
             else:
                 kinds = {
                     "norm (rms)": (ops, "rmsnorm", lambda t: 13 * t * W * 14.0, lambda b: 13 * b * W * 14.0, "hbm"),
@@ -1090,75 +1048,70 @@ def workload_tagulix(a) -> int:
                     "gate/up product + gated unit": (fast, "linear_swiglu_bf16", lambda t: 6 * 2.0 * t * W * 2 * F, lambda b: 6 * W * 2 * F * 2.0, "tensor"),
                 }
             kinds = {k: v for k, v in kinds.items() if hasattr(v[0], v[1])}
-            res = {}
-            pre_ms = time_prefill(eng, T, runs=5)
-            b64 = time_decode_onward(eng, 64, ctx_len, steps, a.warmup, "v")
-            b8 = time_decode_onward(eng, 8, ctx_len, steps, a.warmup, "w")
-            res["prefill"] = {"ms": round(pre_ms, 3), "tokens_per_s": round(T / pre_ms * 1e3, 1)}
-            res["decode_b8"] = {"ms_per_step": round(b8, 4), "tokens_per_s": round(8 / b8 * 1e3, 1)}
-            res["decode_b64"] = {"ms_per_step": round(b64, 4), "tokens_per_s": round(64 / b64 * 1e3, 1)}
-            spans = {k: [] for k in kinds}
-            real = {k: getattr(v[0], v[1]) for k, v in kinds.items()}
+            line["models"][model] = measure_design(eng, kinds, T, ctx_len, steps, a.warmup, pk)
+            del eng
+            torch.cuda.empty_cache()
+        print(json.dumps(line), flush=True)
+    return 0
 
-            def timed(kind):
-                def call(*x, **kw):
-                    e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
-                    e0.record()
-                    out = real[kind](*x, **kw)
-                    e1.record()
-                    spans[kind].append((e0, e1))
-                    return out
-                return call
 
-            def step_times(run):
-                best = {}
-                for _ in range(4):
-                    for k in spans:
-                        spans[k].clear()
-                    run()
-                    torch.cuda.synchronize()
-                    for k, evs in spans.items():
-                        us = sum(e0.elapsed_time(e1) for e0, e1 in evs) * 1e3
-                        best[k] = min(best.get(k, us), us)
-                return best
+# The Losalorn design beside the Pogarax and the Tagulix design at equal size (--workload losalorn)
+def losalorn_config(size: dict):
+    """A Losalorn configuration of the width, head counts and vocabulary of the other designs' workloads and six layer
+    runs a token: layers 1 and 2 run twice.  Gated delta rule (heads x 64 x 128, q/k heads halved, 4 taps: Pogarax's
+    sizes) and attention (heads of 128, window 1,024, 64 dimensions rotated: Tagulix's "attention" layer) in turn, a dense
+    feed-forward in every layer."""
+    from airun_b200.config import LosalornConfig
+    W, F, H, G = size["width"], size["ff"], size["heads"], size["kv_heads"]
+    mlp = dict(kind="dense", ff=F, limit=7.0)
+    delta = dict(type="delta", mixer=dict(heads=H, kv_heads=H // 2, dim=64, vdim=128, conv=4), mlp=mlp)
+    att = dict(type="attention", mixer=dict(heads=H, kv_heads=G, dim=128, vdim=128, scale=128 ** -0.5, mask=dict(size=1024),
+                                            rot=dict(dims=64, base=50000.0, scaling=dict(factor=4.0, low=1.0, high=4.0, original=8192))), mlp=mlp)
+    return LosalornConfig.from_dict(dict(architecture="Losalorn", vocab=VEDIZEN_VOCAB, width=W, norm=dict(eps=1e-5), embedding=dict(scale=W ** 0.5),
+                                         logit_softcap=30.0, loop=dict(start=1, stop=3, times=2), layers=[delta, att, delta, att]))
 
-            toks = torch.randint(0, eng.config.vocab_size, (T,), generator=torch.Generator().manual_seed(3)).tolist()
-            rids = [f"k{i}" for i in range(64)]
-            count = [0]
 
-            def run_prefill():
-                count[0] += 1
-                eng.manager.add_request(f"kp{count[0]}")
-                eng.runner.step([StepEntry(f"kp{count[0]}", toks, (T - 1,))])
-                eng.manager.free_request(f"kp{count[0]}")
+def losalorn_kinds(size: dict, ctx_len: int) -> dict:
+    """Kind -> (module, function, work at t tokens of one prompt, work at a batch of b single tokens, bound)."""
+    from airun_b200.kernels import fast, ops
+    from airun_b200.parts.residual_input import MixWithEmbedding
+    W, F, H, G = size["width"], size["ff"], size["heads"], size["kv_heads"]
+    n_d, n_a = 3, 3                                                   # runs of each mixer among the six
+    tri = lambda t: t * (t + 1) / 2                                   # keys all tokens of a t-token prompt see together
+    win = lambda t: tri(min(t, 1024)) + max(0, t - 1024) * 1024.0     # the same under a window of 1,024
+    return {
+        "norms on both sides + add, in one pass": (ops, "sandwich_norm", lambda t: 12 * t * W * 14.0, lambda b: 12 * b * W * 14.0, "hbm"),
+        "stream mixed with the embedding (twice)": (MixWithEmbedding, "forward", lambda t: 2 * 4.0 * t * W * W, lambda b: 2 * 4.0 * W * W, "tensor"),
+        "rotation + cache write": (ops, "qkv_prepare", lambda t: n_a * t * (6 * H * 128 + G * (4 * 128 + 2 * 192.0)),
+                                   lambda b: n_a * b * (6 * H * 128 + G * (4 * 128 + 2 * 192.0)), "hbm"),
+        "attention (window; keys are the values)": (fast, "softmax_attention_bf16", lambda t: n_a * H * 4.0 * 128 * win(t),
+                                                    lambda b: n_a * b * min(ctx_len, 1024) * G * 192 * 2.0, "tensor"),
+        "delta rule: convolution": (ops, "short_conv", lambda t: n_d * t * (H * 64 + H * 128) * 8.0, lambda b: n_d * b * (H * 64 + H * 128) * 8.0, "hbm"),
+        "delta rule: recurrence": (ops, "recurrent_state", lambda t: t * n_d * H * 64 * 128 * 9.0, lambda b: b * n_d * H * 64 * 128 * 8.0, "fp32"),
+        "norm and gate of the heads": (ops, "gla_out_gate", lambda t: n_d * t * H * 128 * 10.0, lambda b: n_d * b * H * 128 * 10.0, "hbm"),
+        "gate/up product + gated unit": (fast, "linear_glu_clamped_bf16", lambda t: 6 * 2.0 * t * W * 2 * F, lambda b: 6 * W * 2 * F * 2.0, "tensor"),
+    }
 
-            def run_decode():
-                eng.runner.step([StepEntry(r, [toks[j]], (0,)) for j, r in enumerate(rids)])
 
-            graphs, eng.runner.use_graphs = eng.runner.use_graphs, False
-            for k, v in kinds.items():
-                setattr(v[0], v[1], timed(k))
-            try:
-                pre_t = step_times(run_prefill)
-                fill_contexts(eng, rids, ctx_len)
-                dec_t = step_times(run_decode)
-            finally:
-                for k, v in kinds.items():
-                    setattr(v[0], v[1], real[k])
-                eng.runner.use_graphs = graphs
-            for r in rids:
-                eng.manager.free_request(r)
-            res["kernels"] = {}
-            for kind, (_, _, work_p, work_d, bound) in kinds.items():
-                pre_us, dec_us = max(pre_t[kind], 1e-3), max(dec_t[kind], 1e-3)
-                row = {"prefill_us": round(pre_us, 1), "decode_b64_us": round(dec_us, 1)}
-                if bound == "hbm":
-                    row["prefill_frac_of_hbm"] = round(work_p(T) / pre_us / 1e3 / pk["hbm_gbs"], 4)
-                else:
-                    row["prefill_frac_of_bf16_peak"] = round(work_p(T) / pre_us * 1e6 / (pk["bf16_tflops"] * 1e12), 4)
-                row["decode_b64_frac_of_hbm"] = round(work_d(64) / dec_us / 1e3 / pk["hbm_gbs"], 4)
-                res["kernels"][kind] = row
-            line["models"][model] = res
+def workload_losalorn(a) -> int:
+    """Prefill (one 2,048-token prompt) and decode (batch 8 and 64 at a context of 1,024) of the Losalorn design, of the
+    Pogarax design (which has its gated delta rule with a decay per channel) and of the Tagulix design (which has its
+    windowed softmax attention) at equal size, and each kind of kernel inside those steps (``measure_design``).  One JSON
+    line per size."""
+    import torch
+    from airun_b200 import Engine, EngineOptions
+    pk = peaks()
+    T, ctx_len, steps = 2048, 1024, max(8, min(a.steps, 32))
+    for name in (a.sizes.split(",") if a.sizes else list(VEDIZEN_SIZES)):
+        size = VEDIZEN_SIZES[name]
+        line = {"workload": "losalorn", "size": size, "layer_runs": 6, "vocab": VEDIZEN_VOCAB, "dtype": "bf16",
+                "data": "synthetic, random weights", "prompt": T, "decode_context": ctx_len, "peaks": pk["source"], "models": {}}
+        for model, cfg, kinds in (("losalorn", losalorn_config(size), losalorn_kinds), ("pogarax", pogarax_pair(size)[0], pogarax_kinds),
+                                  ("tagulix", tagulix_pair(size)[0], tagulix_kinds)):
+            eng = Engine.from_config(cfg, seed=0, options=EngineOptions(
+                dtype="bfloat16", page_size=16, cache_tokens=64 * (ctx_len + 4 * steps + 64) + 4096, max_batch_tokens=T,
+                max_requests=64, max_context=max(T, ctx_len + 4 * steps + 64)))
+            line["models"][model] = measure_design(eng, kinds(size, ctx_len), T, ctx_len, steps, a.warmup, pk)
             del eng
             torch.cuda.empty_cache()
         print(json.dumps(line), flush=True)
@@ -1344,15 +1297,17 @@ def main() -> int:
     ap.add_argument("--skip-points", action="store_true")
     ap.add_argument("--decode-only", action="store_true", help="time the decode step only (for profiling runs)")
     ap.add_argument("--prefill-only", action="store_true", help="time the 2,048-token prompt only (for profiling runs)")
-    ap.add_argument("--workload", default="decode", choices=("decode", "serve", "long", "ablate", "vedizen", "pogarax", "gamanex", "tagulix"),
+    ap.add_argument("--workload", default="decode", choices=("decode", "serve", "long", "ablate", "vedizen", "pogarax", "gamanex", "tagulix",
+                                                               "losalorn"),
                     help="decode: the headline line; serve: 128 requests continuously batched (Qwen3-1.7B shape); "
                          "long: a 32,768-token prompt, then decoding alone and as 16 forks (Qwen3-32B shape); "
                          "ablate: the decode step timed with one kind of kernel left out at a time; "
                          "vedizen: prefill and decode of the Vedizen design beside the Qwen3 decoder at equal size; "
                          "pogarax: the same for the Pogarax design beside the Vedizen design; "
                          "gamanex: the same for the Gamanex design beside the Qwen3 decoder; "
-                         "tagulix: the same for the Tagulix design beside the Qwen3 decoder")
-    ap.add_argument("--sizes", default="", help="vedizen / pogarax / gamanex / tagulix: widths to run, comma separated (default: 2048,4096)")
+                         "tagulix: the same for the Tagulix design beside the Qwen3 decoder; "
+                         "losalorn: the same for the Losalorn design beside the Pogarax and the Tagulix design")
+    ap.add_argument("--sizes", default="", help="vedizen / pogarax / gamanex / tagulix / losalorn: widths to run, comma separated (default: 2048,4096)")
     ap.add_argument("--requests", type=int, default=128, help="serve: requests")
     ap.add_argument("--new-tokens", type=int, default=None, help="serve / long: tokens decoded per request")
     ap.add_argument("--budget", type=int, default=512, help="serve: tokens per step")
@@ -1381,6 +1336,8 @@ def main() -> int:
         return workload_gamanex(a)
     if a.workload == "tagulix":
         return workload_tagulix(a)
+    if a.workload == "losalorn":
+        return workload_losalorn(a)
 
     import torch
     from airun_b200 import Engine, EngineOptions, Qwen3Config
