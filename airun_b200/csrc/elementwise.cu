@@ -24,6 +24,17 @@ __global__ void embed_kernel(const TTab* __restrict__ table, const int32_t* __re
     const TTab* src = table + (size_t)id * H;
     float* dst = out + (size_t)t * H;
     // scale 1 (no scaling, as the reference) leaves the value as it is: x * 1.0f is exact
+    if ((H & 3) == 0 && ((uintptr_t)src & (4 * sizeof(TTab) - 1)) == 0 && ((uintptr_t)dst & 15) == 0) {
+#pragma unroll 4
+        for (int i = 4 * threadIdx.x; i < H; i += 4 * blockDim.x) {
+            __align__(16) TTab v[4];
+            if (sizeof(TTab) == 2) *reinterpret_cast<uint2*>(v) = *reinterpret_cast<const uint2*>(src + i);
+            else *reinterpret_cast<uint4*>(v) = *reinterpret_cast<const uint4*>(src + i);
+            *reinterpret_cast<float4*>(dst + i) = make_float4(to_f32<TTab>(v[0]) * scale, to_f32<TTab>(v[1]) * scale,
+                                                              to_f32<TTab>(v[2]) * scale, to_f32<TTab>(v[3]) * scale);
+        }
+        return;
+    }
     for (int i = threadIdx.x; i < H; i += blockDim.x) dst[i] = to_f32<TTab>(src[i]) * scale;
 }
 
@@ -397,14 +408,20 @@ AIRUN_EXPORT int airun_fill_random(void* out, int out_dtype, long long n, unsign
 __global__ void soft_cap_kernel(float* __restrict__ x, long long n, float cap) {
     pdl_trigger();
     pdl_wait();
-    const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
-    if (i < n) x[i] = cap * tanhf(x[i] / cap);
+    const long long i = 4 * ((long long)blockIdx.x * blockDim.x + threadIdx.x);
+    if (i + 4 <= n && ((uintptr_t)x & 15) == 0) {
+        float4 v = *reinterpret_cast<float4*>(x + i);
+        v.x = cap * tanhf(v.x / cap); v.y = cap * tanhf(v.y / cap); v.z = cap * tanhf(v.z / cap); v.w = cap * tanhf(v.w / cap);
+        *reinterpret_cast<float4*>(x + i) = v;
+    } else {
+        for (long long j = i; j < n && j < i + 4; ++j) x[j] = cap * tanhf(x[j] / cap);
+    }
 }
 
 AIRUN_EXPORT int airun_soft_cap(float* x, long long n, float cap, cudaStream_t stream) {
     if (n < 0 || !(cap > 0.0f)) return AIRUN_ERR_ARG;
     if (n == 0) return AIRUN_OK;
-    const long long blocks = (n + 255) / 256;
+    const long long blocks = (n + 1023) / 1024;
     if (blocks > 0x7fffffffll) return AIRUN_ERR_ARG;
     airun_launch(soft_cap_kernel, dim3((unsigned)blocks), dim3(256), 0, stream, x, n, cap);
     return airun_launch_status();

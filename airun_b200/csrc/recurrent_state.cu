@@ -62,6 +62,82 @@ __global__ __launch_bounds__(256) void short_conv_kernel(
     for (int c = n_unit_heads * unit_dim + threadIdx.x; c < C; c += blockDim.x) out[(size_t)t * C + c] = s_y[c];
 }
 
+// The same for 1 to 4 taps and everything in multiples of four on 16-byte boundaries.  A warp takes one unit (a head that is
+// made a unit vector, or 128 * NV of the remaining channels) of TOK consecutive rows of the batch, a lane four neighbouring
+// channels (NV times): the rows the tokens read are loaded at once, each of them once for all the taps it serves, and the
+// weights, which no kernel writes, before the kernel in front has finished.
+template <int TAPS, int NV, int TOK>
+__global__ __launch_bounds__(128) void short_conv_rows_kernel(
+    const float* __restrict__ in, long long in_stride, const float* __restrict__ w, const float* __restrict__ state,
+    long long slot_stride, long long tail_off, int max_slots, const int32_t* __restrict__ req_of_token,
+    const int32_t* __restrict__ cu_tokens, const int32_t* __restrict__ state_slots, int num_reqs, float* __restrict__ out, int T,
+    int C, int n_unit_heads, int q_heads, int unit_dim, float unit_eps, float q_scale, int* __restrict__ err) {
+    pdl_trigger();
+    const int lane = threadIdx.x & 31, unit = blockIdx.y * 4 + (threadIdx.x >> 5), t0 = blockIdx.x * TOK;
+    const bool is_head = unit < n_unit_heads;
+    const int c0 = is_head ? unit * unit_dim : n_unit_heads * unit_dim + (unit - n_unit_heads) * 128 * NV;
+    const int width = is_head ? unit_dim : min(128 * NV, C - c0);
+    if (width <= 0) return;
+    float wt[NV][4][TAPS];
+#pragma unroll
+    for (int v = 0; v < NV; ++v)
+#pragma unroll
+        for (int e = 0; e < 4; ++e)
+#pragma unroll
+            for (int j = 0; j < TAPS; ++j) wt[v][e][j] = 4 * lane + 128 * v < width ? w[(size_t)(c0 + 4 * lane + 128 * v + e) * TAPS + j] : 0.0f;
+    pdl_wait();
+    const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+    // rows t0 - (TAPS-1) .. t0 + TOK - 1; those ahead of the first token's request are not read
+    const int first_req = req_of_token[t0];
+    const int i0 = first_req >= 0 && first_req < num_reqs ? t0 - cu_tokens[first_req] : 0;
+    float4 x[TAPS - 1 + TOK][NV];
+#pragma unroll
+    for (int m = 0; m < TAPS - 1 + TOK; ++m) {
+        const int row = t0 - (TAPS - 1) + m;
+        const bool on = row < T && (m >= TAPS - 1 || i0 >= TAPS - 1 - m);
+#pragma unroll
+        for (int v = 0; v < NV; ++v)
+            x[m][v] = on && 4 * lane + 128 * v < width ? *reinterpret_cast<const float4*>(in + (size_t)row * in_stride + c0 + 4 * lane + 128 * v) : zero;
+    }
+#pragma unroll
+    for (int k = 0; k < TOK; ++k) {
+        const int t = t0 + k;
+        if (t >= T) return;
+        const int req = req_of_token[t];
+        if (req < 0) continue;
+        const int slot = req < num_reqs ? state_slots[req] : -1;
+        if (slot < 0 || slot >= max_slots) {
+            if (lane == 0) atomicOr(err, AIRUN_DEV_BAD_REQ);
+            continue;
+        }
+        const int i = t - cu_tokens[req];
+        const float* tail = state + (size_t)slot * slot_stride + tail_off;
+        float4 y[NV];
+        float ss = 0.0f;
+#pragma unroll
+        for (int v = 0; v < NV; ++v) {
+            const bool on = 4 * lane + 128 * v < width;
+            float4 acc = zero;
+#pragma unroll
+            for (int j = 0; j < TAPS; ++j) {
+                float4 xv = x[k + j][v];
+                if (i < TAPS - 1 - j) xv = on ? *reinterpret_cast<const float4*>(tail + (size_t)(i + j) * C + c0 + 4 * lane + 128 * v) : zero;
+                acc.x = fmaf(wt[v][0][j], xv.x, acc.x); acc.y = fmaf(wt[v][1][j], xv.y, acc.y);
+                acc.z = fmaf(wt[v][2][j], xv.z, acc.z); acc.w = fmaf(wt[v][3][j], xv.w, acc.w);
+            }
+            acc.x = acc.x / (1.0f + expf(-acc.x)); acc.y = acc.y / (1.0f + expf(-acc.y));
+            acc.z = acc.z / (1.0f + expf(-acc.z)); acc.w = acc.w / (1.0f + expf(-acc.w));
+            y[v] = acc;
+            ss = fmaf(acc.x, acc.x, fmaf(acc.y, acc.y, fmaf(acc.z, acc.z, fmaf(acc.w, acc.w, ss))));
+        }
+        const float inv = is_head ? (1.0f / sqrtf(warp_sum(ss) + unit_eps)) * (unit < q_heads ? q_scale : 1.0f) : 1.0f;
+#pragma unroll
+        for (int v = 0; v < NV; ++v)
+            if (4 * lane + 128 * v < width)
+                *reinterpret_cast<float4*>(out + (size_t)t * C + c0 + 4 * lane + 128 * v) = make_float4(y[v].x * inv, y[v].y * inv, y[v].z * inv, y[v].w * inv);
+    }
+}
+
 AIRUN_EXPORT int airun_short_conv(const float* in, long long in_stride, const float* w, int taps, const float* state,
                                   long long slot_stride, long long tail_off, int max_slots, const int32_t* req_of_token,
                                   const int32_t* cu_tokens, const int32_t* state_slots, int num_reqs, float* out, int T, int C,
@@ -71,6 +147,24 @@ AIRUN_EXPORT int airun_short_conv(const float* in, long long in_stride, const fl
         (long long)n_unit_heads * unit_dim > C || C > 48 * 1024 / 4)
         return AIRUN_ERR_ARG;
     if (T == 0) return AIRUN_OK;
+    const bool vec = taps <= 4 && C % 4 == 0 && in_stride % 4 == 0 && slot_stride % 4 == 0 && tail_off % 4 == 0 && unit_dim % 4 == 0 &&
+                     unit_dim <= 256 && (((uintptr_t)in | (uintptr_t)state | (uintptr_t)out) & 15) == 0;
+    if (vec) {
+        const int nv = n_unit_heads > 0 && unit_dim > 128 ? 2 : 1;
+        const dim3 units(1, ceil_div_i(n_unit_heads + ceil_div_i(C - n_unit_heads * unit_dim, 128 * nv), 4));
+#define SC_LAUNCH(TAPS, NV, TOK) \
+        airun_launch(short_conv_rows_kernel<TAPS, NV, TOK>, dim3(ceil_div_i(T, TOK), units.y), dim3(128), 0, stream, in, in_stride, w, state, \
+                     slot_stride, tail_off, max_slots, req_of_token, cu_tokens, state_slots, num_reqs, out, T, C, n_unit_heads, q_heads, \
+                     unit_dim, unit_eps, q_scale, err)
+#define SC_TOK(TAPS) do { if (nv == 2) SC_LAUNCH(TAPS, 2, 2); else if (T <= 128) SC_LAUNCH(TAPS, 1, 1); else SC_LAUNCH(TAPS, 1, 8); } while (0)
+        if (taps == 1) SC_TOK(1);
+        else if (taps == 2) SC_TOK(2);
+        else if (taps == 3) SC_TOK(3);
+        else SC_TOK(4);
+#undef SC_TOK
+#undef SC_LAUNCH
+        return airun_launch_status();
+    }
     airun_launch(short_conv_kernel, dim3(T), dim3(256), (size_t)C * sizeof(float), stream, in, in_stride, w, taps, state, slot_stride,
                  tail_off, max_slots, req_of_token, cu_tokens, state_slots, num_reqs, out, C, n_unit_heads, q_heads, unit_dim,
                  unit_eps, q_scale, err);
@@ -126,8 +220,8 @@ AIRUN_EXPORT int airun_token_shift(const float* x, const float* mu, int n_mix, c
 // one token to the next.  The key channels of a lane are every DG-th group of four, so the lanes of a column read
 // neighbouring float4 of the token's q, k and decay from shared memory.  (Eight lanes a column from 33 key channels
 // on: what bounds a prompt is the chain of its tokens, and a warp's instructions per token halve.)  Tokens are staged through shared memory
-// a few at a time by asynchronous copies into one of two stages.  The block (request, 0, 0) also moves the request's small state on: the last inputs of the
-// short convolution (delta rule) or the last token's x (time mix).
+// a few at a time by asynchronous copies into one of two stages.  The blocks of a request also move its small state on, a
+// share of the channels each: the last inputs of the short convolution (delta rule) or the last token's x (time mix).
 #define RS_TT 16
 #define RS_DELTA 0
 #define RS_WKV 1
@@ -143,10 +237,32 @@ struct RecurrentArgs {
     const int32_t* cu_tokens; const int32_t* state_slots;
     float* out;                                                          // [T][heads * Dv]
     int heads, kv_rep, D, Dv;                                            // head h reads q/k head h / kv_rep
-    // the small state moved on by block (r, 0, 0)
+    // the small state, moved on by all blocks of the request
     const float* tail_src; long long tail_src_stride; long long tail_off; int tail_rows, tail_width;
     int* err;
 };
+
+// The request's small state: its last `tail_rows` rows become the last rows of (what it held, then this step's rows).  A
+// thread owns whole columns; row s comes from a later row, so a batch of rows that is read before it is written, in
+// ascending order, never reads what was written.
+__device__ __forceinline__ void rs_move_tail(const RecurrentArgs& a, int slot, int t0, int n) {
+    if (a.tail_rows <= 0) return;
+    float* tail = a.state + (size_t)slot * a.slot_stride + a.tail_off;
+    const int R = a.tail_rows, Wd = a.tail_width, share = blockIdx.y * gridDim.z + blockIdx.z;
+    for (int c = share * blockDim.x + threadIdx.x; c < Wd; c += blockDim.x * gridDim.y * gridDim.z) {
+        for (int s0 = 0; s0 < R; s0 += 4) {
+            float v[4];
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+                const int src = s0 + i + n;
+                v[i] = s0 + i >= R ? 0.0f : src < R ? tail[(size_t)src * Wd + c] : a.tail_src[(size_t)(t0 + src - R) * a.tail_src_stride + c];
+            }
+#pragma unroll
+            for (int i = 0; i < 4; ++i)
+                if (s0 + i < R) tail[(size_t)(s0 + i) * Wd + c] = v[i];
+        }
+    }
+}
 
 __device__ __forceinline__ void rs_cp4(float* smem, const float* gmem) {
     asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"((uint32_t)__cvta_generic_to_shared(smem)), "l"(gmem) : "memory");
@@ -374,20 +490,280 @@ __global__ __launch_bounds__(128) void recurrent_state_kernel(RecurrentArgs a) {
             if (d < D) sbase[(size_t)d * Dv] = S[i];
         }
     }
-    // the small state: its last `tail_rows` rows become the last rows of (what it held, then this step's rows)
-    if (blockIdx.y == 0 && blockIdx.z == 0 && a.tail_rows > 0) {
-        float* tail = a.state + (size_t)slot * a.slot_stride + a.tail_off;
-        const int R = a.tail_rows, Wd = a.tail_width;
-        for (int c = threadIdx.x; c < Wd; c += 128) {
-            for (int s = 0; s < R; ++s) {            // row s comes from a later row: ascending s never reads what it wrote
-                const int src = s + n;
-                tail[(size_t)s * Wd + c] = src < R ? tail[(size_t)src * Wd + c]
-                                                   : a.tail_src[(size_t)(t0 + src - R) * a.tail_src_stride + c];
-            }
+    rs_move_tail(a, slot, t0, n);
+}
+
+// ------------------------------------------------------------------------------------------ chunks of eight tokens
+// The delta rule with one decay per head, eight tokens at a time.  With S0 the state ahead of a chunk, G_i = g_0 .. g_i and
+// L_ij = g_(j+1) .. g_i, unrolling the recurrence gives
+//     u_i + beta_i sum_{j<i} L_ij (k_i . k_j) u_j = beta_i (v_i - G_i S0^T k_i)
+//     o_i = G_i S0^T q_i + sum_{j<=i} L_ij (q_i . k_j) u_j
+//     S   = G_7 S0 + sum_j L_7j k_j u_j
+// The matrix on the left depends on keys, decays and betas alone: its inverse, times beta, is the same for every value
+// column.  delta_chunk_coef_kernel works out, for all chunks of all requests at once, the rows of that inverse, of
+// L_ij (q_i . k_j), G_i and L_7i (RS_COEF floats a token and head); delta_chunk_kernel then walks the chunks of a request.
+// The sums over key channels (S0^T k_i, S0^T q_i) of the eight tokens do not wait for one another, so a chunk costs one
+// chain of dot products, a few shuffles and one update of the state where eight tokens cost eight.  All float32.
+#define RS_CHUNK 8
+#define RS_COEF 20
+
+// Sums of x[0..N-1] over groups of N lanes: lane l of the group ends with the sum of x[l], in x[0].
+template <int N>
+__device__ __forceinline__ void rs_scatter_sum(float (&x)[N], int lane) {
+#pragma unroll
+    for (int off = N / 2; off >= 1; off >>= 1) {
+        const bool up = (lane & off) != 0;
+#pragma unroll
+        for (int j = 0; j < off; ++j) {
+            const float send = up ? x[j] : x[j + off], keep = up ? x[j + off] : x[j];
+            x[j] = keep + __shfl_xor_sync(0xffffffffu, send, off);
         }
     }
 }
 
+// One warp per (chunk, head); blockIdx.x counts the chunks of all requests.  coef [T][heads][RS_COEF].
+template <int SL>      // D <= 32 * SL
+__global__ __launch_bounds__(128) void delta_chunk_coef_kernel(RecurrentArgs a, int num_reqs, float* __restrict__ coef) {
+    pdl_trigger();
+    pdl_wait();
+    __shared__ float s_dot[4][64], s_m[4][RS_CHUNK][RS_CHUNK];
+    int b = blockIdx.x, row0 = -1, nt = 0;
+    for (int r = 0; r < num_reqs; ++r) {
+        const int t0 = a.cu_tokens[r], n = a.cu_tokens[r + 1] - t0;
+        if (n <= 0) continue;
+        const int chunks = (n + RS_CHUNK - 1) / RS_CHUNK;
+        if (b < chunks) { row0 = t0 + b * RS_CHUNK; nt = min(RS_CHUNK, n - b * RS_CHUNK); break; }
+        b -= chunks;
+    }
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, head = blockIdx.y * 4 + warp;
+    if (row0 < 0 || head >= a.heads) return;
+    const float* qh = a.q + (size_t)(head / a.kv_rep) * a.D;
+    const float* kh = a.k + (size_t)(head / a.kv_rep) * a.D;
+    // the 28 products k_i . k_j (j < i), then the 36 products q_i . k_j (j <= i)
+    float acc[64];
+#pragma unroll
+    for (int e = 0; e < 64; ++e) acc[e] = 0.0f;
+#pragma unroll
+    for (int sl = 0; sl < SL; ++sl) {
+        const int d = lane + 32 * sl;
+        float kk[RS_CHUNK], qq[RS_CHUNK];
+#pragma unroll
+        for (int i = 0; i < RS_CHUNK; ++i) {
+            const bool on = i < nt && d < a.D;
+            kk[i] = on ? kh[(size_t)(row0 + i) * a.k_stride + d] : 0.0f;
+            qq[i] = on ? qh[(size_t)(row0 + i) * a.q_stride + d] : 0.0f;
+        }
+        int e = 0;
+#pragma unroll
+        for (int i = 0; i < RS_CHUNK; ++i)
+#pragma unroll
+            for (int j = 0; j < i; ++j) { acc[e] = fmaf(kk[i], kk[j], acc[e]); ++e; }
+#pragma unroll
+        for (int i = 0; i < RS_CHUNK; ++i)
+#pragma unroll
+            for (int j = 0; j <= i; ++j) { acc[e] = fmaf(qq[i], kk[j], acc[e]); ++e; }
+    }
+    float half[2][32];
+    // 64 sums over 32 lanes: value 2l and 2l + 1 end in lane l
+#pragma unroll
+    for (int e = 0; e < 32; ++e) { half[0][e] = acc[2 * e]; half[1][e] = acc[2 * e + 1]; }
+    rs_scatter_sum<32>(half[0], lane);
+    rs_scatter_sum<32>(half[1], lane);
+    s_dot[warp][2 * lane] = half[0][0];
+    s_dot[warp][2 * lane + 1] = half[1][0];
+    __syncwarp();
+    const int c = lane & (RS_CHUNK - 1);                 // lanes 8.. repeat what lanes 0..7 do and store nothing
+    float g = 1.0f, beta = 0.0f;
+    if (c < nt) {
+        const float z = a.g[(size_t)(row0 + c) * a.g_stride + head] + a.dt_bias[head];
+        g = expf(-expf(a.a_log[head]) * (fmaxf(z, 0.0f) + log1pf(expf(-fabsf(z)))));
+        beta = 1.0f / (1.0f + expf(-a.beta[(size_t)(row0 + c) * a.beta_stride + head]));
+    }
+    // column c of L_ij k_i . k_j and of L_ij q_i . k_j; the decays up to and after token c
+    float qk[RS_CHUNK], before = 1.0f, after = 1.0f, L = 1.0f;
+#pragma unroll
+    for (int i = 0; i < RS_CHUNK; ++i) {
+        const float gi = __shfl_sync(0xffffffffu, g, i);
+        if (i <= c) before *= gi;
+        if (i > c) { after *= gi; L *= gi; }
+        qk[i] = i >= c ? L * s_dot[warp][28 + i * (i + 1) / 2 + c] : 0.0f;
+        if (lane < RS_CHUNK) s_m[warp][i][c] = i > c ? L * s_dot[warp][i * (i - 1) / 2 + c] : 0.0f;
+    }
+    __syncwarp();
+    // column c of (I + diag(beta) M)^-1 diag(beta) by forward substitution
+    float x[RS_CHUNK];
+#pragma unroll
+    for (int i = 0; i < RS_CHUNK; ++i) {
+        const float bi = __shfl_sync(0xffffffffu, beta, i);
+        float sum = 0.0f;
+#pragma unroll
+        for (int j = 0; j < i; ++j) sum = fmaf(s_m[warp][i][j], x[j], sum);
+        x[i] = i < c ? 0.0f : i == c ? bi : -bi * sum;
+    }
+    if (lane < RS_CHUNK) {
+        float* dst = coef + ((size_t)row0 * a.heads + head) * RS_COEF;
+        const size_t step = (size_t)a.heads * RS_COEF;
+#pragma unroll
+        for (int i = 0; i < RS_CHUNK; ++i)
+            if (i < nt) { dst[i * step + c] = x[i]; dst[i * step + RS_CHUNK + c] = qk[i]; }
+        if (c < nt) { dst[c * step + 2 * RS_CHUNK] = before; dst[c * step + 2 * RS_CHUNK + 1] = after; }
+    }
+}
+
+// One block per (request, head, 16 value columns), 128 threads: a column is shared by eight neighbouring lanes with NS key
+// channels each, and lane l of a column also stands for token l of the chunk.
+template <int NS>
+__global__ __launch_bounds__(128, NS <= 16 ? 4 : 1) void delta_chunk_kernel(RecurrentArgs a, const float* __restrict__ coef) {
+    pdl_trigger();
+    pdl_wait();
+    constexpr int DG = 8, DP = NS * DG, COLS = 16, TT = NS >= 32 ? 8 : 16;
+    __shared__ __align__(16) float s_q[2][TT][DP], s_k[2][TT][DP], s_v[2][TT][COLS], s_c[2][TT][RS_COEF];
+    const int r = blockIdx.x, head = blockIdx.y, col0 = blockIdx.z * COLS;
+    const int t0 = a.cu_tokens[r], n = a.cu_tokens[r + 1] - t0;
+    if (n <= 0) return;
+    const int slot = a.state_slots[r];
+    if (slot < 0 || slot >= a.max_slots) {
+        if (threadIdx.x == 0) atomicOr(a.err, AIRUN_DEV_BAD_REQ);
+        return;
+    }
+    const int D = a.D, Dv = a.Dv;
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    const int dg = lane & (DG - 1), cl = warp * (32 / DG) + lane / DG, col = col0 + cl;
+    const bool col_ok = col < Dv;
+    const int ncol = min(COLS, Dv - col0);
+    // both stages start as zeros: padding and rows beyond the last token hold numbers whose weight is zero
+    for (int e = threadIdx.x; e < 2 * TT * DP; e += 128) { (&s_q[0][0][0])[e] = 0.0f; (&s_k[0][0][0])[e] = 0.0f; }
+    for (int e = threadIdx.x; e < 2 * TT * COLS; e += 128) (&s_v[0][0][0])[e] = 0.0f;
+    __syncthreads();
+    const float* qh = a.q + (size_t)(head / a.kv_rep) * D;
+    const float* kh = a.k + (size_t)(head / a.kv_rep) * D;
+    const float* vh = a.v + (size_t)head * Dv + col0;
+    const bool vec = (D % 4 == 0) && ((a.q_stride | a.k_stride) % 4 == 0) && ((((uintptr_t)qh | (uintptr_t)kh) & 15) == 0);
+    const bool vvec = (ncol % 4 == 0) && (a.v_stride % 4 == 0) && (((uintptr_t)vh & 15) == 0);
+    auto stage = [&](int base, int buf) {
+        const int nt = min(TT, n - base);
+        if (vec) {
+            const int per = D / 4;
+            for (int e = threadIdx.x; e < nt * per; e += 128) {
+                const int tt = e / per, d = (e - tt * per) * 4;
+                const size_t row = (size_t)(t0 + base + tt);
+                rs_cp16(&s_q[buf][tt][d], qh + row * a.q_stride + d);
+                rs_cp16(&s_k[buf][tt][d], kh + row * a.k_stride + d);
+            }
+        } else {
+            for (int e = threadIdx.x; e < nt * D; e += 128) {
+                const int tt = e / D, d = e - tt * D;
+                const size_t row = (size_t)(t0 + base + tt);
+                rs_cp4(&s_q[buf][tt][d], qh + row * a.q_stride + d);
+                rs_cp4(&s_k[buf][tt][d], kh + row * a.k_stride + d);
+            }
+        }
+        if (vvec) {
+            const int per = ncol / 4;
+            for (int e = threadIdx.x; e < nt * per; e += 128) {
+                const int tt = e / per, c = (e - tt * per) * 4;
+                rs_cp16(&s_v[buf][tt][c], vh + (size_t)(t0 + base + tt) * a.v_stride + c);
+            }
+        } else {
+            for (int e = threadIdx.x; e < nt * ncol; e += 128) {
+                const int tt = e / ncol, c = e - tt * ncol;
+                rs_cp4(&s_v[buf][tt][c], vh + (size_t)(t0 + base + tt) * a.v_stride + c);
+            }
+        }
+        for (int e = threadIdx.x; e < TT * (RS_COEF / 4); e += 128) {
+            const int tt = e / (RS_COEF / 4), c = (e - tt * (RS_COEF / 4)) * 4;
+            if (tt < nt) rs_cp16(&s_c[buf][tt][c], coef + ((size_t)(t0 + base + tt) * a.heads + head) * RS_COEF + c);
+            else *reinterpret_cast<float4*>(&s_c[buf][tt][c]) = make_float4(0.f, 0.f, 0.f, 0.f);
+        }
+        asm volatile("cp.async.commit_group;" ::: "memory");
+    };
+    stage(0, 0);
+    float* sbase = a.state + (size_t)slot * a.slot_stride + (size_t)head * D * Dv + (col_ok ? col : 0);
+    float S[NS];                                  // channel of register i: group of four (i / 4) * DG + dg, element i % 4
+#pragma unroll
+    for (int i = 0; i < NS; ++i) {
+        const int d = ((i >> 2) * DG + dg) * 4 + (i & 3);
+        S[i] = (col_ok && d < D) ? sbase[(size_t)d * Dv] : 0.0f;
+    }
+    float* orow = a.out + (size_t)t0 * ((size_t)a.heads * Dv) + (size_t)head * Dv + col;
+    int it = 0;
+    for (int base = 0; base < n; base += TT, ++it) {
+        const int buf = it & 1;
+        if (base + TT < n) {
+            stage(base + TT, buf ^ 1);            // that stage was last read before the barrier that ended the iteration before
+            asm volatile("cp.async.wait_group 1;" ::: "memory");
+        } else {
+            asm volatile("cp.async.wait_group 0;" ::: "memory");
+        }
+        __syncthreads();
+#pragma unroll 1
+        for (int c0 = 0; c0 < TT && base + c0 < n; c0 += RS_CHUNK) {
+            const int nt = min(RS_CHUNK, n - base - c0);
+            float p[RS_CHUNK], oq[RS_CHUNK];
+#pragma unroll
+            for (int i = 0; i < RS_CHUNK; ++i) { p[i] = 0.0f; oq[i] = 0.0f; }
+#pragma unroll
+            for (int i4 = 0; i4 < NS / 4; ++i4) {
+#pragma unroll
+                for (int i = 0; i < RS_CHUNK; ++i) {
+                    const float4 k4 = *reinterpret_cast<const float4*>(&s_k[buf][c0 + i][(i4 * DG + dg) * 4]);
+                    const float4 q4 = *reinterpret_cast<const float4*>(&s_q[buf][c0 + i][(i4 * DG + dg) * 4]);
+                    p[i] = fmaf(S[4 * i4 + 0], k4.x, p[i]); oq[i] = fmaf(S[4 * i4 + 0], q4.x, oq[i]);
+                    p[i] = fmaf(S[4 * i4 + 1], k4.y, p[i]); oq[i] = fmaf(S[4 * i4 + 1], q4.y, oq[i]);
+                    p[i] = fmaf(S[4 * i4 + 2], k4.z, p[i]); oq[i] = fmaf(S[4 * i4 + 2], q4.z, oq[i]);
+                    p[i] = fmaf(S[4 * i4 + 3], k4.w, p[i]); oq[i] = fmaf(S[4 * i4 + 3], q4.w, oq[i]);
+                }
+            }
+            rs_scatter_sum<RS_CHUNK>(p, lane);
+            rs_scatter_sum<RS_CHUNK>(oq, lane);
+            // this lane's token from here on: c0 + dg
+            const float* cf = &s_c[buf][c0 + dg][0];
+            const float4 ta = *reinterpret_cast<const float4*>(cf), tb = *reinterpret_cast<const float4*>(cf + 4);
+            const float4 qa = *reinterpret_cast<const float4*>(cf + 8), qb = *reinterpret_cast<const float4*>(cf + 12);
+            const float2 dec = *reinterpret_cast<const float2*>(cf + 16);         // decay up to the token; from after it to the chunk's end
+            const float rest = fmaf(-dec.x, p[0], s_v[buf][c0 + dg][cl]);
+            const float tm[RS_CHUNK] = {ta.x, ta.y, ta.z, ta.w, tb.x, tb.y, tb.z, tb.w};
+            const float qk[RS_CHUNK] = {qa.x, qa.y, qa.z, qa.w, qb.x, qb.y, qb.z, qb.w};
+            float u0 = 0.0f, u1 = 0.0f;
+#pragma unroll
+            for (int j = 0; j < RS_CHUNK; j += 2) {
+                u0 = fmaf(tm[j], __shfl_sync(0xffffffffu, rest, j, DG), u0);
+                u1 = fmaf(tm[j + 1], __shfl_sync(0xffffffffu, rest, j + 1, DG), u1);
+            }
+            const float u = u0 + u1, ul = u * dec.y;
+            const float whole = __shfl_sync(0xffffffffu, dec.x, nt - 1, DG);
+#pragma unroll
+            for (int i = 0; i < NS; ++i) S[i] *= whole;
+            float o0 = dec.x * oq[0], o1 = 0.0f;
+#pragma unroll
+            for (int j = 0; j < RS_CHUNK; ++j) {
+                const float uj = __shfl_sync(0xffffffffu, u, j, DG), wj = __shfl_sync(0xffffffffu, ul, j, DG);
+                if (j & 1) o1 = fmaf(qk[j], uj, o1);
+                else o0 = fmaf(qk[j], uj, o0);
+#pragma unroll
+                for (int i4 = 0; i4 < NS / 4; ++i4) {
+                    const float4 k4 = *reinterpret_cast<const float4*>(&s_k[buf][c0 + j][(i4 * DG + dg) * 4]);
+                    S[4 * i4 + 0] = fmaf(k4.x, wj, S[4 * i4 + 0]);
+                    S[4 * i4 + 1] = fmaf(k4.y, wj, S[4 * i4 + 1]);
+                    S[4 * i4 + 2] = fmaf(k4.z, wj, S[4 * i4 + 2]);
+                    S[4 * i4 + 3] = fmaf(k4.w, wj, S[4 * i4 + 3]);
+                }
+            }
+            if (col_ok && dg < nt) orow[(size_t)(base + c0 + dg) * ((size_t)a.heads * Dv)] = o0 + o1;
+        }
+        __syncthreads();
+    }
+    if (col_ok) {
+#pragma unroll
+        for (int i = 0; i < NS; ++i) {
+            const int d = ((i >> 2) * DG + dg) * 4 + (i & 3);
+            if (d < D) sbase[(size_t)d * Dv] = S[i];
+        }
+    }
+    rs_move_tail(a, slot, t0, n);
+}
+
+// `coef` (delta with one decay per head; [T][heads][RS_COEF] floats, 16-byte aligned, may be null): chunks of eight tokens.
 AIRUN_EXPORT int airun_recurrent_state(int mode, const float* q, const float* k, const float* v, const float* g,
                                        long long q_stride, long long k_stride, long long v_stride, long long g_stride,
                                        const float* beta, long long beta_stride, const float* a_log, const float* dt_bias,
@@ -395,7 +771,7 @@ AIRUN_EXPORT int airun_recurrent_state(int mode, const float* q, const float* k,
                                        long long slot_stride, int max_slots, const int32_t* cu_tokens, const int32_t* state_slots,
                                        int num_reqs, float* out, int heads, int kv_rep, int D, int Dv, const float* tail_src,
                                        long long tail_src_stride, long long tail_off, int tail_rows, int tail_width,
-                                       int long_chains, int* err, cudaStream_t stream) {
+                                       int long_chains, float* coef, int T, int* err, cudaStream_t stream) {
     if (num_reqs < 0 || heads <= 0 || heads > 65535 || kv_rep <= 0 || heads % kv_rep || D <= 0 || D > 256 || Dv <= 0 || !state ||
         !cu_tokens || !state_slots || !err || !q || !k || !v || !g || !out || slot_stride < (long long)heads * D * Dv)
         return AIRUN_ERR_ARG;
@@ -412,6 +788,20 @@ AIRUN_EXPORT int airun_recurrent_state(int mode, const float* q, const float* k,
     RecurrentArgs a = {q, k, v, g, q_stride, k_stride, v_stride, g_stride, beta, beta_stride, a_log, dt_bias, bonus, state, slot_stride, max_slots,
                        cu_tokens, state_slots, out, heads, kv_rep, D, Dv, tail_src, tail_src_stride, tail_off, tail_rows,
                        tail_width, err};
+    if (coef) {
+        if (mode != RS_DELTA_HEAD || T <= 0 || ((uintptr_t)coef & 15)) return AIRUN_ERR_ARG;
+        const dim3 cgrid(T / RS_CHUNK + num_reqs, ceil_div_i(heads, 4)), mgrid(num_reqs, heads, ceil_div_i(Dv, 16));
+        if (mgrid.z > 65535) return AIRUN_ERR_ARG;
+#define RS_COEFS(SL) airun_launch(delta_chunk_coef_kernel<SL>, cgrid, dim3(128), 0, stream, a, num_reqs, coef)
+#define RS_CHUNKS(NS) airun_launch(delta_chunk_kernel<NS>, mgrid, dim3(128), 0, stream, a, (const float*)coef)
+        if (D <= 32) { RS_COEFS(1); RS_CHUNKS(4); }
+        else if (D <= 64) { RS_COEFS(2); RS_CHUNKS(8); }
+        else if (D <= 128) { RS_COEFS(4); RS_CHUNKS(16); }
+        else { RS_COEFS(8); RS_CHUNKS(32); }
+#undef RS_COEFS
+#undef RS_CHUNKS
+        return airun_launch_status();
+    }
     dim3 grid(num_reqs, heads, tiles);
 #define RS_LAUNCH(NS, DG) \
     do { if (mode == RS_DELTA) airun_launch(recurrent_state_kernel<RS_DELTA, NS, DG>, grid, dim3(128), 0, stream, a); \

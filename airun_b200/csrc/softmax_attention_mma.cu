@@ -696,35 +696,29 @@ __global__ __launch_bounds__(128) void softmax_attention_group_kernel(const XamP
 }
 
 // The slices of every single token merged in slice order (each brought to the common maximum, the sink joining the
-// denominator); a block per request, a head at a time per warp.
-__global__ __launch_bounds__(256) void xam_reduce_kernel(const XamParams p) {
+// denominator).  One block per (request, head): lane s of every warp holds slice s's maximum and sum (at most 32 slices),
+// a thread adds up one column.
+__global__ __launch_bounds__(128) void xam_reduce_kernel(const XamParams p) {
     pdl_trigger();
     pdl_wait();
-    const int r = blockIdx.x;
+    const int r = blockIdx.x, head = blockIdx.y;
     const int tok = p.cu_tokens[r];
     if (p.cu_tokens[r + 1] - tok != 1) return;
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, Dv = p.Dv;
-    const size_t width = (size_t)p.nh * (Dv + 2);
-    for (int head = warp; head < p.nh; head += 8) {
-        const float sink2 = p.sink ? p.sink[head] * XAM_LOG2E : -INFINITY;
-        float top = sink2;
-        for (int s = 0; s < p.splits; ++s) top = fmaxf(top, p.partial[((size_t)s * p.T + tok) * width + (size_t)p.nh * Dv + 2 * head]);
-        float den = p.sink ? xam_exp2(sink2 - top) : 0.0f;
-        for (int s = 0; s < p.splits; ++s) {
-            const float* ml = p.partial + ((size_t)s * p.T + tok) * width + (size_t)p.nh * Dv + 2 * head;
-            den = fmaf(ml[1], ml[0] == -INFINITY ? 0.0f : xam_exp2(ml[0] - top), den);
-        }
-        const float inv = den > 0.0f ? p.out_scale / den : 0.0f;
-        for (int c = lane; c < Dv; c += 32) {
-            float acc = 0.0f;
-            for (int s = 0; s < p.splits; ++s) {
-                const float* base = p.partial + ((size_t)s * p.T + tok) * width;
-                const float m = base[(size_t)p.nh * Dv + 2 * head];
-                acc = fmaf(base[(size_t)head * Dv + c], m == -INFINITY ? 0.0f : xam_exp2(m - top), acc);
-            }
-            p.out[(size_t)tok * p.out_stride + (size_t)head * Dv + c] = __float2bfloat16_rn(acc * inv);
-        }
-    }
+    const int lane = threadIdx.x & 31, c = threadIdx.x, Dv = p.Dv;
+    const size_t width = (size_t)p.nh * (Dv + 2), slice = (size_t)p.T * width;
+    const float* base = p.partial + (size_t)tok * width;
+    const float* ml = base + (size_t)p.nh * Dv + 2 * head;
+    const float m = lane < p.splits ? ml[lane * slice] : -INFINITY, l = lane < p.splits ? ml[lane * slice + 1] : 0.0f;
+    const float sink2 = p.sink ? p.sink[head] * XAM_LOG2E : -INFINITY;
+    const float top = fmaxf(warp_max(m), sink2);
+    const float w = m == -INFINITY ? 0.0f : xam_exp2(m - top);
+    const float den = warp_sum(l * w) + (p.sink ? xam_exp2(sink2 - top) : 0.0f);
+    const float inv = den > 0.0f ? p.out_scale / den : 0.0f;
+    const float* col = base + (size_t)head * Dv + min(c, Dv - 1);
+    float acc = 0.0f;
+#pragma unroll 4
+    for (int s = 0; s < p.splits; ++s) acc = fmaf(col[s * slice], __shfl_sync(0xffffffffu, w, s), acc);
+    if (c < Dv) p.out[(size_t)tok * p.out_stride + (size_t)head * Dv + c] = __float2bfloat16_rn(acc * inv);
 }
 
 template <int DP, int DVP, bool ONE>
@@ -741,7 +735,7 @@ static int xag_launch(const XamParams& p, cudaStream_t stream) {
     airun_launch(softmax_attention_group_kernel<DP, DVP, ONE>, dim3(p.nkv, p.num_reqs, p.splits), dim3(128), smem, stream, p);
     int rc = airun_launch_status();
     if (rc != AIRUN_OK || p.splits <= 1) return rc;
-    airun_launch(xam_reduce_kernel, dim3(p.num_reqs), dim3(256), 0, stream, p);
+    airun_launch(xam_reduce_kernel, dim3(p.num_reqs, p.nh), dim3(128), 0, stream, p);
     return airun_launch_status();
 }
 
@@ -825,7 +819,7 @@ AIRUN_EXPORT int airun_softmax_attention_group(const void* q, void* out, long lo
     XamParams p;
     if (!xam_fill(p, q, out, out_stride, pool, block_table, max_blocks, cu_tokens, context_lens, num_reqs, num_pages, page_size,
                   nh, nkv, D, Dv, scale, table, table_len, sink, window, out_scale, tail, err) ||
-        nh / nkv > 16 || num_reqs > 65535 || splits < 1 || splits > 65535 || (splits > 1 && (!partial || T <= 0)))
+        nh / nkv > 16 || num_reqs > 65535 || splits < 1 || splits > 32 || (splits > 1 && (!partial || T <= 0)))
         return AIRUN_ERR_ARG;
     if (num_reqs == 0) return AIRUN_OK;
     p.splits = splits; p.partial = partial; p.T = T;
