@@ -610,14 +610,41 @@ __global__ __launch_bounds__(128) void delta_chunk_coef_kernel(RecurrentArgs a, 
     }
 }
 
-// One block per (request, head, 16 value columns), 128 threads: a column is shared by eight neighbouring lanes with NS key
-// channels each, and lane l of a column also stands for token l of the chunk.
+// two float32 numbers in a register pair: d = a * b + c and a * b, both halves at once
+typedef unsigned long long rs_pair;
+__device__ __forceinline__ rs_pair rs_fma2(rs_pair a, rs_pair b, rs_pair c) {
+    rs_pair d;
+    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
+    return d;
+}
+__device__ __forceinline__ rs_pair rs_mul2(rs_pair a, rs_pair b) {
+    rs_pair d;
+    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+    return d;
+}
+__device__ __forceinline__ rs_pair rs_pack(float lo, float hi) {
+    rs_pair d;
+    asm("mov.b64 %0, {%1, %2};" : "=l"(d) : "f"(lo), "f"(hi));
+    return d;
+}
+__device__ __forceinline__ float2 rs_unpack(rs_pair v) {
+    float2 d;
+    asm("mov.b64 {%0, %1}, %2;" : "=f"(d.x), "=f"(d.y) : "l"(v));
+    return d;
+}
+
+// One block per (request, head, 16 value columns), 256 threads: a column is shared by sixteen neighbouring lanes with NS key
+// channels each.  After the sums over key channels lane l < 8 of a column holds token l's prediction and stands for its
+// write, lane l >= 8 holds token l - 8's read-out of the old state and stands for its output.  (What bounds a prompt is how
+// long one chunk takes, with few warps an SM: sixteen lanes a column instead of eight are twice the warps for the same work.)
 template <int NS>
-__global__ __launch_bounds__(128, NS <= 16 ? 4 : 1) void delta_chunk_kernel(RecurrentArgs a, const float* __restrict__ coef) {
+__global__ __launch_bounds__(256, NS <= 8 ? 2 : 1) void delta_chunk_kernel(RecurrentArgs a, const float* __restrict__ coef) {
     pdl_trigger();
     pdl_wait();
-    constexpr int DG = 8, DP = NS * DG, COLS = 16, TT = NS >= 32 ? 8 : 16;
+    constexpr int DG = 16, DP = NS * DG, COLS = 16, TT = NS >= 16 ? 8 : 16, NT = 256;
+    constexpr bool KEEP_K = NS <= 8;              // the keys of a chunk stay in registers from the dot products to the update
     __shared__ __align__(16) float s_q[2][TT][DP], s_k[2][TT][DP], s_v[2][TT][COLS], s_c[2][TT][RS_COEF];
+    __shared__ __align__(16) float s_x[NT / 32][32 / DG][3][RS_CHUNK];        // per warp and column: what its lanes tell one another
     const int r = blockIdx.x, head = blockIdx.y, col0 = blockIdx.z * COLS;
     const int t0 = a.cu_tokens[r], n = a.cu_tokens[r + 1] - t0;
     if (n <= 0) return;
@@ -628,136 +655,140 @@ __global__ __launch_bounds__(128, NS <= 16 ? 4 : 1) void delta_chunk_kernel(Recu
     }
     const int D = a.D, Dv = a.Dv;
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-    const int dg = lane & (DG - 1), cl = warp * (32 / DG) + lane / DG, col = col0 + cl;
+    const int dg = lane & (DG - 1), tok = dg & (RS_CHUNK - 1), cl = warp * (32 / DG) + lane / DG, col = col0 + cl;
     const bool col_ok = col < Dv;
     const int ncol = min(COLS, Dv - col0);
     // both stages start as zeros: padding and rows beyond the last token hold numbers whose weight is zero
-    for (int e = threadIdx.x; e < 2 * TT * DP; e += 128) { (&s_q[0][0][0])[e] = 0.0f; (&s_k[0][0][0])[e] = 0.0f; }
-    for (int e = threadIdx.x; e < 2 * TT * COLS; e += 128) (&s_v[0][0][0])[e] = 0.0f;
+    for (int e = threadIdx.x; e < 2 * TT * DP; e += NT) { (&s_q[0][0][0])[e] = 0.0f; (&s_k[0][0][0])[e] = 0.0f; }
+    for (int e = threadIdx.x; e < 2 * TT * COLS; e += NT) (&s_v[0][0][0])[e] = 0.0f;
     __syncthreads();
-    const float* qh = a.q + (size_t)(head / a.kv_rep) * D;
-    const float* kh = a.k + (size_t)(head / a.kv_rep) * D;
-    const float* vh = a.v + (size_t)head * Dv + col0;
+    const float* qh = a.q + (size_t)(head / a.kv_rep) * D + (size_t)t0 * a.q_stride;
+    const float* kh = a.k + (size_t)(head / a.kv_rep) * D + (size_t)t0 * a.k_stride;
+    const float* vh = a.v + (size_t)head * Dv + col0 + (size_t)t0 * a.v_stride;
+    const float* ch = coef + ((size_t)t0 * a.heads + head) * RS_COEF;
+    // A thread copies the same piece of a row, of every step-th row: 16 bytes, or one number where the rows allow no more.
     const bool vec = (D % 4 == 0) && ((a.q_stride | a.k_stride) % 4 == 0) && ((((uintptr_t)qh | (uintptr_t)kh) & 15) == 0);
     const bool vvec = (ncol % 4 == 0) && (a.v_stride % 4 == 0) && (((uintptr_t)vh & 15) == 0);
+    const int dper = vec ? D / 4 : min(D, NT), drows = NT / dper, drow = threadIdx.x / dper, dcol = (threadIdx.x - drow * dper) * (vec ? 4 : 1);
+    const int vper = vvec ? ncol / 4 : ncol, vrows = NT / vper, vrow = threadIdx.x / vper, vcol = (threadIdx.x - vrow * vper) * (vvec ? 4 : 1);
+    constexpr int CPER = RS_COEF / 4, CROWS = NT / CPER;
+    const int crow = threadIdx.x / CPER, ccol = (threadIdx.x - crow * CPER) * 4;
     auto stage = [&](int base, int buf) {
         const int nt = min(TT, n - base);
-        if (vec) {
-            const int per = D / 4;
-            for (int e = threadIdx.x; e < nt * per; e += 128) {
-                const int tt = e / per, d = (e - tt * per) * 4;
-                const size_t row = (size_t)(t0 + base + tt);
-                rs_cp16(&s_q[buf][tt][d], qh + row * a.q_stride + d);
-                rs_cp16(&s_k[buf][tt][d], kh + row * a.k_stride + d);
+        if (drow < drows)
+            for (int tt = drow; tt < nt; tt += drows) {
+                const float* qr = qh + (size_t)(base + tt) * a.q_stride;
+                const float* kr = kh + (size_t)(base + tt) * a.k_stride;
+                if (vec) {
+                    rs_cp16(&s_q[buf][tt][dcol], qr + dcol);
+                    rs_cp16(&s_k[buf][tt][dcol], kr + dcol);
+                } else {
+                    for (int d = dcol; d < D; d += dper) { rs_cp4(&s_q[buf][tt][d], qr + d); rs_cp4(&s_k[buf][tt][d], kr + d); }
+                }
             }
-        } else {
-            for (int e = threadIdx.x; e < nt * D; e += 128) {
-                const int tt = e / D, d = e - tt * D;
-                const size_t row = (size_t)(t0 + base + tt);
-                rs_cp4(&s_q[buf][tt][d], qh + row * a.q_stride + d);
-                rs_cp4(&s_k[buf][tt][d], kh + row * a.k_stride + d);
+        if (vrow < vrows)
+            for (int tt = vrow; tt < nt; tt += vrows) {
+                if (vvec) rs_cp16(&s_v[buf][tt][vcol], vh + (size_t)(base + tt) * a.v_stride + vcol);
+                else rs_cp4(&s_v[buf][tt][vcol], vh + (size_t)(base + tt) * a.v_stride + vcol);
             }
-        }
-        if (vvec) {
-            const int per = ncol / 4;
-            for (int e = threadIdx.x; e < nt * per; e += 128) {
-                const int tt = e / per, c = (e - tt * per) * 4;
-                rs_cp16(&s_v[buf][tt][c], vh + (size_t)(t0 + base + tt) * a.v_stride + c);
+        if (crow < CROWS)
+            for (int tt = crow; tt < TT; tt += CROWS) {
+                if (tt < nt) rs_cp16(&s_c[buf][tt][ccol], ch + (size_t)(base + tt) * a.heads * RS_COEF + ccol);
+                else *reinterpret_cast<float4*>(&s_c[buf][tt][ccol]) = make_float4(0.f, 0.f, 0.f, 0.f);
             }
-        } else {
-            for (int e = threadIdx.x; e < nt * ncol; e += 128) {
-                const int tt = e / ncol, c = e - tt * ncol;
-                rs_cp4(&s_v[buf][tt][c], vh + (size_t)(t0 + base + tt) * a.v_stride + c);
-            }
-        }
-        for (int e = threadIdx.x; e < TT * (RS_COEF / 4); e += 128) {
-            const int tt = e / (RS_COEF / 4), c = (e - tt * (RS_COEF / 4)) * 4;
-            if (tt < nt) rs_cp16(&s_c[buf][tt][c], coef + ((size_t)(t0 + base + tt) * a.heads + head) * RS_COEF + c);
-            else *reinterpret_cast<float4*>(&s_c[buf][tt][c]) = make_float4(0.f, 0.f, 0.f, 0.f);
-        }
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
     stage(0, 0);
     float* sbase = a.state + (size_t)slot * a.slot_stride + (size_t)head * D * Dv + (col_ok ? col : 0);
-    float S[NS];                                  // channel of register i: group of four (i / 4) * DG + dg, element i % 4
+    rs_pair S[NS / 2];                            // channel of number i: group of four (i / 4) * DG + dg, element i % 4
 #pragma unroll
-    for (int i = 0; i < NS; ++i) {
-        const int d = ((i >> 2) * DG + dg) * 4 + (i & 3);
-        S[i] = (col_ok && d < D) ? sbase[(size_t)d * Dv] : 0.0f;
+    for (int i = 0; i < NS / 2; ++i) {
+        float v[2];
+#pragma unroll
+        for (int h = 0; h < 2; ++h) {
+            const int d = (((2 * i + h) >> 2) * DG + dg) * 4 + ((2 * i + h) & 3);
+            v[h] = (col_ok && d < D) ? sbase[(size_t)d * Dv] : 0.0f;
+        }
+        S[i] = rs_pack(v[0], v[1]);
     }
     float* orow = a.out + (size_t)t0 * ((size_t)a.heads * Dv) + (size_t)head * Dv + col;
+    float (*sx)[RS_CHUNK] = s_x[warp][lane / DG];
     int it = 0;
     for (int base = 0; base < n; base += TT, ++it) {
         const int buf = it & 1;
-        if (base + TT < n) {
-            stage(base + TT, buf ^ 1);            // that stage was last read before the barrier that ended the iteration before
-            asm volatile("cp.async.wait_group 1;" ::: "memory");
-        } else {
-            asm volatile("cp.async.wait_group 0;" ::: "memory");
-        }
-        __syncthreads();
+        asm volatile("cp.async.wait_group 0;" ::: "memory");
+        __syncthreads();                                      // this stage is there, and nobody reads the other one any more
+        if (base + TT < n) stage(base + TT, buf ^ 1);
 #pragma unroll 1
         for (int c0 = 0; c0 < TT && base + c0 < n; c0 += RS_CHUNK) {
             const int nt = min(RS_CHUNK, n - base - c0);
-            float p[RS_CHUNK], oq[RS_CHUNK];
+            rs_pair p2[RS_CHUNK], o2[RS_CHUNK];
+            ulonglong2 kr[KEEP_K ? RS_CHUNK : 1][KEEP_K ? NS / 4 : 1];
 #pragma unroll
-            for (int i = 0; i < RS_CHUNK; ++i) { p[i] = 0.0f; oq[i] = 0.0f; }
+            for (int i = 0; i < RS_CHUNK; ++i) { p2[i] = 0ull; o2[i] = 0ull; }
 #pragma unroll
             for (int i4 = 0; i4 < NS / 4; ++i4) {
 #pragma unroll
                 for (int i = 0; i < RS_CHUNK; ++i) {
-                    const float4 k4 = *reinterpret_cast<const float4*>(&s_k[buf][c0 + i][(i4 * DG + dg) * 4]);
-                    const float4 q4 = *reinterpret_cast<const float4*>(&s_q[buf][c0 + i][(i4 * DG + dg) * 4]);
-                    p[i] = fmaf(S[4 * i4 + 0], k4.x, p[i]); oq[i] = fmaf(S[4 * i4 + 0], q4.x, oq[i]);
-                    p[i] = fmaf(S[4 * i4 + 1], k4.y, p[i]); oq[i] = fmaf(S[4 * i4 + 1], q4.y, oq[i]);
-                    p[i] = fmaf(S[4 * i4 + 2], k4.z, p[i]); oq[i] = fmaf(S[4 * i4 + 2], q4.z, oq[i]);
-                    p[i] = fmaf(S[4 * i4 + 3], k4.w, p[i]); oq[i] = fmaf(S[4 * i4 + 3], q4.w, oq[i]);
+                    const ulonglong2 k4 = *reinterpret_cast<const ulonglong2*>(&s_k[buf][c0 + i][(i4 * DG + dg) * 4]);
+                    const ulonglong2 q4 = *reinterpret_cast<const ulonglong2*>(&s_q[buf][c0 + i][(i4 * DG + dg) * 4]);
+                    if (KEEP_K) kr[KEEP_K ? i : 0][KEEP_K ? i4 : 0] = k4;
+                    p2[i] = rs_fma2(S[2 * i4], k4.x, p2[i]); o2[i] = rs_fma2(S[2 * i4], q4.x, o2[i]);
+                    p2[i] = rs_fma2(S[2 * i4 + 1], k4.y, p2[i]); o2[i] = rs_fma2(S[2 * i4 + 1], q4.y, o2[i]);
                 }
             }
-            rs_scatter_sum<RS_CHUNK>(p, lane);
-            rs_scatter_sum<RS_CHUNK>(oq, lane);
-            // this lane's token from here on: c0 + dg
-            const float* cf = &s_c[buf][c0 + dg][0];
-            const float4 ta = *reinterpret_cast<const float4*>(cf), tb = *reinterpret_cast<const float4*>(cf + 4);
-            const float4 qa = *reinterpret_cast<const float4*>(cf + 8), qb = *reinterpret_cast<const float4*>(cf + 12);
-            const float2 dec = *reinterpret_cast<const float2*>(cf + 16);         // decay up to the token; from after it to the chunk's end
-            const float rest = fmaf(-dec.x, p[0], s_v[buf][c0 + dg][cl]);
-            const float tm[RS_CHUNK] = {ta.x, ta.y, ta.z, ta.w, tb.x, tb.y, tb.z, tb.w};
-            const float qk[RS_CHUNK] = {qa.x, qa.y, qa.z, qa.w, qb.x, qb.y, qb.z, qb.w};
-            float u0 = 0.0f, u1 = 0.0f;
+            float sum[2 * RS_CHUNK];
 #pragma unroll
-            for (int j = 0; j < RS_CHUNK; j += 2) {
-                u0 = fmaf(tm[j], __shfl_sync(0xffffffffu, rest, j, DG), u0);
-                u1 = fmaf(tm[j + 1], __shfl_sync(0xffffffffu, rest, j + 1, DG), u1);
+            for (int i = 0; i < RS_CHUNK; ++i) {
+                const float2 pv = rs_unpack(p2[i]), ov = rs_unpack(o2[i]);
+                sum[i] = pv.x + pv.y; sum[RS_CHUNK + i] = ov.x + ov.y;
             }
-            const float u = u0 + u1, ul = u * dec.y;
-            const float whole = __shfl_sync(0xffffffffu, dec.x, nt - 1, DG);
+            rs_scatter_sum<2 * RS_CHUNK>(sum, lane);
+            // this lane's token from here on: c0 + tok; its row of the inverse (its write) or of the products (its output)
+            const float* cf = &s_c[buf][c0 + tok][0];
+            const float2 dec = *reinterpret_cast<const float2*>(cf + 16);         // decay up to the token; from after it to the chunk's end
+            const ulonglong2 ra = *reinterpret_cast<const ulonglong2*>(cf + (dg & RS_CHUNK)), rb = *reinterpret_cast<const ulonglong2*>(cf + (dg & RS_CHUNK) + 4);
+            if (dg < RS_CHUNK) sx[0][tok] = fmaf(-dec.x, sum[0], s_v[buf][c0 + tok][cl]);
+            __syncwarp();
+            auto row_times = [&](const float* v) {
+                const ulonglong2 va = *reinterpret_cast<const ulonglong2*>(v), vb = *reinterpret_cast<const ulonglong2*>(v + 4);
+                const float2 t = rs_unpack(rs_fma2(rb.y, vb.y, rs_fma2(rb.x, vb.x, rs_fma2(ra.y, va.y, rs_mul2(ra.x, va.x)))));
+                return t.x + t.y;
+            };
+            const float u = row_times(sx[0]);
+            if (dg < RS_CHUNK) { sx[1][tok] = u; sx[2][tok] = u * dec.y; }
+            const float whole = s_c[buf][c0 + nt - 1][16];
+            const rs_pair w2 = rs_pack(whole, whole);
 #pragma unroll
-            for (int i = 0; i < NS; ++i) S[i] *= whole;
-            float o0 = dec.x * oq[0], o1 = 0.0f;
+            for (int i = 0; i < NS / 2; ++i) S[i] = rs_mul2(S[i], w2);
+            __syncwarp();
+            const float4 wa = *reinterpret_cast<const float4*>(&sx[2][0]), wb = *reinterpret_cast<const float4*>(&sx[2][4]);
+            const float w[RS_CHUNK] = {wa.x, wa.y, wa.z, wa.w, wb.x, wb.y, wb.z, wb.w};
 #pragma unroll
             for (int j = 0; j < RS_CHUNK; ++j) {
-                const float uj = __shfl_sync(0xffffffffu, u, j, DG), wj = __shfl_sync(0xffffffffu, ul, j, DG);
-                if (j & 1) o1 = fmaf(qk[j], uj, o1);
-                else o0 = fmaf(qk[j], uj, o0);
+                const rs_pair wj = rs_pack(w[j], w[j]);
 #pragma unroll
                 for (int i4 = 0; i4 < NS / 4; ++i4) {
-                    const float4 k4 = *reinterpret_cast<const float4*>(&s_k[buf][c0 + j][(i4 * DG + dg) * 4]);
-                    S[4 * i4 + 0] = fmaf(k4.x, wj, S[4 * i4 + 0]);
-                    S[4 * i4 + 1] = fmaf(k4.y, wj, S[4 * i4 + 1]);
-                    S[4 * i4 + 2] = fmaf(k4.z, wj, S[4 * i4 + 2]);
-                    S[4 * i4 + 3] = fmaf(k4.w, wj, S[4 * i4 + 3]);
+                    const ulonglong2 k4 = KEEP_K ? kr[KEEP_K ? j : 0][KEEP_K ? i4 : 0]
+                                                 : *reinterpret_cast<const ulonglong2*>(&s_k[buf][c0 + j][(i4 * DG + dg) * 4]);
+                    S[2 * i4] = rs_fma2(k4.x, wj, S[2 * i4]);
+                    S[2 * i4 + 1] = rs_fma2(k4.y, wj, S[2 * i4 + 1]);
                 }
             }
-            if (col_ok && dg < nt) orow[(size_t)(base + c0 + dg) * ((size_t)a.heads * Dv)] = o0 + o1;
+            const float o = fmaf(dec.x, sum[0], row_times(sx[1]));
+            if (col_ok && dg >= RS_CHUNK && tok < nt) orow[(size_t)(base + c0 + tok) * ((size_t)a.heads * Dv)] = o;
+            __syncwarp();                                     // the lanes' numbers are read before the next chunk's are written
         }
-        __syncthreads();
     }
     if (col_ok) {
 #pragma unroll
-        for (int i = 0; i < NS; ++i) {
-            const int d = ((i >> 2) * DG + dg) * 4 + (i & 3);
-            if (d < D) sbase[(size_t)d * Dv] = S[i];
+        for (int i = 0; i < NS / 2; ++i) {
+            const float2 v = rs_unpack(S[i]);
+#pragma unroll
+            for (int h = 0; h < 2; ++h) {
+                const int d = (((2 * i + h) >> 2) * DG + dg) * 4 + ((2 * i + h) & 3);
+                if (d < D) sbase[(size_t)d * Dv] = h ? v.y : v.x;
+            }
         }
     }
     rs_move_tail(a, slot, t0, n);
@@ -793,11 +824,14 @@ AIRUN_EXPORT int airun_recurrent_state(int mode, const float* q, const float* k,
         const dim3 cgrid(T / RS_CHUNK + num_reqs, ceil_div_i(heads, 4)), mgrid(num_reqs, heads, ceil_div_i(Dv, 16));
         if (mgrid.z > 65535) return AIRUN_ERR_ARG;
 #define RS_COEFS(SL) airun_launch(delta_chunk_coef_kernel<SL>, cgrid, dim3(128), 0, stream, a, num_reqs, coef)
-#define RS_CHUNKS(NS) airun_launch(delta_chunk_kernel<NS>, mgrid, dim3(128), 0, stream, a, (const float*)coef)
-        if (D <= 32) { RS_COEFS(1); RS_CHUNKS(4); }
-        else if (D <= 64) { RS_COEFS(2); RS_CHUNKS(8); }
-        else if (D <= 128) { RS_COEFS(4); RS_CHUNKS(16); }
-        else { RS_COEFS(8); RS_CHUNKS(32); }
+#define RS_CHUNKS(NS) airun_launch(delta_chunk_kernel<NS>, mgrid, dim3(256), 0, stream, a, (const float*)coef)
+        if (D <= 32) RS_COEFS(1);
+        else if (D <= 64) RS_COEFS(2);
+        else if (D <= 128) RS_COEFS(4);
+        else RS_COEFS(8);
+        if (D <= 64) RS_CHUNKS(4);
+        else if (D <= 128) RS_CHUNKS(8);
+        else RS_CHUNKS(16);
 #undef RS_COEFS
 #undef RS_CHUNKS
         return airun_launch_status();
