@@ -581,6 +581,60 @@ def check_decay_attention(dev) -> Tuple[float, float]:
     return max(_rel(o, want), _rel(act, gated)), 2e-5
 
 
+def check_sandwich_norm(dev) -> Tuple[float, float]:
+    """v = x + y / rms(y) * a, then v / rms(v) * b, in one pass; and v as two bfloat16 halves."""
+    from .kernels import ops
+    worst = 0.0
+    for T, n in ((5, 100), (90, 1024)):
+        x, y, a, b = torch.randn(T, n), torch.randn(T, n), 1 + 0.3 * torch.randn(n), 1 + 0.3 * torch.randn(n)
+        rms = lambda t: t / torch.sqrt((t * t).mean(-1, keepdim=True) + 1e-5)
+        v = x.double() + rms(y.double()) * a.double()
+        xd, out = x.to(dev), torch.empty(T, n, device=dev)
+        ops.sandwich_norm(xd, out, y=y.to(dev), w_post=a.to(dev), eps_post=1e-5, w_pre=b.to(dev), eps_pre=1e-5)
+        two = torch.empty(T, 2 * n, device=dev, dtype=torch.bfloat16)
+        ops.sandwich_norm(xd, two, mode=ops.SANDWICH_SPLIT, write_back=False)
+        worst = max(worst, _rel(xd, v), _rel(out, rms(v) * b.double()), _rel(two[:, :n].float() + two[:, n:].float(), v))
+    return worst, 2e-5
+
+
+def check_delta_rule(dev) -> Tuple[float, float]:
+    """The delta rule with one decay per head: a request of 40 tokens beside one of 3 (chunks of eight tokens), then one
+    more token each (token by token)."""
+    from types import SimpleNamespace
+    from .engine.batch import Workspace
+    from .kernels import ops
+    heads, D, Dv, lens = 3, 24, 20, [41, 4]
+    kd, vd, T = heads * D, heads * Dv, sum(lens)
+    unit = lambda t: t / t.norm(dim=-1, keepdim=True)
+    q, k = (unit(torch.randn(T, heads, D)).reshape(T, kd) for _ in range(2))
+    v, beta, a = torch.randn(T, vd), torch.randn(T, heads), torch.randn(T, heads) - 2.0
+    a_log, dt = 0.5 * torch.randn(heads), torch.randn(heads)
+    state, err = torch.zeros(2, heads * D * Dv, device=dev), torch.zeros(1, dtype=torch.int32, device=dev)
+    got, at = torch.zeros(T, vd), [0, lens[0]]
+    for part in ([slice(b, b + n - 1) for b, n in zip(at, lens)], [slice(b + n - 1, b + n) for b, n in zip(at, lens)]):
+        cat = lambda t: torch.cat([t[s] for s in part]).to(dev)
+        sizes = [s.stop - s.start for s in part]
+        cu = torch.tensor([0, sizes[0], sum(sizes)], dtype=torch.int32, device=dev)
+        ctx = SimpleNamespace(cu_tokens=cu, state_slots=torch.tensor([1, 0], dtype=torch.int32, device=dev), num_reqs=2, err=err,
+                              ws=Workspace(dev, 1 << 20))
+        o = torch.empty(sum(sizes), vd, device=dev)
+        ops.recurrent_state(ops.RECURRENCE_DELTA_HEAD, cat(q), cat(k), cat(v), cat(a), state, ctx, o, heads, 1, D, Dv, beta=cat(beta),
+                            a_log=a_log.to(dev), dt_bias=dt.to(dev))
+        for s, rows in zip(part, o.cpu().split(sizes)):
+            got[s] = rows
+    g = torch.exp(-torch.exp(a_log.double()) * torch.nn.functional.softplus(a.double() + dt.double()))
+    want = torch.zeros(T, vd, dtype=torch.float64)
+    for b, n in zip(at, lens):
+        S = torch.zeros(heads, D, Dv, dtype=torch.float64)
+        for t in range(b, b + n):
+            kt, qt = k[t].double().view(heads, D), q[t].double().view(heads, D)
+            S = g[t][:, None, None] * S
+            u = torch.sigmoid(beta[t].double())[:, None] * (v[t].double().view(heads, Dv) - torch.einsum("hdv,hd->hv", S, kt))
+            S = S + kt[:, :, None] * u[:, None, :]
+            want[t] = torch.einsum("hdv,hd->hv", S, qt).reshape(vd)
+    return _rel(got, want), 2e-5
+
+
 CHECKS: List[Tuple[str, Callable]] = [
     ("embedding gather", check_embedding),
     ("rmsnorm + residual add", check_rmsnorm),
@@ -601,6 +655,8 @@ CHECKS: List[Tuple[str, Callable]] = [
     ("product, tcgen05 with an activation in the epilogue", check_gemm_tc_activation),
     ("residual of several streams: write, read and norm", check_streams),
     ("decayed linear attention: recurrence, norm over all heads and gate", check_decay_attention),
+    ("norms on both sides of a sub-layer in one pass", check_sandwich_norm),
+    ("delta rule with a decay per head: chunks and single tokens", check_delta_rule),
     ("sampling", check_sampling),
     ("largest logits of a row", check_largest_logits),
 ]
