@@ -1066,7 +1066,7 @@ def losalorn_config(size: dict):
     mlp = dict(kind="dense", ff=F, limit=7.0)
     delta = dict(type="delta", mixer=dict(heads=H, kv_heads=H // 2, dim=64, vdim=128, conv=4), mlp=mlp)
     att = dict(type="attention", mixer=dict(heads=H, kv_heads=G, dim=128, vdim=128, scale=128 ** -0.5, mask=dict(size=1024),
-                                            rot=dict(dims=64, base=50000.0, scaling=dict(factor=4.0, low=1.0, high=4.0, original=8192))), mlp=mlp)
+                                            rot=dict(dims=64, base=500000.0, scaling=dict(factor=8.0, low=1.0, high=4.0, original=8192))), mlp=mlp)
     return LosalornConfig.from_dict(dict(architecture="Losalorn", vocab=VEDIZEN_VOCAB, width=W, norm=dict(eps=1e-5), embedding=dict(scale=W ** 0.5),
                                          logit_softcap=30.0, loop=dict(start=1, stop=3, times=2), layers=[delta, att, delta, att]))
 
