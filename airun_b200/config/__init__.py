@@ -7,6 +7,7 @@ from .pogarax import PogaraxConfig
 from .gamanex import GamanexConfig
 from .tagulix import TagulixConfig
 from .losalorn import LosalornConfig
+from .pirerax import PireraxConfig
 
 
 def _register_builtin() -> None:
@@ -17,6 +18,7 @@ def _register_builtin() -> None:
     register_architecture("Gamanex", GamanexConfig, build_decoder)
     register_architecture("Tagulix", TagulixConfig, build_decoder)
     register_architecture("Losalorn", LosalornConfig, build_decoder)
+    register_architecture("Pirerax", PireraxConfig, build_decoder)
 
 
 _register_builtin()

@@ -644,8 +644,10 @@ __device__ __forceinline__ void sandwich_put(TOut* __restrict__ out, int i, int 
     }
 }
 
-template <typename TOut, int VEC>
+// PAIR: two results join at once, x + mult * (y / rms(y) * w_post + y2 / rms(y2) * w_post2); without it mult is not read.
+template <typename TOut, int VEC, bool PAIR>
 __global__ __launch_bounds__(512) void sandwich_norm_kernel(float* __restrict__ x, const float* __restrict__ y, const float* __restrict__ w_post,
+                                     const float* __restrict__ y2, const float* __restrict__ w_post2, float mult,
                                      const float* __restrict__ w_pre, TOut* __restrict__ out, const int32_t* __restrict__ rows,
                                      int n, float eps_post, float eps_pre, int write_back, int mode) {
     pdl_trigger();
@@ -668,10 +670,16 @@ __global__ __launch_bounds__(512) void sandwich_norm_kernel(float* __restrict__ 
         load(y ? w_post : nullptr, wa[k], threadIdx.x + k * blockDim.x, 0.0f);
         load(mode == SANDWICH_NORM ? w_pre : nullptr, wb[k], threadIdx.x + k * blockDim.x, 1.0f);
     }
+    float y2k[PAIR ? KEEP : 1][VEC], wa2[PAIR ? KEEP : 1][VEC];
+    if (PAIR) {
+#pragma unroll
+        for (int k = 0; k < KEEP; ++k) load(w_post2, wa2[PAIR ? k : 0], threadIdx.x + k * blockDim.x, 0.0f);
+    }
     pdl_wait();
     const int r = blockIdx.x, src = rows ? rows[r] : r;
     float* xr = x + (size_t)src * n;
     const float* yr = y ? y + (size_t)src * n : nullptr;
+    const float* y2r = PAIR ? y2 + (size_t)src * n : nullptr;
     TOut* outr = out ? out + (size_t)r * (mode == SANDWICH_SPLIT ? 2 * n : n) : nullptr;
     const int tail0 = (threadIdx.x + KEEP * blockDim.x) * VEC, tstep = blockDim.x * VEC;       // a row longer than the registers hold
     float ss = 0.0f;
@@ -679,8 +687,9 @@ __global__ __launch_bounds__(512) void sandwich_norm_kernel(float* __restrict__ 
     for (int k = 0; k < KEEP; ++k) {
         load(xr, v[k], threadIdx.x + k * blockDim.x, 0.0f);
         load(yr, yk[k], threadIdx.x + k * blockDim.x, 0.0f);
+        if (PAIR) load(y2r, y2k[PAIR ? k : 0], threadIdx.x + k * blockDim.x, 0.0f);
     }
-    float inv_y = 0.0f;
+    float inv_y = 0.0f, inv_y2 = 0.0f;
     if (yr) {
 #pragma unroll
         for (int k = 0; k < KEEP; ++k)
@@ -690,6 +699,18 @@ __global__ __launch_bounds__(512) void sandwich_norm_kernel(float* __restrict__ 
 #pragma unroll
             for (int e = 0; e < VEC; ++e) ss = fmaf(yr[i + e], yr[i + e], ss);
         inv_y = 1.0f / sqrtf(block_sum(ss, red) / (float)n + eps_post);
+        if (PAIR) {
+            float s2 = 0.0f;
+#pragma unroll
+            for (int k = 0; k < KEEP; ++k)
+#pragma unroll
+                for (int e = 0; e < VEC; ++e) s2 = fmaf(y2k[PAIR ? k : 0][e], y2k[PAIR ? k : 0][e], s2);
+            for (int i = tail0; i < n; i += tstep)
+#pragma unroll
+                for (int e = 0; e < VEC; ++e) s2 = fmaf(y2r[i + e], y2r[i + e], s2);
+            inv_y2 = mult / sqrtf(block_sum(s2, red) / (float)n + eps_post);
+            inv_y *= mult;
+        }
     }
     ss = 0.0f;
 #pragma unroll
@@ -698,6 +719,7 @@ __global__ __launch_bounds__(512) void sandwich_norm_kernel(float* __restrict__ 
 #pragma unroll
         for (int e = 0; e < VEC; ++e) {
             v[k][e] += yk[k][e] * inv_y * wa[k][e];
+            if (PAIR) v[k][e] += y2k[PAIR ? k : 0][e] * inv_y2 * wa2[PAIR ? k : 0][e];
             ss = fmaf(v[k][e], v[k][e], ss);
         }
         if (yr && write_back && i < nv) {
@@ -708,7 +730,8 @@ __global__ __launch_bounds__(512) void sandwich_norm_kernel(float* __restrict__ 
     for (int i = tail0; i < n; i += tstep)
 #pragma unroll
         for (int e = 0; e < VEC; ++e) {
-            const float u = xr[i + e] + (yr ? yr[i + e] * inv_y * w_post[i + e] : 0.0f);
+            float u = xr[i + e] + (yr ? yr[i + e] * inv_y * w_post[i + e] : 0.0f);
+            if (PAIR) u += y2r[i + e] * inv_y2 * w_post2[i + e];
             if (yr && write_back) xr[i + e] = u;
             ss = fmaf(u, u, ss);
         }
@@ -733,31 +756,34 @@ __global__ __launch_bounds__(512) void sandwich_norm_kernel(float* __restrict__ 
     for (int i = tail0; i < n; i += tstep)
 #pragma unroll
         for (int e = 0; e < VEC; ++e) {
-            const float u = xr[i + e] + (yr && !write_back ? yr[i + e] * inv_y * w_post[i + e] : 0.0f);
+            float u = xr[i + e] + (yr && !write_back ? yr[i + e] * inv_y * w_post[i + e] : 0.0f);
+            if (PAIR && !write_back) u += y2r[i + e] * inv_y2 * w_post2[i + e];
             sandwich_put<TOut>(outr, i + e, n, mode, u, inv, mode == SANDWICH_NORM ? w_pre[i + e] : 1.0f);
         }
 }
 
-AIRUN_EXPORT int airun_sandwich_norm(float* x, const float* y, const float* w_post, const float* w_pre, void* out, int out_dtype,
-                                     const int32_t* rows, int n_rows, int n, float eps_post, float eps_pre, int write_back,
+AIRUN_EXPORT int airun_sandwich_norm(float* x, const float* y, const float* w_post, const float* y2, const float* w_post2, float mult,
+                                     const float* w_pre, void* out, int out_dtype, const int32_t* rows, int n_rows, int n, float eps_post, float eps_pre, int write_back,
                                      int mode, cudaStream_t stream) {
-    if (n_rows < 0 || n <= 0 || !x || (y && !w_post) || (!y && !out) || mode < 0 || mode > 2 || (mode == SANDWICH_NORM && out && !w_pre) ||
+    if (n_rows < 0 || n <= 0 || !x || (y && !w_post) || (y2 && (!y || !w_post2)) || (!y && !out) || mode < 0 || mode > 2 || (mode == SANDWICH_NORM && out && !w_pre) ||
         (rows && write_back) || (mode == SANDWICH_SPLIT && out_dtype != AIRUN_DT_BF16) || (mode == SANDWICH_COPY && out_dtype != AIRUN_DT_F32))
         return AIRUN_ERR_ARG;
     if (n_rows == 0) return AIRUN_OK;
-    const bool vec = n % 4 == 0 && (((uintptr_t)x | (uintptr_t)y | (uintptr_t)w_post | (uintptr_t)w_pre | (uintptr_t)out) & 15) == 0;
+    const bool vec = n % 4 == 0 && (((uintptr_t)x | (uintptr_t)y | (uintptr_t)w_post | (uintptr_t)y2 | (uintptr_t)w_post2 | (uintptr_t)w_pre | (uintptr_t)out) & 15) == 0;
     const int nv = vec ? n / 4 : n;
     // many rows: as few threads as hold the row in registers; few rows: more of them, with fewer loads each
     int threads = ((n_rows > 64 ? (nv + KEEP - 1) / KEEP : (nv + 1) / 2) + 31) / 32 * 32;
     if (threads > 512) threads = 512;
     if (threads < 32) threads = 32;
-#define SW_LAUNCH(TOut, VEC) \
-    airun_launch(sandwich_norm_kernel<TOut, VEC>, dim3(n_rows), dim3(threads), 0, stream, x, y, w_post, w_pre, (TOut*)out, rows, n, \
-                 eps_post, eps_pre, write_back, mode)
+#define SW_PAIR(TOut, VEC, PAIR) \
+    airun_launch(sandwich_norm_kernel<TOut, VEC, PAIR>, dim3(n_rows), dim3(threads), 0, stream, x, y, w_post, y2, w_post2, mult, w_pre, \
+                 (TOut*)out, rows, n, eps_post, eps_pre, write_back, mode)
+#define SW_LAUNCH(TOut, VEC) do { if (y2) SW_PAIR(TOut, VEC, true); else SW_PAIR(TOut, VEC, false); } while (0)
     if (out_dtype == AIRUN_DT_F32) { if (vec) SW_LAUNCH(float, 4); else SW_LAUNCH(float, 1); }
     else if (out_dtype == AIRUN_DT_BF16) { if (vec) SW_LAUNCH(__nv_bfloat16, 4); else SW_LAUNCH(__nv_bfloat16, 1); }
     else return AIRUN_ERR_UNSUPPORTED;
 #undef SW_LAUNCH
+#undef SW_PAIR
     return airun_launch_status();
 }
 

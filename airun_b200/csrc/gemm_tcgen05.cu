@@ -1096,7 +1096,8 @@ static int gemm_launch(const void* x, const void* W, void* out, int M, int N, in
 // rows of out.  epi 0: float32 [M][N]; 1: bfloat16 [M][N]; 2: SwiGLU over interleaved gate/up rows, bfloat16 [M][N/2].
 // ``seg`` (int32 [n_seg + 1]) lives on the device; rows from seg[n_seg] on are left as they are.
 static int gemm_grouped(const void* x, const void* W, void* out, int M, int N, int K, long long ldx, long long ldc, int epi,
-                        const int32_t* seg, int n_seg, int* err, cudaStream_t stream, int act);
+                        const int32_t* seg, int n_seg, int* err, cudaStream_t stream, int act, float glu_limit = 0.0f,
+                        float glu_slope = 0.0f);
 
 AIRUN_EXPORT int airun_gemm_tcgen05_grouped(const void* x, const void* W, void* out, int M, int N, int K, long long ldx,
                                             long long ldc, int epi, const int32_t* seg, int n_seg, int* err,
@@ -1112,8 +1113,16 @@ AIRUN_EXPORT int airun_gemm_tcgen05_grouped_act(const void* x, const void* W, vo
     return gemm_grouped(x, W, out, M, N, K, ldx, ldc, epi, seg, n_seg, err, stream, 1 + mode);
 }
 
+// The grouped gate/up product with the clamped gated unit in its epilogue (see gated_unit above): out bfloat16 [M, N/2].
+AIRUN_EXPORT int airun_gemm_tcgen05_grouped_glu(const void* x, const void* W, void* out, int M, int N, int K, long long ldx,
+                                                long long ldc, const int32_t* seg, int n_seg, float limit, float slope, int* err,
+                                                cudaStream_t stream) {
+    if (!(limit > 0.0f)) return AIRUN_ERR_ARG;
+    return gemm_grouped(x, W, out, M, N, K, ldx, ldc, EPI_SWIGLU, seg, n_seg, err, stream, 0, limit, slope);
+}
+
 static int gemm_grouped(const void* x, const void* W, void* out, int M, int N, int K, long long ldx, long long ldc, int epi,
-                        const int32_t* seg, int n_seg, int* err, cudaStream_t stream, int act) {
+                        const int32_t* seg, int n_seg, int* err, cudaStream_t stream, int act, float glu_limit, float glu_slope) {
     if (M <= 0 || N <= 0 || K <= 0 || !err || !seg || n_seg <= 0) return M == 0 ? AIRUN_OK : AIRUN_ERR_ARG;
     if (K % 8 != 0 || ldx % 8 != 0 || ((uintptr_t)x & 15) || ((uintptr_t)W & 15)) return AIRUN_ERR_ARG;
     if (epi == EPI_SWIGLU && (N % 32 != 0)) return AIRUN_ERR_ARG;
@@ -1130,6 +1139,8 @@ static int gemm_grouped(const void* x, const void* W, void* out, int M, int N, i
     p.seg = seg;
     p.n_seg = n_seg;
     p.act = act;
+    p.glu_limit = glu_limit;
+    p.glu_slope = glu_slope;
     CUtensorMap ma, mb;
     int r;
     if ((r = make_map(&ma, x, M, K, ldx, BM)) != AIRUN_OK) return r;

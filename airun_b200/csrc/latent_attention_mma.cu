@@ -11,6 +11,7 @@
 //                    tiles arrive by cp.async in two stages (the next one is on its way while this one is used);
 //   single tokens:   one row tile, key tiles of 128 rows of which each of the 8 warps takes 16, one stage; the warps'
 //                    (maximum, sum, output) are merged through shared memory at the end, in warp order.
+// Each head's result may be times a sigmoid (`gate`, see latent_attention.cu).
 // A cached row is found through the request's block table.  A group of TOK batch rows that straddles two requests is handled
 // request by request.  Every row keeps its own maximum and sum, so a token's result does not depend on the batch.
 #include "common.cuh"
@@ -47,6 +48,8 @@ struct LatentMmaArgs {
     int T, num_reqs, num_pages, page_size, H, R, rd, window;
     float scale_log2;             // scale * log2(e)
     const float* sink;
+    const float* gate;            // [T][gate_stride]: head h's result is times sigmoid(gate[t][h]); null: no gate
+    long long gate_stride;
     int hg, tok;                  // heads of a CTA, tokens of a CTA
     int kd16, kdp;                // the row padded to k-steps of 16; the shared-memory row stride in elements
     int* err;
@@ -260,7 +263,8 @@ __global__ __launch_bounds__(32 * RW * KW, 1) void latent_attention_mma_kernel(L
                     wgt[w] = s_m[w * 16 + r] == -INFINITY ? 0.0f : exp2f(s_m[w * 16 + r] - gm);
                     gl += s_l[w * 16 + r] * wgt[w];
                 }
-                const float inv = gl > 0.0f ? 1.0f / gl : 0.0f;
+                float inv = gl > 0.0f ? 1.0f / gl : 0.0f;
+                if (a.gate) inv /= 1.0f + __expf(-a.gate[(size_t)(tb + tl) * a.gate_stride + h]);
                 __nv_bfloat16* dst = a.out + ((size_t)(tb + tl) * a.H + h) * a.R;
                 for (int c = cs; c < LM_CW && c0 + c < a.R; c += 8) {
                     float v = 0.0f;
@@ -281,7 +285,8 @@ __global__ __launch_bounds__(32 * RW * KW, 1) void latent_attention_mma_kernel(L
                     scale_o = m == -INFINITY ? 0.0f : exp2f(m - mf);
                     l = l * scale_o + exp2f(sk - mf);
                 }
-                const float inv = l > 0.0f ? scale_o / l : 0.0f;
+                float inv = l > 0.0f ? scale_o / l : 0.0f;
+                if (a.gate) inv /= 1.0f + __expf(-a.gate[(size_t)(tb + tl) * a.gate_stride + h]);
                 __nv_bfloat16* dst = a.out + ((size_t)(tb + tl) * a.H + h) * a.R + c0;
 #pragma unroll
                 for (int nt = 0; nt < LM_NT; ++nt) {
@@ -301,10 +306,11 @@ __global__ __launch_bounds__(32 * RW * KW, 1) void latent_attention_mma_kernel(L
 AIRUN_EXPORT int airun_latent_attention_mma(const void* qlat, void* out, const void* pool, const int32_t* block_table,
                                             int max_blocks, const int32_t* positions, const int32_t* req_of_token, int T,
                                             int num_reqs, int num_pages, int page_size, int H, int R, int rd, float scale,
-                                            int window, const float* sink, int single, int* err, cudaStream_t stream) {
+                                            int window, const float* sink, const float* gate, long long gate_stride, int single,
+                                            int* err, cudaStream_t stream) {
     const int KD = R + rd;
     if (T < 0 || H <= 0 || R <= 0 || rd < 0 || KD % 8 != 0 || KD > 1024 || page_size <= 0 || num_pages <= 0 || max_blocks <= 0 ||
-        window < 0 || !err || (((uintptr_t)qlat | (uintptr_t)pool) & 15))
+        window < 0 || !err || (gate && gate_stride < H) || (((uintptr_t)qlat | (uintptr_t)pool) & 15))
         return AIRUN_ERR_ARG;
     if (T == 0) return AIRUN_OK;
     LatentMmaArgs a = {};
@@ -312,7 +318,7 @@ AIRUN_EXPORT int airun_latent_attention_mma(const void* qlat, void* out, const v
     a.block_table = block_table; a.max_blocks = max_blocks; a.positions = positions; a.req_of_token = req_of_token;
     a.T = T; a.num_reqs = num_reqs; a.num_pages = num_pages; a.page_size = page_size; a.H = H; a.R = R; a.rd = rd; a.window = window;
     a.scale_log2 = scale * 1.4426950408889634f;
-    a.sink = sink; a.err = err;
+    a.sink = sink; a.gate = gate; a.gate_stride = gate_stride; a.err = err;
     a.kd16 = (KD + 15) / 16 * 16;
     a.kdp = a.kd16 + 8;
     // prompt portions: 8 row tiles (128 rows) a CTA when its queries and two key tiles fit the shared memory, else 4;

@@ -74,18 +74,23 @@ __global__ __launch_bounds__(128) void moe_route_kernel(
         for (int k = 0; k < top; ++k) wts[(size_t)t * top + k] /= total;
 }
 
-// Routing by softmax scores with a correction and groups.  z [T][n_out] are the router's outputs, of which the first
+// Routing by groups, by softmax scores with a correction or by sigmoid scores.  z [T][n_out] are the router's outputs, of which the first
 // `num_real` stand for experts with matrices and the rest for experts that return their input; all of them take part in
 // the softmax, the groups and the choice alike.
-//   s = softmax(z) over all outputs;   c = s + correction  (the choice score; the weights use s)
-//   the outputs form `groups` equal runs of neighbours; a run's score is its largest c, and only outputs of the `keep`
-//   best runs can be chosen (the others count as minus infinity: c may be negative)
-//   the `top` largest c are chosen (equal: the lower id);  weight = s / (sum of the chosen s + 1e-20) * weight_scale
+//   s = softmax(z) over all outputs, or sigmoid(z) each (`sigmoid_scores`);   c = s + correction  (the choice score; the
+//   weights use s)
+//   the outputs form `groups` equal runs of neighbours; a run's score is its largest c, or the sum of its two largest
+//   (`group_best` 2; a run of one has one), and only outputs of the `keep` best runs can be chosen (the others count as
+//   minus infinity: c may be negative)
+//   the `top` largest c are chosen (equal: the lower id);  weight = s / (sum of the chosen s + 1e-20) * weight_scale, or
+//   without `renorm` s * weight_scale
+// Sigmoid scores without a correction are ranked by their logits: the order is the same, and scores that round to 1 are
+// still told apart.
 // One warp per token.  Only experts with matrices are counted into segments.
 __global__ __launch_bounds__(128) void moe_route_grouped_kernel(
     const float* __restrict__ z, long long z_stride, const float* __restrict__ correction, int T, int n_out, int num_real, int top,
-    int groups, int keep, float weight_scale, const int32_t* __restrict__ req_of_token, int32_t* __restrict__ ids,
-    float* __restrict__ wts, int32_t* __restrict__ rank, int32_t* __restrict__ counts) {
+    int groups, int keep, int sigmoid_scores, int group_best, int renorm, float weight_scale, const int32_t* __restrict__ req_of_token,
+    int32_t* __restrict__ ids, float* __restrict__ wts, int32_t* __restrict__ rank, int32_t* __restrict__ counts) {
     pdl_trigger();
     pdl_wait();
     extern __shared__ float s_all[];                     // [4][2 * n_out + groups]
@@ -106,25 +111,37 @@ __global__ __launch_bounds__(128) void moe_route_grouped_kernel(
         zmax = fmaxf(zmax, v);
     }
     zmax = warp_max(zmax);
-    float zsum = 0.0f;
-    for (int e = lane; e < n_out; e += 32) {
-        const float v = expf(s_score[e] - zmax);
-        s_score[e] = v;
-        zsum += v;
-    }
-    zsum = warp_sum(zsum);
-    for (int e = lane; e < n_out; e += 32) {
-        const float sc = s_score[e] / zsum;
-        s_score[e] = sc;
-        s_choice[e] = sc + (correction ? correction[e] : 0.0f);
+    if (sigmoid_scores) {
+        for (int e = lane; e < n_out; e += 32) {
+            const float v = s_score[e], sc = 1.0f / (1.0f + expf(-v));
+            s_score[e] = sc;
+            s_choice[e] = correction ? sc + correction[e] : v;
+        }
+    } else {
+        float zsum = 0.0f;
+        for (int e = lane; e < n_out; e += 32) {
+            const float v = expf(s_score[e] - zmax);
+            s_score[e] = v;
+            zsum += v;
+        }
+        zsum = warp_sum(zsum);
+        for (int e = lane; e < n_out; e += 32) {
+            const float sc = s_score[e] / zsum;
+            s_score[e] = sc;
+            s_choice[e] = sc + (correction ? correction[e] : 0.0f);
+        }
     }
     __syncwarp();
     if (groups > 1) {
         const int per = n_out / groups;
         for (int g = lane; g < groups; g += 32) {
-            float best = -INFINITY;
-            for (int e = g * per; e < (g + 1) * per; ++e) best = fmaxf(best, s_choice[e]);
-            s_group[g] = best;
+            const float* c = sigmoid_scores && !correction ? s_score : s_choice;
+            float best = -INFINITY, second = -INFINITY;
+            for (int e = g * per; e < (g + 1) * per; ++e) {
+                second = fmaxf(second, fminf(best, c[e]));
+                best = fmaxf(best, c[e]);
+            }
+            s_group[g] = group_best == 2 && per > 1 ? best + second : best;
         }
         __syncwarp();
         // a run is kept when fewer than `keep` runs beat it (a run beats another with a larger score, or an equal one and a lower id)
@@ -163,7 +180,8 @@ __global__ __launch_bounds__(128) void moe_route_grouped_kernel(
         __syncwarp();
     }
     if (lane == 0)
-        for (int k = 0; k < top; ++k) wts[(size_t)t * top + k] = wts[(size_t)t * top + k] / (total + 1e-20f) * weight_scale;
+        for (int k = 0; k < top; ++k)
+            wts[(size_t)t * top + k] = (renorm ? wts[(size_t)t * top + k] / (total + 1e-20f) : wts[(size_t)t * top + k]) * weight_scale;
 }
 
 __global__ void moe_offsets_kernel(const int32_t* __restrict__ counts, int32_t* __restrict__ seg, int E) {
@@ -233,15 +251,16 @@ AIRUN_EXPORT int airun_moe_route(const float* z, long long z_stride, const float
 }
 
 AIRUN_EXPORT int airun_moe_route_grouped(const float* z, long long z_stride, const float* correction, int T, int n_out, int num_real,
-                                         int top, int groups, int keep, float weight_scale, const int32_t* req_of_token, int32_t* ids,
-                                         float* wts, int32_t* rank, int32_t* counts, int32_t* seg, cudaStream_t stream) {
+                                         int top, int groups, int keep, int sigmoid_scores, int group_best, int renorm,
+                                         float weight_scale, const int32_t* req_of_token, int32_t* ids, float* wts,
+                                         int32_t* rank, int32_t* counts, int32_t* seg, cudaStream_t stream) {
     if (T < 0 || n_out <= 0 || z_stride < n_out || n_out > MOE_MAX_EXPERTS || num_real <= 0 || num_real > n_out || top <= 0 || groups <= 0 ||
-        n_out % groups != 0 || keep <= 0 || keep > groups || top > (n_out / groups) * keep || !z || !req_of_token || !ids || !wts || !rank ||
+        n_out % groups != 0 || keep <= 0 || keep > groups || group_best < 1 || group_best > 2 || top > (n_out / groups) * keep || !z || !req_of_token || !ids || !wts || !rank ||
         !counts || !seg)
         return AIRUN_ERR_ARG;
     if (T == 0) return AIRUN_OK;
     airun_launch(moe_route_grouped_kernel, dim3(ceil_div_i(T, 4)), dim3(128), (size_t)4 * (2 * n_out + groups) * sizeof(float), stream, z,
-                 z_stride, correction, T, n_out, num_real, top, groups, keep, weight_scale, req_of_token, ids, wts, rank, counts);
+                 z_stride, correction, T, n_out, num_real, top, groups, keep, sigmoid_scores, group_best, renorm, weight_scale, req_of_token, ids, wts, rank, counts);
     airun_launch(moe_offsets_kernel, dim3(1), dim3(32), 0, stream, (const int32_t*)counts, seg, num_real);
     return airun_launch_status();
 }

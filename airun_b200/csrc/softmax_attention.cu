@@ -2,6 +2,7 @@
 //
 //   q = Wq h (+ bq),  k = Wk h (+ bk),  v = Wv h (+ bv)                  the products are the caller's, biases are added here
 //   q, k <- x / rms(x) * w            per head, one weight vector for all heads        (`q_w`, `k_w`: before the rotation)
+//                                     or ONE root mean square over all heads of the token, a weight per row (`whole_norm`)
 //   q, k <- rotation by the position  (none, pairs (i, i + r/2), or pairs (2i, 2i + 1)) over the first r dimensions
 //   q, k <- x / rms(x)                per head, no weight                              (`unit_norm`: after the rotation)
 //   q <- q * (1 + coef * ln(floor((p + 1) / every) + 1))                               (`temp_every` > 0)
@@ -9,6 +10,8 @@
 //   p_ij = exp(s_ij) / (sum over visible j' of exp(s_ij') + exp(sink_h))               (`sink`: one more term of the denominator
 //                                                                                       that has no key and no value)
 //   o_i = out_scale * sum_j p_ij v_j,     j visible iff j <= i and (window == 0 or i - j < window)
+//   o_i <- o_i * sigmoid(gate_i)                                                       (`gate`: a number per element, a product of the
+//                                                                                       same input as q, k and v)
 //
 // Query head h reads KV head h / (heads / kv_heads); key rows have D elements, value rows Dv.  Norms, angles, the
 // temperature, scores, the softmax and the sum over keys are float32; q, keys and values are stored in the type of
@@ -40,7 +43,7 @@ __device__ __forceinline__ void xa_store4(__nv_bfloat16* dst, float4 v) {
 template <typename T>
 __global__ __launch_bounds__(32 * XA_PREP_WARPS) void qkv_prepare_kernel(
     const float* __restrict__ proj, long long proj_stride, const float* __restrict__ bias, const float* __restrict__ q_w,
-    const float* __restrict__ k_w, int unit_norm, float eps, int rope_kind, int rdim, const float* __restrict__ inv_freq,
+    const float* __restrict__ k_w, int whole_norm, int unit_norm, float eps, int rope_kind, int rdim, const float* __restrict__ inv_freq,
     const int32_t* __restrict__ rope_positions, float temp_coef, int temp_every, T* __restrict__ q_out, T* __restrict__ pool,
     const int32_t* __restrict__ block_table, int max_blocks, const int32_t* __restrict__ positions,
     const int32_t* __restrict__ req_of_token, int num_reqs, int num_pages, int page_size, int nh, int nkv, int D, int Dv,
@@ -77,6 +80,20 @@ __global__ __launch_bounds__(32 * XA_PREP_WARPS) void qkv_prepare_kernel(
     __shared__ float s_cos[16 * XA_MAX_PER_LANE], s_sin[16 * XA_MAX_PER_LANE];
     if (rope_kind != XA_ROPE_NONE)
         for (int i = threadIdx.x; i < (rdim >> 1); i += blockDim.x) sincosf(rpos * inv_freq[i], &s_sin[i], &s_cos[i]);
+    // one root mean square over all rows of q and one over all rows of k, worked out ahead of the heads
+    float whole_q = 1.0f, whole_k = 1.0f;
+    if (whole_norm) {
+        __shared__ float s_red[33];
+        const int qn = nh * D, kn = store ? nkv * D : 0;
+        float sq = 0.0f, sk = 0.0f;
+        for (int c = threadIdx.x; c < qn + kn; c += blockDim.x) {
+            const float v = row[c] + (bias ? bias[c] : 0.0f);
+            if (c < qn) sq = fmaf(v, v, sq);
+            else sk = fmaf(v, v, sk);
+        }
+        whole_q = 1.0f / sqrtf(block_sum(sq, s_red) / (float)qn + eps);
+        if (kn) whole_k = 1.0f / sqrtf(block_sum(sk, s_red) / (float)kn + eps);
+    }
     __syncthreads();
     const float temp = temp_every > 0 ? 1.0f + temp_coef * logf((float)((pos + 1) / temp_every) + 1.0f) : 1.0f;
     const int units = nh + (store ? nkv : 0);
@@ -95,6 +112,7 @@ __global__ __launch_bounds__(32 * XA_PREP_WARPS) void qkv_prepare_kernel(
             const bool is_q = u < nh;
             const int col0 = u * D;
             const float* w = is_q ? q_w : k_w;
+            if (w && whole_norm) w += is_q ? col0 : col0 - nh * D;
             float4 x[2];
             float ss = 0.0f;
 #pragma unroll
@@ -111,7 +129,7 @@ __global__ __launch_bounds__(32 * XA_PREP_WARPS) void qkv_prepare_kernel(
                 ss = fmaf(x[i].x, x[i].x, ss); ss = fmaf(x[i].y, x[i].y, ss); ss = fmaf(x[i].z, x[i].z, ss); ss = fmaf(x[i].w, x[i].w, ss);
             }
             if (w) {
-                const float inv = 1.0f / sqrtf(warp_sum(ss) / (float)D + eps);
+                const float inv = whole_norm ? (is_q ? whole_q : whole_k) : 1.0f / sqrtf(warp_sum(ss) / (float)D + eps);
 #pragma unroll
                 for (int i = 0; i < 2; ++i) {
                     const int d = 4 * lane + 128 * i;
@@ -198,6 +216,7 @@ __global__ __launch_bounds__(32 * XA_PREP_WARPS) void qkv_prepare_kernel(
         const bool is_q = u < nh;
         const int col0 = u * D;                      // q heads and k heads follow each other in the row
         const float* w = is_q ? q_w : k_w;
+        if (w && whole_norm) w += is_q ? col0 : col0 - nh * D;
         float x[XA_MAX_PER_LANE];
         float ss = 0.0f;
 #pragma unroll
@@ -207,7 +226,7 @@ __global__ __launch_bounds__(32 * XA_PREP_WARPS) void qkv_prepare_kernel(
             ss = fmaf(x[i], x[i], ss);
         }
         if (w) {
-            const float inv = 1.0f / sqrtf(warp_sum(ss) / (float)D + eps);
+            const float inv = whole_norm ? (is_q ? whole_q : whole_k) : 1.0f / sqrtf(warp_sum(ss) / (float)D + eps);
 #pragma unroll
             for (int i = 0; i < XA_MAX_PER_LANE; ++i) {
                 const int d = lane + 32 * i;
@@ -274,7 +293,7 @@ __global__ __launch_bounds__(32 * XA_PREP_WARPS) void qkv_prepare_kernel(
 }
 
 AIRUN_EXPORT int airun_qkv_prepare(const float* proj, long long proj_stride, const float* bias, const float* q_w, const float* k_w,
-                                   int unit_norm, float eps, int rope_kind, int rdim, const float* inv_freq,
+                                   int whole_norm, int unit_norm, float eps, int rope_kind, int rdim, const float* inv_freq,
                                    const int32_t* rope_positions, float temp_coef, int temp_every, void* q_out, void* pool,
                                    int dtype, const int32_t* block_table, int max_blocks, const int32_t* positions,
                                    const int32_t* req_of_token, int T, int num_reqs, int num_pages, int page_size, int nh,
@@ -282,12 +301,12 @@ AIRUN_EXPORT int airun_qkv_prepare(const float* proj, long long proj_stride, con
     if (T < 0 || nh <= 0 || nkv <= 0 || D <= 0 || D > 32 * XA_MAX_PER_LANE || Dv <= 0 || temp_every < 0 || !err || !positions ||
         !req_of_token || !proj || !q_out || rdim < 0 || rdim > D || (rdim & 1) ||
         (rope_kind != XA_ROPE_NONE && rdim > 0 && !inv_freq) || rope_kind < 0 || rope_kind > 2 ||
-        (one_row && (Dv != D || k_w || unit_norm || (rope_kind == XA_ROPE_NONE && rdim > 0))) ||
+        (whole_norm && (!q_w || (store && !k_w))) || (one_row && (Dv != D || k_w || unit_norm || (rope_kind == XA_ROPE_NONE && rdim > 0))) ||
         (store && (!pool || !block_table || page_size <= 0 || num_pages <= 0 || max_blocks <= 0)))
         return AIRUN_ERR_ARG;
     if (T == 0) return AIRUN_OK;
 #define XP_LAUNCH(TT) airun_launch(qkv_prepare_kernel<TT>, dim3(T), dim3(32 * XA_PREP_WARPS), 0, stream, proj, proj_stride, bias, q_w, \
-        k_w, unit_norm, eps, rope_kind, rdim, inv_freq, rope_positions, temp_coef, temp_every, (TT*)q_out, (TT*)pool, block_table, \
+        k_w, whole_norm, unit_norm, eps, rope_kind, rdim, inv_freq, rope_positions, temp_coef, temp_every, (TT*)q_out, (TT*)pool, block_table, \
         max_blocks, positions, req_of_token, num_reqs, num_pages, page_size, nh, nkv, D, Dv, store, one_row, err)
     if (dtype == AIRUN_DT_F32) XP_LAUNCH(float);
     else if (dtype == AIRUN_DT_BF16) XP_LAUNCH(__nv_bfloat16);
@@ -305,7 +324,7 @@ __global__ __launch_bounds__(32 * XA_WARPS) void softmax_attention_kernel(
     const int32_t* __restrict__ block_table, int max_blocks, const int32_t* __restrict__ positions,
     const int32_t* __restrict__ req_of_token, int num_reqs, int num_pages, int page_size, int nh, int nkv, int D, int Dv,
     float scale, const float* __restrict__ table, int table_len, const float* __restrict__ sink, int window, float out_scale,
-    int tail, int* __restrict__ err) {
+    int tail, const float* __restrict__ gate, long long gate_stride, int* __restrict__ err) {
     pdl_trigger();
     pdl_wait();
     extern __shared__ float s_acc[];           // [XA_WARPS][Dv], then [XA_WARPS] maxima and [XA_WARPS] sums
@@ -386,7 +405,9 @@ __global__ __launch_bounds__(32 * XA_WARPS) void softmax_attention_kernel(
         float o = 0.0f;
 #pragma unroll
         for (int w = 0; w < XA_WARPS; ++w) o = fmaf(s_acc[(size_t)w * Dv + d], f[w], o);
-        dst[d] = from_f32<T>(o * inv);
+        o *= inv;
+        if (gate) o /= 1.0f + expf(-gate[(size_t)t * gate_stride + (size_t)head * Dv + d]);
+        dst[d] = from_f32<T>(o);
     }
 }
 
@@ -394,17 +415,19 @@ AIRUN_EXPORT int airun_softmax_attention(const void* q, void* out, long long out
                                          const int32_t* block_table, int max_blocks, const int32_t* positions,
                                          const int32_t* req_of_token, int T, int num_reqs, int num_pages, int page_size,
                                          int nh, int nkv, int D, int Dv, float scale, const float* table, int table_len,
-                                         const float* sink, int window, float out_scale, int tail, int* err, cudaStream_t stream) {
+                                         const float* sink, int window, float out_scale, int tail, const float* gate,
+                                         long long gate_stride, int* err, cudaStream_t stream) {
     if (T < 0 || nh <= 0 || nkv <= 0 || nh % nkv != 0 || D <= 0 || D > 32 * XA_MAX_PER_LANE || Dv <= 0 ||
         Dv > 32 * XA_MAX_PER_LANE || page_size <= 0 || num_pages <= 0 || max_blocks <= 0 || window < 0 || !err || nh > 65535 ||
-        out_stride < (long long)nh * Dv || (table && table_len <= 0) || tail > D || (tail >= 0 && Dv != D))
+        out_stride < (long long)nh * Dv || (table && table_len <= 0) || tail > D || (tail >= 0 && Dv != D) ||
+        (gate && gate_stride < (long long)nh * Dv))
         return AIRUN_ERR_ARG;
     if (T == 0) return AIRUN_OK;
     dim3 grid(T, nh);
     const size_t smem = ((size_t)XA_WARPS * Dv + 2 * XA_WARPS) * sizeof(float);
 #define XA_LAUNCH(TT) airun_launch(softmax_attention_kernel<TT>, grid, dim3(32 * XA_WARPS), smem, stream, (const TT*)q, (TT*)out, \
         out_stride, (const TT*)pool, block_table, max_blocks, positions, req_of_token, num_reqs, num_pages, page_size, nh, nkv, D, Dv, \
-        scale, table, table_len, sink, window, out_scale, tail, err)
+        scale, table, table_len, sink, window, out_scale, tail, gate, gate_stride, err)
     if (dtype == AIRUN_DT_F32) XA_LAUNCH(float);
     else if (dtype == AIRUN_DT_BF16) XA_LAUNCH(__nv_bfloat16);
     else return AIRUN_ERR_UNSUPPORTED;

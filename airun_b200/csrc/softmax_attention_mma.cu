@@ -4,6 +4,7 @@
 //
 //   s_ij = scale * q_i . k_j + table[h][min(i - j, table_len - 1)]
 //   o_i = out_scale * sum_j exp(s_ij) v_j / (sum_j exp(s_ij) + exp(sink_h))     over j <= i (and i - j < window)
+//   o_i <- o_i * sigmoid(gate_i)     (`gate`: a number per element of o; null: nothing)
 //
 // One CTA (4 warps) takes up to 64 consecutive tokens of one request and one query head; a warp owns 16 of them and
 // keeps, per row, a running maximum and sum: a key tile's scores (float32, kept as log2 of the weights) lower the
@@ -47,6 +48,16 @@ __device__ __forceinline__ float xam_exp2(float x) {
     float e;
     asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(x));
     return e;
+}
+
+// two neighbouring results of a row, gated when there is a gate, rounded and stored (c: the first one's dimension)
+__device__ __forceinline__ void xam_put2(__nv_bfloat16* dst, const float* gate, int c, int Dv, float v0, float v1) {
+    if (c >= Dv) return;
+    if (gate) v0 /= 1.0f + __expf(-gate[c]);
+    dst[c] = __float2bfloat16_rn(v0);
+    if (c + 1 >= Dv) return;
+    if (gate) v1 /= 1.0f + __expf(-gate[c + 1]);
+    dst[c + 1] = __float2bfloat16_rn(v1);
 }
 
 // ---- bulk copies (one instruction a row, carried out by the copy engine) and the barrier that counts their bytes
@@ -103,6 +114,8 @@ struct XamParams {
     int table_len;
     const float* sink;            // [nh]: exp(sink) joins the denominator; null: no sink
     float out_scale;
+    const float* gate;            // [T][gate_stride] float32, columns head * Dv + d: the result is times its sigmoid; null: no gate
+    long long gate_stride;
     int window;
     int tail;                     // one row for key and value: elements before the value begins; -1: rows of their own
     int skip_single;              // requests that bring ONE token are left to the kernel for single tokens
@@ -411,12 +424,9 @@ __global__ __launch_bounds__(128) void softmax_attention_mma_kernel(const XamPar
         const float inv = den > 0.0f ? p.out_scale * f / den : 0.0f;
         if (row >= n) continue;
         __nv_bfloat16* dst = p.out + (size_t)(first + row) * p.out_stride + (size_t)head * Dv;
+        const float* gate = p.gate ? p.gate + (size_t)(first + row) * p.gate_stride + (size_t)head * Dv : nullptr;
 #pragma unroll
-        for (int i = 0; i < DVP / 8; ++i) {
-            const int c = i * 8 + 2 * t;
-            if (c < Dv) dst[c] = __float2bfloat16_rn(O[i][2 * h] * inv);
-            if (c + 1 < Dv) dst[c + 1] = __float2bfloat16_rn(O[i][2 * h + 1] * inv);
-        }
+        for (int i = 0; i < DVP / 8; ++i) xam_put2(dst, gate, i * 8 + 2 * t, Dv, O[i][2 * h] * inv, O[i][2 * h + 1] * inv);
     }
 }
 
@@ -685,12 +695,9 @@ __global__ __launch_bounds__(128) void softmax_attention_group_kernel(const XamP
             const float d = den[h] * fo + (p.sink ? xam_exp2(sink2 - all) : 0.0f);
             const float inv = d > 0.0f ? p.out_scale * fo / d : 0.0f;
             __nv_bfloat16* dst = p.out + (size_t)tok * p.out_stride + col;
+            const float* gate = p.gate ? p.gate + (size_t)tok * p.gate_stride + col : nullptr;
 #pragma unroll
-            for (int i = 0; i < DVP / 8; ++i) {
-                const int c = i * 8 + 2 * t;
-                if (c < Dv) dst[c] = __float2bfloat16_rn(O[i][2 * h] * inv);
-                if (c + 1 < Dv) dst[c + 1] = __float2bfloat16_rn(O[i][2 * h + 1] * inv);
-            }
+            for (int i = 0; i < DVP / 8; ++i) xam_put2(dst, gate, i * 8 + 2 * t, Dv, O[i][2 * h] * inv, O[i][2 * h + 1] * inv);
         }
     }
 }
@@ -718,7 +725,9 @@ __global__ __launch_bounds__(128) void xam_reduce_kernel(const XamParams p) {
     float acc = 0.0f;
 #pragma unroll 4
     for (int s = 0; s < p.splits; ++s) acc = fmaf(col[s * slice], __shfl_sync(0xffffffffu, w, s), acc);
-    if (c < Dv) p.out[(size_t)tok * p.out_stride + (size_t)head * Dv + c] = __float2bfloat16_rn(acc * inv);
+    acc *= inv;
+    if (c < Dv && p.gate) acc /= 1.0f + __expf(-p.gate[(size_t)tok * p.gate_stride + (size_t)head * Dv + c]);
+    if (c < Dv) p.out[(size_t)tok * p.out_stride + (size_t)head * Dv + c] = __float2bfloat16_rn(acc);
 }
 
 template <int DP, int DVP, bool ONE>
@@ -756,7 +765,8 @@ static int xam_launch(const XamParams& p, int max_tiles, cudaStream_t stream) {
 static bool xam_fill(XamParams& p, const void* q, void* out, long long out_stride, const void* pool, const int32_t* block_table,
                      int max_blocks, const int32_t* cu_tokens, const int32_t* context_lens, int num_reqs, int num_pages,
                      int page_size, int nh, int nkv, int D, int Dv, float scale, const float* table, int table_len,
-                     const float* sink, int window, float out_scale, int tail, int* err) {
+                     const float* sink, int window, float out_scale, int tail, const float* gate, long long gate_stride, int* err) {
+    if (gate && gate_stride < (long long)nh * Dv) return false;
     if (tail > D || (tail >= 0 && Dv != D)) return false;
     if (num_reqs < 0 || nh <= 0 || nkv <= 0 || nh % nkv != 0 || D <= 0 || D > 128 || Dv <= 0 || Dv > 128 || page_size <= 0 ||
         num_pages <= 0 || max_blocks <= 0 || window < 0 || !err || nh > 65535 || out_stride < (long long)nh * Dv || !cu_tokens ||
@@ -766,7 +776,7 @@ static bool xam_fill(XamParams& p, const void* q, void* out, long long out_strid
     p.pool = (const __nv_bfloat16*)pool; p.block_table = block_table; p.max_blocks = max_blocks;
     p.cu_tokens = cu_tokens; p.context_lens = context_lens; p.num_reqs = num_reqs; p.num_pages = num_pages;
     p.page_size = page_size; p.nh = nh; p.nkv = nkv; p.D = D; p.Dv = Dv; p.scale = scale;
-    p.table = table; p.table_len = table_len; p.sink = sink; p.out_scale = out_scale; p.window = window; p.tail = tail; p.skip_single = 0;
+    p.table = table; p.table_len = table_len; p.sink = sink; p.out_scale = out_scale; p.gate = gate; p.gate_stride = gate_stride; p.window = window; p.tail = tail; p.skip_single = 0;
     p.partial = nullptr; p.splits = 1; p.T = 0; p.err = err;
     return true;
 }
@@ -796,10 +806,10 @@ AIRUN_EXPORT int airun_softmax_attention_mma(const void* q, void* out, long long
                                              const int32_t* context_lens, int num_reqs, int max_tiles, int num_pages,
                                              int page_size, int nh, int nkv, int D, int Dv, float scale, const float* table,
                                              int table_len, const float* sink, int window, float out_scale, int tail,
-                                             int skip_single, int* err, cudaStream_t stream) {
+                                             const float* gate, long long gate_stride, int skip_single, int* err, cudaStream_t stream) {
     XamParams p;
     if (max_tiles < 0 || !xam_fill(p, q, out, out_stride, pool, block_table, max_blocks, cu_tokens, context_lens, num_reqs, num_pages,
-                                   page_size, nh, nkv, D, Dv, scale, table, table_len, sink, window, out_scale, tail, err))
+                                   page_size, nh, nkv, D, Dv, scale, table, table_len, sink, window, out_scale, tail, gate, gate_stride, err))
         return AIRUN_ERR_ARG;
     if (num_reqs == 0 || max_tiles == 0) return AIRUN_OK;
     p.skip_single = skip_single;
@@ -814,11 +824,12 @@ AIRUN_EXPORT int airun_softmax_attention_group(const void* q, void* out, long lo
                                                const int32_t* block_table, int max_blocks, const int32_t* cu_tokens,
                                                const int32_t* context_lens, int num_reqs, int num_pages, int page_size,
                                                int nh, int nkv, int D, int Dv, float scale, const float* table, int table_len,
-                                               const float* sink, int window, float out_scale, int tail, int splits,
+                                               const float* sink, int window, float out_scale, int tail, const float* gate,
+                                               long long gate_stride, int splits,
                                                float* partial, int T, int* err, cudaStream_t stream) {
     XamParams p;
     if (!xam_fill(p, q, out, out_stride, pool, block_table, max_blocks, cu_tokens, context_lens, num_reqs, num_pages, page_size,
-                  nh, nkv, D, Dv, scale, table, table_len, sink, window, out_scale, tail, err) ||
+                  nh, nkv, D, Dv, scale, table, table_len, sink, window, out_scale, tail, gate, gate_stride, err) ||
         nh / nkv > 16 || num_reqs > 65535 || splits < 1 || splits > 32 || (splits > 1 && (!partial || T <= 0)))
         return AIRUN_ERR_ARG;
     if (num_reqs == 0) return AIRUN_OK;

@@ -268,10 +268,10 @@ class DecoderModel:
         if isinstance(delta, PostNormWrite):            # the last result joins the stream on the final norm's way
             if hasattr(self.final_norm, "fusable"):
                 w, eps = self.final_norm.fusable()
-                ops.sandwich_norm(x, hsel, y=delta.y, w_post=delta.weight, eps_post=delta.eps, w_pre=w, eps_pre=eps, rows=want_rows[:n_want])
+                ops.sandwich_norm(x, hsel, w_pre=w, eps_pre=eps, rows=want_rows[:n_want], **delta.norm_args())
                 delta = hsel
             else:
-                ops.sandwich_norm(x, None, y=delta.y, w_post=delta.weight, eps_post=delta.eps)
+                ops.sandwich_norm(x, None, **delta.norm_args())
                 delta = None
         if delta is not hsel:
             self.final_norm.forward(ctx, x, hsel, delta=delta, rows=want_rows[:n_want])
@@ -285,8 +285,12 @@ class DecoderModel:
         if isinstance(pending, torch.Tensor):
             return x[:T] + pending[:T]
         if isinstance(pending, PostNormWrite):
-            y = pending.y[:T]
-            return x[:T] + y / torch.sqrt((y * y).mean(dim=-1, keepdim=True) + pending.eps) * pending.weight
+            out = x[:T].clone()
+            for y, w in ((pending.y, pending.weight), (pending.y2, pending.weight2)):
+                if y is not None:
+                    y = y[:T]
+                    out += pending.mult * (y / torch.sqrt((y * y).mean(dim=-1, keepdim=True) + pending.eps) * w)
+            return out
         return x[:T] if pending is None or isinstance(pending, CastActivations) else None
 
     def _forward_streams(self, ctx, x: torch.Tensor, want_rows: Optional[torch.Tensor], n_want: int) -> Optional[torch.Tensor]:

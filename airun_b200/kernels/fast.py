@@ -226,11 +226,11 @@ GROUPED_MAX_TILES = 1024
 
 
 def grouped_linear_bf16(ctx, x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, seg: torch.Tensor, swiglu_group: int = 0,
-                        act: Optional[int] = None) -> bool:
+                        act: Optional[int] = None, glu: Optional[Tuple[float, float]] = None) -> bool:
     """Rows seg[e] .. seg[e+1]-1 of x [M, K] times w[e]^T (w [E, N, K]) on tcgen05, the segments read from the device.
     ``act`` (an ``ops.ACT_*``; not with ``swiglu_group``): the activation applied to the finished sums in the epilogue.
     ``swiglu_group`` 16: the rows of w[e] alternate between blocks of 16 gate and 16 up rows and out is the gated
-    unit's result, bfloat16 [M, N/2]; 0: out [M, N] float32 or bfloat16.  False when the kernel does not take the
+    unit's result, bfloat16 [M, N/2] (SwiGLU, or the clamped unit with ``glu`` = (limit, slope)); 0: out [M, N] float32 or bfloat16.  False when the kernel does not take the
     sizes (the caller then uses the plain grouped product)."""
     M, K = x.shape
     E, N = w.shape[0], w.shape[1]
@@ -255,6 +255,14 @@ def grouped_linear_bf16(ctx, x: torch.Tensor, w: torch.Tensor, out: torch.Tensor
         _check(f(_p(x), _p(w), _p(out), M, N, K, x.stride(0) if M > 1 else max(K, x.stride(0)),
                  out.stride(0) if M > 1 else max(out.shape[1], out.stride(0)), epi, _p(seg), E, int(act), _p(ctx.err), _stream()),
                "gemm_tcgen05_grouped_act")
+        return True
+    if swiglu_group and glu is not None:
+        f = _fn("gemm_tcgen05", "airun_gemm_tcgen05_grouped_glu",
+                [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_longlong, c_longlong, c_void_p, c_int, c_float, c_float, c_void_p,
+                 c_void_p])
+        _check(f(_p(x), _p(w), _p(out), M, N, K, x.stride(0) if M > 1 else max(K, x.stride(0)),
+                 out.stride(0) if M > 1 else max(out.shape[1], out.stride(0)), _p(seg), E, float(glu[0]), float(glu[1]), _p(ctx.err),
+                 _stream()), "gemm_tcgen05_grouped_glu")
         return True
     f = _fn("gemm_tcgen05", "airun_gemm_tcgen05_grouped",
             [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_longlong, c_longlong, c_int, c_void_p, c_int, c_void_p, c_void_p])
@@ -648,7 +656,7 @@ def diff_attention_bf16(ctx, q, out, cache, part) -> bool:
     return True
 
 
-def latent_attention_bf16(ctx, qlat, out, cache, part) -> bool:
+def latent_attention_bf16(ctx, qlat, out, cache, part, gate: Optional[torch.Tensor] = None) -> bool:
     """Attention over a cached latent on the tensor cores (csrc/latent_attention_mma.cu): prompt portions with several
     tokens a CTA, steps of single tokens with one token a CTA whose warps share the keys.  False: the caller runs the
     plain kernel (rows that are no multiple of 8 elements, or too long for the shared memory)."""
@@ -657,7 +665,7 @@ def latent_attention_bf16(ctx, qlat, out, cache, part) -> bool:
     if ("latent_attention" in DISABLED or qlat.dtype != torch.bfloat16 or cache.pool.dtype != torch.bfloat16 or KD % 8
             or KD > 640):
         return False
-    _cuda(qlat, out, cache.pool, cache.block_table, ctx.positions, ctx.req_of_token, ctx.err, part.sink)
+    _cuda(qlat, out, cache.pool, cache.block_table, ctx.positions, ctx.req_of_token, ctx.err, part.sink, gate)
     T = qlat.shape[0]
     _need(tuple(qlat.shape) == (T, H * KD) and qlat.is_contiguous() and tuple(out.shape) == (T, H * R) and out.is_contiguous()
           and out.dtype == torch.bfloat16, "qlat / out must be contiguous bfloat16 [T, H*(R+rd)] / [T, H*R]")
@@ -666,10 +674,10 @@ def latent_attention_bf16(ctx, qlat, out, cache, part) -> bool:
     _need(qlat.data_ptr() % 16 == 0 and pool.data_ptr() % 16 == 0, "qlat and the cache pages must begin on 16-byte boundaries")
     f = _fn("latent_attention_mma", "airun_latent_attention_mma",
             [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
-             c_float, c_int, c_void_p, c_int, c_void_p, c_void_p])
+             c_float, c_int, c_void_p, c_void_p, c_longlong, c_int, c_void_p, c_void_p])
     _check(f(_p(qlat), _p(out), _p(pool), _p(bt), bt.stride(0), _p(ctx.positions), _p(ctx.req_of_token), T, int(ctx.num_reqs),
              pool.shape[0], int(cache.page_size), H, R, rd, float(part.scale), int(part.window), _p(part.sink),
-             1 if getattr(ctx, "decode_only", False) else 0, _p(ctx.err), _stream()), "latent_attention_mma")
+             _p(gate), ops.attention_gate(gate, T, H), 1 if getattr(ctx, "decode_only", False) else 0, _p(ctx.err), _stream()), "latent_attention_mma")
     return True
 
 
@@ -762,8 +770,8 @@ def sigmoid_attention_bf16(ctx, q, out, cache, part) -> bool:
     return True
 
 
-def softmax_attention_bf16(ctx, q, out, cache, part) -> bool:
-    """Softmax attention with a window, a distance table, a sink and a factor on the tensor cores
+def softmax_attention_bf16(ctx, q, out, cache, part, gate: Optional[torch.Tensor] = None) -> bool:
+    """Softmax attention with a window, a distance table, a sink, a factor and a gate on the tensor cores
     (csrc/softmax_attention_mma.cu) for every row of the batch: prompt portions in tiles of 64 tokens of one head, single
     tokens with the query heads of a KV head as the rows and their keys cut into slices; False: the caller runs the
     plain kernel (head sizes above 128)."""
@@ -771,7 +779,7 @@ def softmax_attention_bf16(ctx, q, out, cache, part) -> bool:
     if ("softmax_attention" in DISABLED or q.dtype != torch.bfloat16 or cache.pool.dtype != torch.bfloat16 or D > 128 or Dv > 128
             or q.data_ptr() % 16 or cache.pool.data_ptr() % 16):
         return False
-    _cuda(q, out, cache.pool, cache.block_table, ctx.cu_tokens, ctx.context_lens, ctx.err, part.table, part.sink)
+    _cuda(q, out, cache.pool, cache.block_table, ctx.cu_tokens, ctx.context_lens, ctx.err, part.table, part.sink, gate)
     T = q.shape[0]
     _need(tuple(q.shape) == (T, nh * D) and q.is_contiguous(), "q must be contiguous [T, heads*D]")
     _need(tuple(out.shape) == (T, nh * Dv) and out.stride(1) == 1 and out.dtype == torch.bfloat16,
@@ -792,9 +800,9 @@ def softmax_attention_bf16(ctx, q, out, cache, part) -> bool:
     common = [_p(q), _p(out), out.stride(0) if T > 1 else max(out.shape[1], out.stride(0)), _p(pool), _p(bt), bt.stride(0),
               _p(ctx.cu_tokens), _p(ctx.context_lens), int(ctx.num_reqs)]
     consts = [pool.shape[0], int(cache.page_size), nh, nkv, D, Dv, float(part.scale), _p(part.table), int(table_len), _p(part.sink),
-              int(part.window), float(part.out_scale), tail]
+              int(part.window), float(part.out_scale), tail, _p(gate), ops.attention_gate(gate, T, nh * Dv)]
     sig = [c_void_p, c_void_p, c_longlong, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int]
-    csig = [c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_void_p, c_int, c_void_p, c_int, c_float, c_int]
+    csig = [c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_void_p, c_int, c_void_p, c_int, c_float, c_int, c_void_p, c_longlong]
     # requests that bring ONE token go to the kernel whose product rows are the query heads of a KV head (groups of up
     # to 16), which finds them on the device; the tile kernel then skips them
     single = "softmax_group" not in DISABLED and nh // nkv <= 16

@@ -264,16 +264,22 @@ SANDWICH_NORM, SANDWICH_COPY, SANDWICH_SPLIT = 0, 1, 2
 def sandwich_norm(x: torch.Tensor, out: Optional[torch.Tensor], y: Optional[torch.Tensor] = None,
                   w_post: Optional[torch.Tensor] = None, eps_post: float = 0.0, w_pre: Optional[torch.Tensor] = None,
                   eps_pre: float = 0.0, rows: Optional[torch.Tensor] = None, mode: int = SANDWICH_NORM,
-                  write_back: bool = True) -> None:
+                  write_back: bool = True, y2: Optional[torch.Tensor] = None, w_post2: Optional[torch.Tensor] = None,
+                  mult: float = 1.0) -> None:
     """v = x [+ y / rms(y) * w_post] and, in the same pass, ``out`` by ``mode``: v / rms(v) * w_pre (SANDWICH_NORM), v in
     float32 (SANDWICH_COPY) or v as two bfloat16 halves side by side, [T, 2n], whose sum is v to 16 bits (SANDWICH_SPLIT).
-    v becomes x unless ``rows`` picks the rows (out[0..len(rows))) or ``write_back`` is False."""
-    _cuda(x, out, y, w_post, w_pre, rows)
+    v becomes x unless ``rows`` picks the rows (out[0..len(rows))) or ``write_back`` is False.  With ``y2`` two normed
+    results join at once, v = x + mult * (y / rms(y) * w_post + y2 / rms(y2) * w_post2), eps_post in both."""
+    _cuda(x, out, y, w_post, w_pre, rows, y2, w_post2)
     _need(x.dtype == torch.float32 and x.dim() == 2 and x.is_contiguous(), "x must be contiguous float32 [T, n]")
     T, n = x.shape
     if y is not None:
         _need(y.dtype == torch.float32 and y.shape == x.shape and y.is_contiguous(), "y must match x")
-    for w in (w_post, w_pre):
+    _need((y2 is None) == (w_post2 is None) and (y2 is None or y is not None) and (y2 is not None or mult == 1.0),
+          "a second result comes with its norm weight beside a first one; the factor belongs to the pair")
+    if y2 is not None:
+        _need(y2.dtype == torch.float32 and y2.shape == x.shape and y2.is_contiguous(), "y2 must match x")
+    for w in (w_post, w_pre, w_post2):
         _need(w is None or (w.dtype == torch.float32 and tuple(w.shape) == (n,) and w.is_contiguous()), "norm weights must be float32 [n]")
     n_rows = T
     if rows is not None:
@@ -283,8 +289,9 @@ def sandwich_norm(x: torch.Tensor, out: Optional[torch.Tensor], y: Optional[torc
         _need(out.dim() == 2 and out.shape[0] >= n_rows and out.shape[1] == (2 * n if mode == SANDWICH_SPLIT else n) and out.is_contiguous(),
               "out must be contiguous [rows, n] ([rows, 2n] for a split)")
     f = _fn("elementwise", "airun_sandwich_norm",
-            [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_float, c_float, c_int, c_int, c_void_p])
-    _check(f(_p(x), _p(y), _p(w_post), _p(w_pre), _p(out), _dt(out) if out is not None else DT_F32, _p(rows), n_rows, n,
+            [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_float, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_float, c_float,
+             c_int, c_int, c_void_p])
+    _check(f(_p(x), _p(y), _p(w_post), _p(y2), _p(w_post2), float(mult), _p(w_pre), _p(out), _dt(out) if out is not None else DT_F32, _p(rows), n_rows, n,
              float(eps_post), float(eps_pre), 1 if write_back and rows is None else 0, int(mode), _stream()), "sandwich_norm")
 
 
@@ -692,13 +699,14 @@ def stream_step(xs: torch.Tensor, y: Optional[torch.Tensor] = None, carry: Optio
 def qkv_prepare(proj: torch.Tensor, bias: Optional[torch.Tensor], q_w: Optional[torch.Tensor], k_w: Optional[torch.Tensor],
                 unit_norm: bool, eps: float, rope_kind: int, rotary_dim: int, inv_freq: Optional[torch.Tensor],
                 temp_coef: float, temp_every: int, q_out: torch.Tensor, cache, ctx, nh: int, nkv: int, D: int, Dv: int,
-                store: bool = True, rope_positions: Optional[torch.Tensor] = None, one_row: bool = False) -> None:
+                store: bool = True, rope_positions: Optional[torch.Tensor] = None, one_row: bool = False, whole_norm: bool = False) -> None:
     """What lies between the q/k/v product and the attention (csrc/softmax_attention.cu: qkv_prepare_kernel): biases,
     a weighted root-mean-square norm per head before the rotation (``q_w`` / ``k_w`` float32 [D]), the rotation, an
     unweighted norm per head after it (``unit_norm``), the query temperature; q out, k and v into the token's page.
     ``proj`` float32 rows [q heads | k heads | v heads] (q heads only without ``store``).  ``one_row``: the values are
     the keys before the rotation, so proj has no value columns and a cached row is [key | its first ``rotary_dim``
-    dimensions unrotated], D + rotary_dim elements."""
+    dimensions unrotated], D + rotary_dim elements.  ``whole_norm``: ONE root mean square over all rows of q and one over
+    all rows of k instead of one per head, with weights of those sizes ([nh * D], [nkv * D])."""
     _cuda(proj, bias, q_w, k_w, inv_freq, q_out, cache.pool, cache.block_table, ctx.positions, ctx.req_of_token, ctx.err, rope_positions)
     _rows_f32(proj, "proj")
     T = proj.shape[0]
@@ -709,32 +717,43 @@ def qkv_prepare(proj: torch.Tensor, bias: Optional[torch.Tensor], q_w: Optional[
     _need(q_out.is_contiguous() and tuple(q_out.shape) == (T, nh * D), "q_out must be contiguous [T, heads*D]")
     if bias is not None:
         _need(bias.dtype == torch.float32 and bias.numel() >= width and bias.is_contiguous(), "the biases must be float32 [q | k | v]")
-    for w_ in (q_w, k_w):
-        _need(w_ is None or (w_.dtype == torch.float32 and w_.numel() == D and w_.is_contiguous()), "a q/k norm weight must be float32 [D]")
+    for w_, heads in ((q_w, nh), (k_w, nkv)):
+        _need(w_ is None or (w_.dtype == torch.float32 and w_.numel() == (heads * D if whole_norm else D) and w_.is_contiguous()),
+              "a q/k norm weight must be float32 [D], or [heads * D] for a norm over the whole projection")
     _need(D <= 256, "head sizes above 256 are beyond the kernel")
     pool, bt = cache.pool, cache.block_table
     if store:
         _need(pool.dtype == q_out.dtype and pool.is_contiguous() and pool[0].numel() == nkv * cache.page_size * row,
               "the cache pages do not fit the head sizes or the type of q")
     f = _fn("softmax_attention", "airun_qkv_prepare",
-            [c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_int, c_float, c_int, c_int, c_void_p, c_void_p, c_float, c_int,
+            [c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_int, c_int, c_float, c_int, c_int, c_void_p, c_void_p, c_float, c_int,
              c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
              c_int, c_int, c_void_p, c_void_p])
-    _check(f(_p(proj), _row_stride(proj), _p(bias), _p(q_w), _p(k_w), 1 if unit_norm else 0, float(eps), int(rope_kind),
+    _check(f(_p(proj), _row_stride(proj), _p(bias), _p(q_w), _p(k_w), 1 if whole_norm else 0, 1 if unit_norm else 0, float(eps), int(rope_kind),
              int(rotary_dim), _p(inv_freq), _p(rope_positions), float(temp_coef), int(temp_every), _p(q_out), _p(pool), _dt(q_out),
              _p(bt), bt.stride(0), _p(ctx.positions), _p(ctx.req_of_token), T, int(ctx.num_reqs), pool.shape[0],
              int(cache.page_size), nh, nkv, D, Dv, 1 if store else 0, 1 if one_row else 0, _p(ctx.err), _stream()), "qkv_prepare")
 
 
+def attention_gate(gate: Optional[torch.Tensor], T: int, width: int) -> int:
+    """Checks the gate an attention kernel multiplies its results by (float32 [T, width], before its sigmoid; columns of a
+    wider buffer are fine) and returns its row stride."""
+    if gate is None:
+        return 0
+    _rows_f32(gate, "gate")
+    _need(tuple(gate.shape) == (T, width), f"the gate must be [T, {width}]")
+    return _row_stride(gate)
+
+
 def softmax_attention(q: torch.Tensor, out: torch.Tensor, cache, ctx, nh: int, nkv: int, D: int, Dv: int, scale: float,
                       table: Optional[torch.Tensor] = None, sink: Optional[torch.Tensor] = None, window: int = 0,
-                      out_scale: float = 1.0, tail: int = -1) -> None:
+                      out_scale: float = 1.0, tail: int = -1, gate: Optional[torch.Tensor] = None) -> None:
     """Softmax attention over cache pages in float32 arithmetic (csrc/softmax_attention.cu: softmax_attention_kernel):
     ``table`` float32 [heads, n] adds table[h, min(i - j, n - 1)] to the scaled score, ``sink`` float32 [heads] adds
     exp(sink_h) to the denominator, ``window`` > 0 hides keys with i - j >= window; the result is times ``out_scale``.
     ``out`` may be a column slice of a wider buffer.  ``tail`` >= 0: a cached row of D + tail elements is key (its first D)
-    and value (its last D) at once."""
-    _cuda(q, out, cache.pool, cache.block_table, ctx.positions, ctx.req_of_token, ctx.err, table, sink)
+    and value (its last D) at once.  ``gate`` float32 [T, heads*Dv] (a column slice is fine): the result is times its sigmoid."""
+    _cuda(q, out, cache.pool, cache.block_table, ctx.positions, ctx.req_of_token, ctx.err, table, sink, gate)
     T = q.shape[0]
     _need(q.is_contiguous() and tuple(q.shape) == (T, nh * D), "q must be contiguous [T, heads*D]")
     _need(tuple(out.shape) == (T, nh * Dv) and out.stride(1) == 1 and out.dtype == q.dtype, "out must be row-major [T, heads*Dv] of q's type")
@@ -749,12 +768,13 @@ def softmax_attention(q: torch.Tensor, out: torch.Tensor, cache, ctx, nh: int, n
         table_len = table.shape[1]
     if sink is not None:
         _need(sink.dtype == torch.float32 and sink.numel() == nh and sink.is_contiguous(), "the sinks must be float32 [heads]")
+    gate_stride = attention_gate(gate, T, nh * Dv)
     f = _fn("softmax_attention", "airun_softmax_attention",
             [c_void_p, c_void_p, c_longlong, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int,
-             c_int, c_int, c_int, c_float, c_void_p, c_int, c_void_p, c_int, c_float, c_int, c_void_p, c_void_p])
+             c_int, c_int, c_int, c_float, c_void_p, c_int, c_void_p, c_int, c_float, c_int, c_void_p, c_longlong, c_void_p, c_void_p])
     _check(f(_p(q), _p(out), _row_stride(out), _p(pool), _dt(q), _p(bt), bt.stride(0), _p(ctx.positions), _p(ctx.req_of_token), T,
              int(ctx.num_reqs), pool.shape[0], int(cache.page_size), nh, nkv, D, Dv, float(scale), _p(table), int(table_len),
-             _p(sink), int(window), float(out_scale), int(tail), _p(ctx.err), _stream()), "softmax_attention")
+             _p(sink), int(window), float(out_scale), int(tail), _p(gate), gate_stride, _p(ctx.err), _stream()), "softmax_attention")
 
 
 # ---------------------------------------------------------------- products
@@ -914,7 +934,7 @@ def _latent_pool(pool: torch.Tensor, page_size: int, row: int) -> int:
 
 def latent_prepare(proj: torch.Tensor, wq: torch.Tensor, wkv: Optional[torch.Tensor], eps: float, cq: torch.Tensor,
                    R: int, rd: int, rot_dims: int, inv_freq: Optional[torch.Tensor], rot_mult: float, cache, ctx,
-                   store: bool) -> None:
+                   store: bool, rope_kind: int = ROPE_INTERLEAVED) -> None:
     """cq = rmsnorm(proj[:, :q_rank]) * wq; with ``store`` the token's cache row becomes
     [rmsnorm(proj[:, q_rank : q_rank+R]) * wkv | rotate(proj[:, q_rank+R : q_rank+R+rd])]."""
     _cuda(proj, wq, wkv, cq, inv_freq)
@@ -929,34 +949,46 @@ def latent_prepare(proj: torch.Tensor, wq: torch.Tensor, wkv: Optional[torch.Ten
         _need(pool.dtype == cq.dtype, "the latent query and the cache pages must share a type")
         max_blocks = bt.stride(0)
     f = _fn("latent_attention", "airun_latent_prepare",
-            [c_void_p, c_longlong, c_void_p, c_void_p, c_float, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_float,
+            [c_void_p, c_longlong, c_void_p, c_void_p, c_float, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_float,
              c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p])
-    _check(f(_p(proj), _row_stride(proj), _p(wq), _p(wkv), float(eps), _p(cq), _dt(cq), q_rank, R, rd, rot_dims, _p(inv_freq),
+    _check(f(_p(proj), _row_stride(proj), _p(wq), _p(wkv), float(eps), _p(cq), _dt(cq), q_rank, R, rd, rot_dims, int(rope_kind), _p(inv_freq),
              float(rot_mult), _p(pool), _p(bt), max_blocks, _p(ctx.positions), _p(ctx.req_of_token), T, int(ctx.num_reqs),
              num_pages, int(cache.page_size), 1 if store else 0, _p(ctx.err), _stream()), "latent_prepare")
 
 
 def latent_query(q: torch.Tensor, qn: torch.Tensor, qlat: torch.Tensor, H: int, D: int, R: int, rd: int, rot_dims: int,
-                 inv_freq: Optional[torch.Tensor], rot_mult: float, ctx) -> None:
+                 inv_freq: Optional[torch.Tensor], rot_mult: float, ctx, rope_kind: int = ROPE_INTERLEAVED,
+                 wkv: Optional[torch.Tensor] = None, eps: float = 0.0, cache=None) -> None:
     """q float32 [T, H*(D+rd)] -> qn [T, H*D] (the unrotated parts) and the rotated parts, turned by each token's
-    position, into qlat[t, h, R:] (qlat [T, H*(R+rd)])."""
-    _cuda(q, qn, qlat, inv_freq)
+    position, into qlat[t, h, R:] (qlat [T, H*(R+rd)]).  With ``cache`` the rows of q go on with R + rd more columns, and
+    the token's cache row becomes [rmsnorm(of the first R) * wkv | rotate(the last rd)] in the same launch."""
+    _cuda(q, qn, qlat, inv_freq, wkv)
+    _rows_f32(q, "q")
     T = q.shape[0]
-    _need(q.dtype == torch.float32 and tuple(q.shape) == (T, H * (D + rd)) and q.is_contiguous(), "q must be float32 [T, H*(D+rd)]")
+    _need(q.shape[1] >= H * (D + rd) + (R + rd if cache is not None else 0), "q must be float32 [T, H*(D+rd)] (and R+rd columns to cache)")
+    num_pages = max_blocks = page_size = 0
+    pool = bt = None
+    if cache is not None:
+        pool, bt, page_size = cache.pool, cache.block_table, int(cache.page_size)
+        num_pages, max_blocks = _latent_pool(pool, page_size, R + rd), bt.stride(0)
+        _need(pool.dtype == qn.dtype, "the latent query and the cache pages must share a type")
+        _need(wkv is not None and wkv.dtype == torch.float32 and wkv.numel() == R and wkv.is_contiguous(), "wkv must be float32 [R]")
     _need(tuple(qn.shape) == (T, H * D) and qn.is_contiguous() and tuple(qlat.shape) == (T, H * (R + rd)) and qlat.is_contiguous()
           and qn.dtype == qlat.dtype, "qn / qlat must be contiguous [T, H*D] / [T, H*(R+rd)] of one type")
     f = _fn("latent_attention", "airun_latent_query",
-            [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_float, c_void_p, c_void_p,
-             c_void_p])
-    _check(f(_p(q), _p(qn), _p(qlat), _dt(qn), T, H, D, R, rd, rot_dims, _p(inv_freq), float(rot_mult), _p(ctx.positions),
-             _p(ctx.req_of_token), _stream()), "latent_query")
+            [c_void_p, c_longlong, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_float,
+             c_void_p, c_void_p, c_void_p, c_float, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p])
+    _check(f(_p(q), _row_stride(q), _p(qn), _p(qlat), _dt(qn), T, H, D, R, rd, rot_dims, int(rope_kind), _p(inv_freq), float(rot_mult),
+             _p(ctx.positions), _p(ctx.req_of_token), _p(wkv), float(eps), _p(pool), _p(bt), max_blocks, int(ctx.num_reqs), num_pages,
+             page_size, _p(ctx.err), _stream()), "latent_query")
 
 
 def latent_attention(qlat: torch.Tensor, out: torch.Tensor, cache, ctx, H: int, R: int, rd: int, scale: float, window: int,
-                     sink: Optional[torch.Tensor]) -> None:
+                     sink: Optional[torch.Tensor], gate: Optional[torch.Tensor] = None) -> None:
     """out[t, h] = sum_j p_j c_j over the cached rows [c | kr] each token sees (0 <= pos - j < window, or all with
-    window 0), p the softmax of scale * qlat[t, h] . [c_j | kr_j] with exp(sink[h]) added to its denominator."""
-    _cuda(qlat, out, sink)
+    window 0), p the softmax of scale * qlat[t, h] . [c_j | kr_j] with exp(sink[h]) added to its denominator; times
+    sigmoid(gate[t, h]) with ``gate`` float32 [T, H]."""
+    _cuda(qlat, out, sink, gate)
     T = qlat.shape[0]
     _need(tuple(qlat.shape) == (T, H * (R + rd)) and qlat.is_contiguous() and tuple(out.shape) == (T, H * R) and out.is_contiguous()
           and out.dtype == qlat.dtype, "qlat / out must be contiguous [T, H*(R+rd)] / [T, H*R] of one type")
@@ -967,10 +999,10 @@ def latent_attention(qlat: torch.Tensor, out: torch.Tensor, cache, ctx, H: int, 
         _need(sink.dtype == torch.float32 and sink.numel() == H and sink.is_contiguous(), "sink must be float32 [H]")
     f = _fn("latent_attention", "airun_latent_attention",
             [c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
-             c_int, c_float, c_int, c_void_p, c_void_p, c_void_p])
+             c_int, c_float, c_int, c_void_p, c_void_p, c_longlong, c_void_p, c_void_p])
     _check(f(_p(qlat), _p(out), _dt(qlat), _p(cache.pool), _p(cache.block_table), cache.block_table.stride(0), _p(ctx.positions),
              _p(ctx.req_of_token), T, int(ctx.num_reqs), num_pages, int(cache.page_size), H, R, rd, float(scale), int(window),
-             _p(sink), _p(ctx.err), _stream()), "latent_attention")
+             _p(sink), _p(gate), attention_gate(gate, T, H), _p(ctx.err), _stream()), "latent_attention")
 
 
 # ---------------------------------------------------------------- routed experts
@@ -1029,12 +1061,15 @@ def moe_combine(ys: torch.Tensor, top: int, ids, wts, row_of, scale_output: bool
 
 def moe_route_grouped(logits: torch.Tensor, num_real: int, top: int, groups: int, keep: int, weight_scale: float,
                       correction: Optional[torch.Tensor], req_of_token: torch.Tensor, ids: torch.Tensor, wts: torch.Tensor,
-                      rank: torch.Tensor, counts: torch.Tensor, seg: torch.Tensor) -> None:
+                      rank: torch.Tensor, counts: torch.Tensor, seg: torch.Tensor, sigmoid_scores: bool = False,
+                      group_best: int = 1, renorm: bool = True) -> None:
     """Routing by softmax scores with a correction and groups (csrc/moe.cu: moe_route_grouped_kernel).  ``logits``
     float32 [T, n_out]: the first ``num_real`` outputs are experts with matrices, the rest return their input.  Scores
     are the softmax over all outputs; the choice is by score + ``correction`` inside the ``keep`` best of ``groups``
     equal runs of neighbouring outputs; weights are the chosen scores over their sum (+ 1e-20) times ``weight_scale``.
-    ``counts`` (int32 [num_real]) must be zero on entry; seg [num_real + 1]."""
+    ``counts`` (int32 [num_real]) must be zero on entry; seg [num_real + 1].  ``sigmoid_scores``: scores are sigmoids of
+    the logits; ``group_best`` 2: a group's score is the sum of its two largest; without ``renorm`` the weights are the
+    chosen scores times ``weight_scale``."""
     _cuda(logits, correction, req_of_token, ids, wts, rank, counts, seg)
     _rows_f32(logits, "logits")
     T, n_out = logits.shape
@@ -1049,10 +1084,10 @@ def moe_route_grouped(logits: torch.Tensor, num_real: int, top: int, groups: int
         _need(correction.dtype == torch.float32 and correction.numel() == n_out and correction.is_contiguous(),
               "the correction must be float32 [router outputs]")
     f = _fn("moe", "airun_moe_route_grouped",
-            [c_void_p, c_longlong, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_void_p, c_void_p, c_void_p, c_void_p,
-             c_void_p, c_void_p, c_void_p])
+            [c_void_p, c_longlong, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_void_p, c_void_p,
+             c_void_p, c_void_p, c_void_p, c_void_p, c_void_p])
     _check(f(_p(logits), _row_stride(logits), _p(correction), T, n_out, int(num_real), int(top), int(groups), int(keep),
-             float(weight_scale), _p(req_of_token), _p(ids), _p(wts), _p(rank), _p(counts), _p(seg), _stream()), "moe_route_grouped")
+             1 if sigmoid_scores else 0, int(group_best), 1 if renorm else 0, float(weight_scale), _p(req_of_token), _p(ids), _p(wts), _p(rank), _p(counts), _p(seg), _stream()), "moe_route_grouped")
 
 
 # ---------------------------------------------------------------- attention

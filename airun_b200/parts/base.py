@@ -23,7 +23,8 @@ Head            forward(ctx, h [rows, hidden], out float32 [rows, vocab])
 ResidualInput   begin(ctx, x0) -> kept; forward(ctx, x, pending, kept) -> pending: the residual stream mixed
                   with the embedding ahead of a pass over layers that run several times
 Mixer           cache_spec() -> PagedKVSpec | StateSpec | None
-                forward(ctx, h, cache) -> float32 [T, hidden] (the residual delta)
+                forward(ctx, h, cache) -> float32 [T, hidden] (the residual delta), or a PostNormWrite when its
+                results are normed on their way into the residual (arrangements "pre_norm" takes it)
 FeedForward     forward(ctx, h) -> float32 [T, hidden]
                 Optional, for both: the split form, which lets an arrangement run the output products
                 of several sub-layers as ONE product over their concatenated activations:
@@ -110,10 +111,18 @@ class CastActivations:
 class PostNormWrite:
     """What a block whose sub-layers' results are normed on their way out leaves pending: the result ``y`` [T, H] of its
     last sub-layer and that norm's weight and eps, x += y / rms(y) * weight; the pass that next reads the residual (the
-    next block's first norm, a mix of the residual with the embedding, the final norm) carries it out on its way."""
+    next block's first norm, a mix of the residual with the embedding, the final norm) carries it out on its way.
+    With ``y2`` two normed results join at once, x += mult * (y / rms(y) * weight + y2 / rms(y2) * weight2)."""
     y: torch.Tensor
     weight: torch.Tensor
     eps: float
+    y2: Optional[torch.Tensor] = None
+    weight2: Optional[torch.Tensor] = None
+    mult: float = 1.0
+
+    def norm_args(self) -> dict:
+        """The keyword arguments of ops.sandwich_norm that carry this write out."""
+        return dict(y=self.y, w_post=self.weight, eps_post=self.eps, y2=self.y2, w_post2=self.weight2, mult=self.mult)
 
 
 @dataclass

@@ -10,6 +10,10 @@ In the bfloat16 path, when the parts on both sides allow it (``fuses_norms``), a
 kernel of its own at all: the product that ends a sub-layer adds its result to x, writes
 bfloat16(x * norm weight) and the sums of x^2 per token, and the product that starts the next
 sub-layer scales each token's results by rsqrt(mean x^2 + eps) (parts/base.py NormedActivations).
+
+A mixer may leave its result to be normed on its way into the residual (parts/base.py PostNormWrite); the norm that
+reads the residual next then carries out that norm, the add and its own norm in one pass, and a block that ends with
+such a mixer passes it on to the block behind it.
 """
 from __future__ import annotations
 
@@ -21,12 +25,27 @@ from ..weights.loader import WeightSpec
 from .base import CastActivations, FeedForward, Mixer, Norm, NormedActivations, Part, PostNormWrite, ResidualSink, StreamWrite, register_part
 
 
+def read_residual(ctx, x: torch.Tensor, pending, norm: Norm, dtype: torch.dtype) -> torch.Tensor:
+    """norm(x) in the compute type once what is pending (None, a float32 delta or a PostNormWrite) is in x."""
+    h = ctx.ws.alloc(tuple(x.shape), dtype)
+    if isinstance(pending, PostNormWrite):
+        from ..kernels import ops
+        w, eps = norm.fusable()
+        ops.sandwich_norm(x, h, w_pre=w, eps_pre=eps, **pending.norm_args())
+    else:
+        norm.forward(ctx, x, h, delta=pending)
+    return h
+
+
 class PreNormBlock(Part):
-    def __init__(self, norm1: Norm, mixer: Mixer, norm2: Norm, ffn: FeedForward, dtype: torch.dtype):
+    """x += mixer(norm1(x)), then x += ffn(norm2(x)); the feed-forward may be absent, and then so is norm2."""
+    norm2_belongs_to_ffn = True
+
+    def __init__(self, norm1: Norm, mixer: Mixer, norm2: Optional[Norm], ffn: Optional[FeedForward], dtype: torch.dtype):
         self.norm1, self.mixer, self.norm2, self.ffn, self.dtype = norm1, mixer, norm2, ffn, dtype
 
     def parts(self):
-        return (self.norm1, self.mixer, self.norm2, self.ffn)
+        return tuple(p for p in (self.norm1, self.mixer, self.norm2, self.ffn) if p is not None)
 
     def weight_specs(self) -> List[WeightSpec]:
         return [s for p in self.parts() for s in p.weight_specs()]
@@ -52,27 +71,21 @@ class PreNormBlock(Part):
             and hasattr(self.norm1, "fusable")
 
     def forward(self, ctx, x: torch.Tensor, pending, cache, next_norm: Optional[Norm] = None):
-        """``pending``: what the block before left: None, a float32 delta still to be added to x, or
-        NormedActivations (x is up to date and this block's first norm is already folded in).
+        """``pending``: what the block before left: None, a float32 delta still to be added to x, a
+        PostNormWrite, or NormedActivations (x is up to date and this block's first norm is already folded in).
         ``next_norm``: the norm that will read x next, if it may be folded into this block's last
         product; the block then returns NormedActivations instead of a delta."""
         T, H = x.shape
         bf16 = self.dtype == torch.bfloat16
-        if isinstance(pending, NormedActivations):
-            h = pending
-        else:
-            h = ctx.ws.alloc((T, H), self.dtype)
-            self.norm1.forward(ctx, x, h, delta=pending)
+        h = pending if isinstance(pending, NormedActivations) else read_residual(ctx, x, pending, self.norm1, self.dtype)
+        if self.ffn is None:
+            return self.mixer.forward(ctx, h, cache)
         if bf16 and getattr(self.mixer, "fuses_norms", False) and getattr(self.ffn, "fuses_norms", False) \
                 and hasattr(self.norm2, "fusable"):
             a = self.mixer.forward(ctx, h, cache, sink=ResidualSink(x, *self.norm2.fusable()))
         else:
             a = self.mixer.forward(ctx, h, cache)
-        if isinstance(a, NormedActivations):
-            h2 = a
-        else:
-            h2 = ctx.ws.alloc((T, H), self.dtype)
-            self.norm2.forward(ctx, x, h2, delta=a)
+        h2 = a if isinstance(a, NormedActivations) else read_residual(ctx, x, a, self.norm2, self.dtype)
         if bf16 and next_norm is not None and getattr(self.ffn, "fuses_norms", False):
             return self.ffn.forward(ctx, h2, sink=ResidualSink(x, *next_norm.fusable()))
         return self.ffn.forward(ctx, h2)
@@ -490,14 +503,7 @@ class SandwichBlock(Part):
 
     def _read(self, ctx, x: torch.Tensor, pending, norm: Norm) -> torch.Tensor:
         """The next sub-layer's input: norm(x) once what is pending (a PostNormWrite, or a plain delta) is in x."""
-        from ..kernels import ops
-        h = ctx.ws.alloc(tuple(x.shape), self.dtype)
-        w, eps = norm.fusable()
-        if isinstance(pending, PostNormWrite):
-            ops.sandwich_norm(x, h, y=pending.y, w_post=pending.weight, eps_post=pending.eps, w_pre=w, eps_pre=eps)
-        else:
-            ops.rmsnorm(x, w, eps, h, delta=pending if isinstance(pending, torch.Tensor) else None)
-        return h
+        return read_residual(ctx, x, pending if isinstance(pending, (torch.Tensor, PostNormWrite)) else None, norm, self.dtype)
 
     def forward(self, ctx, x: torch.Tensor, pending, cache, next_norm: Optional[Norm] = None):
         y = self.mixer.forward(ctx, self._read(ctx, x, pending, self.norm1), cache)

@@ -16,7 +16,9 @@ The state, the decays, beta, the unit vectors, the norm and the gate are float32
 and the last ``taps - 1`` inputs of the convolution live side by side in its slot of the cache manager's state
 tensor (one flat float32 row), so prompts cut anywhere, single tokens and whole prompts run the same recurrence.
 The six input projections run as one product over [Wq; Wk; Wv; Wb; Wa1; Wg1], with a silu gate [Wq; Wk; Wv; Wg; Wb; ...].
-A decay per head is worked out inside the recurrence's kernel, from its projection.
+A decay per head is worked out inside the recurrence's kernel, from its projection.  The part has the split form
+(parts/base.py): ``forward_core`` leaves the gated heads, times ``out_scale``, in a buffer, and can be handed the columns
+of a product that an arrangement has run over several parts' stacked input matrices (``proj``).
 """
 from __future__ import annotations
 
@@ -35,7 +37,8 @@ class GatedDeltaRule(Mixer):
 
     def __init__(self, prefix: str, hidden_size: int, num_heads: int, num_kv_heads: int, key_dim: int, value_dim: int,
                  conv_taps: int, norm_eps: float, decay_rank: int = 0, gate_rank: int = 0, decay: str = "channel",
-                 gate: str = "lowrank_sigmoid", unit_eps: float = 1e-6, q_scale: Optional[float] = None, dtype: torch.dtype = torch.bfloat16, device=None,
+                 gate: str = "lowrank_sigmoid", unit_eps: float = 1e-6, q_scale: Optional[float] = None,
+                 out_scale: float = 1.0, dtype: torch.dtype = torch.bfloat16, device=None,
                  names: Optional[Dict[str, str]] = None):
         self.prefix, self.H = prefix, int(hidden_size)
         self.nh, self.nkv, self.D, self.Dv = int(num_heads), int(num_kv_heads), int(key_dim), int(value_dim)
@@ -54,7 +57,7 @@ class GatedDeltaRule(Mixer):
             raise ValueError(f"heads ({num_heads}) must be a multiple of kv_heads ({num_kv_heads})")
         if self.D > 256:
             raise ValueError(f"{self.D} key channels a head are above the recurrence kernel's limit of 256")
-        self.eps, self.unit_eps = float(norm_eps), float(unit_eps)
+        self.eps, self.unit_eps, self.out_scale = float(norm_eps), float(unit_eps), float(out_scale)
         self.q_scale = float(q_scale) if q_scale is not None else self.D ** -0.5
         self.dtype, self.device = dtype, device
         n = dict(q="q", k="k", v="v", q_conv="q.conv", k_conv="k.conv", v_conv="v.conv", beta="b", a_log="A_log", norm="norm",
@@ -63,6 +66,7 @@ class GatedDeltaRule(Mixer):
         n.update(names or {})
         self.names = {k: f"{prefix}.{v}" for k, v in n.items()}
         self.kd, self.vd = self.nkv * self.D, self.nh * self.Dv
+        self.core_width = self.vd
         self.C = 2 * self.kd + self.vd                       # channels that pass the convolution
         self.state_matrix = self.nh * self.D * self.Dv       # the flat state: the matrices, then the convolution's tail
         self.w_in = self.w_out = self.conv_w = self.w_a2 = self.w_g2 = self.dt_bias = self.a_log = self.norm_w = None
@@ -95,16 +99,23 @@ class GatedDeltaRule(Mixer):
         self.w_g2 = None if self.silu_gate else tensors.pop(nm["gate_out"])
         self.w_out = tensors.pop(nm["o"])
         self.dt_bias, self.a_log, self.norm_w = tensors[nm["decay_bias"]], tensors[nm["a_log"]], tensors[nm["norm"]]
+        if self.out_scale != 1.0:           # the norm's weight is the last factor of the heads
+            self.norm_w = self.norm_w * self.out_scale
+
+    def adopt_w_out(self, view: torch.Tensor) -> None:
+        self.w_out = view
 
     # ---- cache ----
     def cache_spec(self):
         return StateSpec((self.state_matrix + (self.taps - 1) * self.C,), torch.float32)
 
     # ---- compute ----
-    def forward(self, ctx, h: torch.Tensor, cache, sink=None):
-        T, ws, C, nh = h.shape[0], ctx.ws, self.C, self.nh
-        proj = ws.alloc((T, C + nh + self.rank_a + self.rank_g), torch.float32)
-        linear(ctx, h, self.w_in, proj)
+    def forward_core(self, ctx, h: torch.Tensor, act: torch.Tensor, cache, proj: Optional[torch.Tensor] = None) -> None:
+        """Writes out_scale * the normed, gated heads into ``act`` ([T, heads * value_dim], rows may be strided)."""
+        T, ws, C, nh = act.shape[0], ctx.ws, self.C, self.nh
+        if proj is None:
+            proj = ws.alloc((T, C + nh + self.rank_a + self.rank_g), torch.float32)
+            linear(ctx, h, self.w_in, proj)
         at = C + (self.rank_g if self.silu_gate else 0)
         qkv, beta, low_a = proj[:, :C], proj[:, at:at + nh], proj[:, at + nh:at + nh + self.rank_a]
         low_g = proj[:, C:at] if self.silu_gate else proj[:, at + nh + self.rank_a:]
@@ -126,10 +137,14 @@ class GatedDeltaRule(Mixer):
                             conv[:, self.kd:2 * self.kd], conv[:, 2 * self.kd:], decay,
                             cache.state, ctx, o, nh, nh // self.nkv, self.D, self.Dv, beta=beta, tail_src=qkv,
                             tail_off=self.state_matrix, tail_rows=self.taps - 1, **per_head)
-        act = ws.alloc((T, self.vd), self.dtype)
         ops.gla_out_gate(o, gate, self.norm_w, self.eps, act, nh, self.Dv, ctx.req_of_token,
                          gate_act=ops.GATE_SILU if self.silu_gate else ops.GATE_AS_IS)
-        delta = ws.alloc((T, self.H), torch.float32)
+
+    def forward(self, ctx, h: torch.Tensor, cache, sink=None):
+        T = h.shape[0]
+        act = ctx.ws.alloc((T, self.vd), self.dtype)
+        self.forward_core(ctx, h, act, cache)
+        delta = ctx.ws.alloc((T, self.H), torch.float32)
         linear(ctx, act, self.w_out, delta)
         return delta
 

@@ -15,7 +15,10 @@ the choice is by s + correction (a learnt number per router output, tensor ``cor
 ``keep_groups`` best of ``groups`` equal runs of neighbouring outputs (a run's score is its largest s + correction),
 the weights are the chosen s over their sum (+ 1e-20) times ``weight_scale``; and ``identity_experts``: the router's
 last outputs stand for experts without matrices that return their input (they take part in the softmax, the groups and
-the choice like the others).
+the choice like the others).  ``group_best=2``: a run's score is the sum of its two largest; with sigmoid ``scores`` the
+runs and the choice go by them, and without ``renormalize`` the weights are the chosen scores themselves (times
+``weight_scale``).  ``expert="clamped_glu"`` with a ``limit``: the gated unit of parts/mlp.py ClampedGLU,
+g = min(Wgate x, limit), u = clamp(Wup x, -limit, limit), expert(x) = Wdown ( g sigmoid(slope g) (u + 1) ).
 
 Everything is decided on the device: a step's rows are sorted by expert into segments of one buffer and every
 expert's matrices meet only their own segment (csrc/moe.cu, the grouped product of csrc/gemm_simt.cu), so the part
@@ -41,7 +44,8 @@ class RoutedExperts(FeedForward):
     def __init__(self, prefix: str, hidden_size: int, intermediate_size: int, num_experts: int, top: int,
                  scores: str = "sigmoid", renormalize: bool = False, weight_on: str = "input", router_bias: bool = False,
                  expert: str = "swiglu", activation: str = "gelu_erf", routing: str = "top", choice_bias: bool = False,
-                 groups: int = 1, keep_groups: int = 1, identity_experts: int = 0, weight_scale: float = 1.0,
+                 groups: int = 1, keep_groups: int = 1, identity_experts: int = 0, weight_scale: float = 1.0, group_best: int = 1,
+                 limit: float = 0.0, slope: float = 1.702,
                  dtype: torch.dtype = torch.bfloat16, device=None, names: Optional[Dict[str, str]] = None):
         self.prefix, self.H, self.I = prefix, int(hidden_size), int(intermediate_size)
         self.E, self.top = int(num_experts), int(top)
@@ -53,20 +57,25 @@ class RoutedExperts(FeedForward):
         self.dtype, self.device = dtype, device
         self.group = INTERLEAVE if self.I % INTERLEAVE == 0 else self.I
         self.router_bias = bool(router_bias)
-        if expert not in ("swiglu", "act") or routing not in ("top", "grouped"):
-            raise ValueError("expert is 'swiglu' or 'act', routing is 'top' or 'grouped'")
+        if expert not in ("swiglu", "act", "clamped_glu") or routing not in ("top", "grouped"):
+            raise ValueError("expert is 'swiglu', 'clamped_glu' or 'act', routing is 'top' or 'grouped'")
+        if (expert == "clamped_glu") != (float(limit) > 0):
+            raise ValueError("a positive limit belongs to expert='clamped_glu'")
+        self.glu = (float(limit), float(slope)) if expert == "clamped_glu" else None
         if expert == "act" and activation not in ops.ACTIVATIONS:
             raise ValueError(f"activation must be one of {sorted(ops.ACTIVATIONS)}")
-        self.gated, self.act_mode = expert == "swiglu", ops.ACTIVATIONS.get(activation, 0)
+        self.gated, self.act_mode = expert != "act", ops.ACTIVATIONS.get(activation, 0)
         self.grouped_routing = routing == "grouped"
-        self.choice_bias, self.groups, self.keep = bool(choice_bias), int(groups), int(keep_groups)
+        self.choice_bias, self.groups, self.keep, self.group_best = bool(choice_bias), int(groups), int(keep_groups), int(group_best)
         self.identity, self.weight_scale = int(identity_experts), float(weight_scale)
         self.n_out = self.E + self.identity
-        if not self.grouped_routing and (self.choice_bias or self.groups != 1 or self.identity or self.weight_scale != 1.0):
+        if not self.grouped_routing and (self.choice_bias or self.groups != 1 or self.identity or self.weight_scale != 1.0 or self.group_best != 1):
             raise ValueError("a correction, groups, identity experts and a weight scale belong to routing='grouped'")
         if self.grouped_routing:
-            if not self.softmax or self.on_input or router_bias:
-                raise ValueError("grouped routing weighs the experts' outputs by softmax scores and has no bias on the logits")
+            if self.on_input or router_bias:
+                raise ValueError("grouped routing weighs the experts' outputs by their scores and has no bias on the logits")
+            if self.group_best not in (1, 2):
+                raise ValueError("a group's score is its largest or the sum of its two largest (group_best 1 or 2)")
             if self.identity < 0 or self.groups < 1 or self.n_out % self.groups or not (1 <= self.keep <= self.groups) \
                     or self.top > self.n_out // self.groups * self.keep:
                 raise ValueError(f"{self.groups} groups must divide the router's {self.n_out} outputs, and the {self.keep} kept "
@@ -131,7 +140,8 @@ class RoutedExperts(FeedForward):
         linear(ctx, h, self.w_router, logits)
         if self.grouped_routing:
             ops.moe_route_grouped(logits[:, :self.n_out], self.E, top, self.groups, self.keep, self.weight_scale, self.correction,
-                                  ctx.req_of_token, ids, wts, rank, self.counts, seg)
+                                  ctx.req_of_token, ids, wts, rank, self.counts, seg, sigmoid_scores=not self.softmax,
+                                  group_best=self.group_best, renorm=self.renorm or self.softmax)
         else:
             ops.moe_route(logits[:, :self.E], top, self.softmax, self.renorm, ctx.req_of_token, ids, wts, rank, self.counts, seg,
                           bias=self.b_router)
@@ -142,13 +152,16 @@ class RoutedExperts(FeedForward):
         if xs.dtype == torch.bfloat16:
             from ..kernels import fast
             if self.gated:
-                fused = fast.grouped_linear_bf16(ctx, xs, self.w_gu, act, seg, swiglu_group=self.group)
+                fused = fast.grouped_linear_bf16(ctx, xs, self.w_gu, act, seg, swiglu_group=self.group, glu=self.glu)
             else:
                 fused = fast.grouped_linear_bf16(ctx, xs, self.w_up, act, seg, act=self.act_mode)
         if not fused and self.gated:
             gu = ws.alloc((M, 2 * self.I), torch.float32)
             grouped_linear(ctx, xs, self.w_gu, gu, seg)
-            ops.swiglu(gu, act, self.group)
+            if self.glu:
+                ops.glu_clamped(gu, act, self.group, *self.glu)
+            else:
+                ops.swiglu(gu, act, self.group)
         elif not fused:
             up = ws.alloc((M, self.I), torch.float32)
             grouped_linear(ctx, xs, self.w_up, up, seg)

@@ -39,7 +39,7 @@ class MixWithEmbedding(ResidualInput):
         """x, with what is pending carried out on the way, as the products of this part read it."""
         split = self.dtype == torch.bfloat16
         op = ctx.ws.alloc((x.shape[0], (2 if split else 1) * self.H), self.dtype)
-        post = dict(y=pending.y, w_post=pending.weight, eps_post=pending.eps) if pending is not None else {}
+        post = pending.norm_args() if pending is not None else {}
         ops.sandwich_norm(x, op, mode=ops.SANDWICH_SPLIT if split else ops.SANDWICH_COPY, write_back=False, **post)
         return op
 

@@ -5,6 +5,8 @@ With h the mixer's input, H query heads and G key/value heads (query head h read
 
     q = Wq h,  k = Wk h,  v = Wv h                      with ``bias``: + bq, bk, bv, and + bo on the output
     ``qk_norm="weight"``   q, k <- x / rms(x) * w       per head, one weight vector for all heads, before the rotation
+    ``qk_norm="projection"``  the same with ONE root mean square over all heads of q (and one over all heads of k), weights
+                           of those sizes
     the position encoding (a registered ``position`` part) on q and k
     ``qk_norm="unit"``     q, k <- x / rms(x)           per head, no weight, after the rotation
     ``temp_every`` > 0     q <- q * (1 + temp_coef * ln(floor((p + 1) / temp_every) + 1))
@@ -14,14 +16,17 @@ With h the mixer's input, H query heads and G key/value heads (query head h read
     p_ij = exp(s_ij) / (sum_j' exp(s_ij') + exp(sink_h)) with ``sink``: one more term of the denominator per head, which
                                                          has no key and no value; ``sink="one"``: the term is 1 for every
                                                          head (sink_h = 0) and no tensor holds it
-    o_i = sum_j p_ij v_j over j <= i (and i - j < window when ``window`` > 0),   out = out_scale * Wo concat_heads(o)
+    o_i = sum_j p_ij v_j over j <= i (and i - j < window when ``window`` > 0)
+    ``gate="element"``     o_i <- o_i * sigmoid(Wg h)    element by element over the concatenated heads, in the attention's
+                                                         own epilogue
+    out = out_scale * Wo concat_heads(o)
 
 ``values="keys"``: v = k as projected, ahead of the rotation; there is no Wv.  Key and value of a token then share one
 cached row (csrc/softmax_attention.cu: ``one_row``) of key_dim + rotated dims elements, in which a value's dimensions
 come in another order; the columns of Wo are put into that order when the weights are loaded.
 
 The bucket of every distance is worked out once, in double precision on the host, into a table per head that the kernels
-index by min(i - j, far).  The three input projections run as one product.  The part has the split form
+index by min(i - j, far).  The input projections (the gate's as well) run as one product.  The part has the split form
 (parts/base.py): ``forward_core`` leaves the heads' results, times ``out_scale``, in a buffer, and can be handed the
 columns of a product that an arrangement has run over several parts' stacked input matrices (``proj``).
 """
@@ -57,6 +62,7 @@ class SoftmaxAttention(Mixer):
                  scale: float, norm_eps: float = 1e-6, bias: bool = False, qk_norm: str = "none",
                  position: str = "none", position_args: Optional[dict] = None, temp_coef: float = 0.0, temp_every: int = 0,
                  distance_rows: int = 0, distance_far: int = 0, sink=False, values: str = "own", window: int = 0, out_scale: float = 1.0,
+                 gate: str = "none",
                  dtype: torch.dtype = torch.bfloat16, device=None, names: Optional[Dict[str, str]] = None):
         self.prefix, self.H = prefix, int(hidden_size)
         self.nh, self.nkv, self.D, self.Dv = int(num_heads), int(num_kv_heads), int(key_dim), int(value_dim)
@@ -66,8 +72,11 @@ class SoftmaxAttention(Mixer):
             raise ValueError(f"heads ({num_heads}) must be a multiple of kv_heads ({num_kv_heads})")
         if self.D > 256 or self.Dv > 256:
             raise ValueError("head sizes above 256 are beyond the attention kernels")
-        if qk_norm not in ("none", "weight", "unit"):
-            raise ValueError("qk_norm is 'none', 'weight' (before the rotation) or 'unit' (after it, without a weight)")
+        if qk_norm not in ("none", "weight", "projection", "unit"):
+            raise ValueError("qk_norm is 'none', 'weight' or 'projection' (before the rotation) or 'unit' (after it, without a weight)")
+        if gate not in ("none", "element"):
+            raise ValueError("gate is 'none' or 'element'")
+        self.gated = gate == "element"
         self.scale, self.eps, self.qk_norm, self.bias = float(scale), float(norm_eps), qk_norm, bool(bias)
         self.temp_coef, self.temp_every = float(temp_coef), int(temp_every or 0)
         self.distance_rows, self.distance_far = int(distance_rows or 0), int(distance_far or 0)
@@ -86,7 +95,7 @@ class SoftmaxAttention(Mixer):
         if rdim > self.D:
             raise ValueError(f"{rdim} rotated dimensions do not fit a head of {self.D}")
         n = dict(q="q", k="k", v="v", o="o", q_bias="q.b", k_bias="k.b", v_bias="v.b", o_bias="o.b", q_norm="q.norm",
-                 k_norm="k.norm", rel="rel", sink="sink")
+                 k_norm="k.norm", rel="rel", sink="sink", gate="g")
         n.update(names or {})
         self.names = {k: f"{prefix}.{v}" for k, v in n.items()}
         self.w_in = self.w_out = self.in_bias = self.output_bias = self.q_norm_w = self.k_norm_w = None
@@ -104,9 +113,12 @@ class SoftmaxAttention(Mixer):
                       WeightSpec(nm["o_bias"], (H,), storage="float32")]
             if self.tail < 0:
                 specs.append(WeightSpec(nm["v_bias"], (vw,), storage="float32"))
-        if self.qk_norm == "weight":
-            specs += [WeightSpec(nm["q_norm"], (self.D,), storage="float32", init="norm"),
-                      WeightSpec(nm["k_norm"], (self.D,), storage="float32", init="norm")]
+        if self.qk_norm in ("weight", "projection"):
+            whole = self.qk_norm == "projection"
+            specs += [WeightSpec(nm["q_norm"], (qw if whole else self.D,), storage="float32", init="norm"),
+                      WeightSpec(nm["k_norm"], (kw if whole else self.D,), storage="float32", init="norm")]
+        if self.gated:
+            specs.append(WeightSpec(nm["gate"], (self.nh * self.Dv, H)))
         if self.distance_rows:
             specs.append(WeightSpec(nm["rel"], (self.distance_rows, self.nh), storage="float32"))
         if self.has_sink and not self.sink_is_one:
@@ -116,15 +128,18 @@ class SoftmaxAttention(Mixer):
     def load_weights(self, tensors: Dict[str, torch.Tensor]) -> None:
         nm = self.names
         which = ("q", "k", "v") if self.tail < 0 else ("q", "k")
-        self.w_in = torch.cat([tensors.pop(nm[k]) for k in which], dim=0).contiguous()
+        self.w_in = torch.cat([tensors.pop(nm[k]) for k in which + (("gate",) if self.gated else ())], dim=0).contiguous()
         self.w_out = tensors.pop(nm["o"])
         if self.tail > 0:       # values, and so the heads' results, hold dimensions tail .. D-1, then 0 .. tail-1
             w = self.w_out.view(self.H, self.nh, self.Dv)
             self.w_out = torch.cat([w[:, :, self.tail:], w[:, :, :self.tail]], dim=2).reshape(self.H, -1).contiguous()
+            if self.gated:       # the gate's rows stand in the results' order too
+                g = self.w_in[-self.core_width:].view(self.nh, self.Dv, self.H)
+                g.copy_(torch.cat([g[:, self.tail:], g[:, :self.tail]], dim=1))
         if self.bias:
             self.in_bias = torch.cat([tensors[nm[k + "_bias"]] for k in which]).contiguous()
             self.output_bias = tensors[nm["o_bias"]]
-        if self.qk_norm == "weight":
+        if self.qk_norm in ("weight", "projection"):
             self.q_norm_w, self.k_norm_w = tensors[nm["q_norm"]], tensors[nm["k_norm"]]
         if self.distance_rows:
             rel = tensors[nm["rel"]]
@@ -159,16 +174,17 @@ class SoftmaxAttention(Mixer):
         kind, rdim, inv_freq = self.pos.fused()
         ops.qkv_prepare(proj, self.in_bias, self.q_norm_w, self.k_norm_w, self.qk_norm == "unit", self.eps, kind, rdim, inv_freq,
                         self.temp_coef, self.temp_every, q, cache, ctx, self.nh, self.nkv, self.D, self.Dv, store=True,
-                        rope_positions=self.pos.rotation_positions(ctx), one_row=self.tail >= 0)
-        self.attend(ctx, q, act, cache)
+                        rope_positions=self.pos.rotation_positions(ctx), one_row=self.tail >= 0,
+                        whole_norm=self.qk_norm == "projection")
+        self.attend(ctx, q, act, cache, proj[:, self.w_in.shape[0] - self.core_width:] if self.gated else None)
 
-    def attend(self, ctx, q: torch.Tensor, out: torch.Tensor, cache) -> None:
+    def attend(self, ctx, q: torch.Tensor, out: torch.Tensor, cache, gate: Optional[torch.Tensor] = None) -> None:
         if q.dtype == torch.bfloat16:
             from ..kernels import fast
-            if fast.softmax_attention_bf16(ctx, q, out, cache, self):
+            if fast.softmax_attention_bf16(ctx, q, out, cache, self, gate):
                 return
         ops.softmax_attention(q, out, cache, ctx, self.nh, self.nkv, self.D, self.Dv, self.scale, self.table, self.sink,
-                              self.window, self.out_scale, tail=self.tail)
+                              self.window, self.out_scale, tail=self.tail, gate=gate)
 
     def forward(self, ctx, h, cache, sink=None, add_bias: bool = True):
         """The residual delta.  With ``add_bias`` False the output bias (``output_bias``, times nothing) is left to the
