@@ -7,10 +7,8 @@
 // them, and keeps 256 of the R output columns in registers (blockIdx.z picks the columns; the scores are computed
 // again for every 256 columns, which is cheaper than a second trip of the probabilities through shared memory).
 //
-//   prompt portions: 8 (or 4) warps = as many row tiles, key tiles of 32 rows, every warp takes all keys of a tile,
-//                    tiles arrive by cp.async in two stages (the next one is on its way while this one is used);
-//   single tokens:   one row tile, key tiles of 128 rows of which each of the 8 warps takes 16, one stage; the warps'
-//                    (maximum, sum, output) are merged through shared memory at the end, in warp order.
+// 8 (or 4) warps = as many row tiles, key tiles of 32 rows, every warp takes all keys of a tile, tiles arrive by cp.async in
+// two stages (the next one is on its way while this one is used).  Single decoded tokens have a kernel of their own below.
 // Each head's result may be times a sigmoid (`gate`, see latent_attention.cu).
 // A cached row is found through the request's block table.  A group of TOK batch rows that straddles two requests is handled
 // request by request.  Every row keeps its own maximum and sum, so a token's result does not depend on the batch.
@@ -50,24 +48,27 @@ struct LatentMmaArgs {
     const float* sink;
     const float* gate;            // [T][gate_stride]: head h's result is times sigmoid(gate[t][h]); null: no gate
     long long gate_stride;
+    const int32_t* cu_tokens;     // where each request's rows begin, [num_reqs + 1]
+    int skip_single;              // requests that bring ONE token are left to the kernel for single tokens
+    float* partial;               // [splits][num_reqs][H * (R + 2)] (sums, then maximum and denominator per head): a single token's key slices
+    int splits;
     int hg, tok;                  // heads of a CTA, tokens of a CTA
     int kd16, kdp;                // the row padded to k-steps of 16; the shared-memory row stride in elements
     int* err;
 };
 
-template <int RW, int KW, int STAGES>
-__global__ __launch_bounds__(32 * RW * KW, 1) void latent_attention_mma_kernel(LatentMmaArgs a) {
+template <int RW>
+__global__ __launch_bounds__(32 * RW, 1) void latent_attention_mma_kernel(LatentMmaArgs a) {
     pdl_trigger();
     pdl_wait();
-    constexpr int NWARP = RW * KW, NTHREAD = 32 * NWARP;
-    constexpr int BN = KW == 1 ? 32 : 16 * KW;   // cached rows of a tile
-    constexpr int WK = BN / KW;                  // cached rows of a tile one warp takes
+    constexpr int NWARP = RW, NTHREAD = 32 * NWARP, STAGES = 2;
+    constexpr int BN = 32;                       // cached rows of a tile
     constexpr int ROWS = 16 * RW;
     extern __shared__ __align__(16) uint8_t lm_smem[];
     __nv_bfloat16* s_q = reinterpret_cast<__nv_bfloat16*>(lm_smem);                  // [ROWS][kdp]
     __nv_bfloat16* s_k = s_q + (size_t)ROWS * a.kdp;                                 // [2][BN][kdp]
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int rw = KW == 1 ? warp : 0, kw = KW == 1 ? 0 : warp;
+    const int rw = warp;
     const int KD = a.R + a.rd, kdp = a.kdp;
     const int t0 = blockIdx.x * a.tok, t1 = min(t0 + a.tok, a.T);
     const int h0 = blockIdx.y * a.hg, c0 = blockIdx.z * LM_CW;
@@ -83,6 +84,10 @@ __global__ __launch_bounds__(32 * RW * KW, 1) void latent_attention_mma_kernel(L
             continue;
         }
         while (te < t1 && a.req_of_token[te] == req) ++te;
+        if (a.skip_single && a.cu_tokens[req + 1] - a.cu_tokens[req] == 1) {      // left to the kernel for single tokens
+            tb = te;
+            continue;
+        }
         const int p_first = a.positions[tb], n_tok = te - tb;
         const int p_last = p_first + n_tok - 1;
         const int j_lo = a.window > 0 ? max(0, p_first - a.window + 1) : 0;
@@ -126,7 +131,7 @@ __global__ __launch_bounds__(32 * RW * KW, 1) void latent_attention_mma_kernel(L
             }
             asm volatile("cp.async.commit_group;" ::: "memory");
         };
-        if (STAGES == 2) load_tile(tile0, 0);
+        load_tile(tile0, 0);
 
         float o[LM_NT][4];
 #pragma unroll
@@ -142,20 +147,19 @@ __global__ __launch_bounds__(32 * RW * KW, 1) void latent_attention_mma_kernel(L
         const int n_pairs = min(LM_NT / 2, (a.R - c0 + 15) / 16);      // pairs of 8 output columns this CTA has
 
         for (int tile = tile0, it = 0; tile < tile_end; ++tile, ++it) {
-            const int buf = STAGES == 2 ? (it & 1) : 0;
-            if (STAGES == 2 && tile + 1 < tile_end) {
+            const int buf = it & 1;
+            if (tile + 1 < tile_end) {
                 load_tile(tile + 1, buf ^ 1);
                 asm volatile("cp.async.wait_group 1;" ::: "memory");
             } else {
-                if (STAGES == 1) load_tile(tile, 0);       // one stage: the warps of a tile wait for it together
                 asm volatile("cp.async.wait_group 0;" ::: "memory");
             }
             __syncthreads();
-            const __nv_bfloat16* kt = s_k + (size_t)buf * BN * kdp + (size_t)kw * WK * kdp;
-            // S = Q K^T for this warp's 16 rows and WK cached rows
-            float s[WK / 8][4];
+            const __nv_bfloat16* kt = s_k + (size_t)buf * BN * kdp;
+            // S = Q K^T for this warp's 16 rows and the tile's cached rows
+            float s[BN / 8][4];
 #pragma unroll
-            for (int i = 0; i < WK / 8; ++i) s[i][0] = s[i][1] = s[i][2] = s[i][3] = 0.0f;
+            for (int i = 0; i < BN / 8; ++i) s[i][0] = s[i][1] = s[i][2] = s[i][3] = 0.0f;
             uint32_t qaddr = lm_saddr(s_q + (size_t)(rw * 16 + (lane & 15)) * kdp + (lane >> 4) * 8);
             uint32_t kaddr = lm_saddr(kt + (size_t)((lane & 7) + ((lane >> 4) << 3)) * kdp + ((lane >> 3) & 1) * 8);
             const uint32_t kstep = (uint32_t)(16 * kdp * 2);
@@ -164,7 +168,7 @@ __global__ __launch_bounds__(32 * RW * KW, 1) void latent_attention_mma_kernel(L
                 uint32_t af[4];
                 lm_ldsm4(af, qaddr);
 #pragma unroll
-                for (int np = 0; np < WK / 16; ++np) {
+                for (int np = 0; np < BN / 16; ++np) {
                     uint32_t bf[4];
                     lm_ldsm4(bf, kaddr + np * kstep);
                     lm_mma(s[2 * np], af, bf[0], bf[1]);
@@ -172,10 +176,10 @@ __global__ __launch_bounds__(32 * RW * KW, 1) void latent_attention_mma_kernel(L
                 }
             }
             // scale, mask, online softmax (base 2)
-            const int jbase = tile * BN + kw * WK + qd * 2;
+            const int jbase = tile * BN + qd * 2;
             float tmax[2] = {-INFINITY, -INFINITY};
 #pragma unroll
-            for (int nt = 0; nt < WK / 8; ++nt)
+            for (int nt = 0; nt < BN / 8; ++nt)
 #pragma unroll
                 for (int e = 0; e < 4; ++e) {
                     const int i = e >> 1, j = jbase + nt * 8 + (e & 1);
@@ -195,7 +199,7 @@ __global__ __launch_bounds__(32 * RW * KW, 1) void latent_attention_mma_kernel(L
             }
             float psum[2] = {0.0f, 0.0f};
 #pragma unroll
-            for (int nt = 0; nt < WK / 8; ++nt)
+            for (int nt = 0; nt < BN / 8; ++nt)
 #pragma unroll
                 for (int e = 0; e < 4; ++e) {
                     const int i = e >> 1;
@@ -216,7 +220,7 @@ __global__ __launch_bounds__(32 * RW * KW, 1) void latent_attention_mma_kernel(L
             // O += P V, V = the first R elements of the same cached rows
             const uint32_t vaddr = lm_saddr(kt + (size_t)((lane & 7) + ((lane >> 3) & 1) * 8) * kdp + c0 + (lane >> 4) * 8);
 #pragma unroll
-            for (int ks = 0; ks < WK / 16; ++ks) {
+            for (int ks = 0; ks < BN / 16; ++ks) {
                 uint32_t pf[4] = {lm_pack(s[2 * ks][0], s[2 * ks][1]), lm_pack(s[2 * ks][2], s[2 * ks][3]),
                                   lm_pack(s[2 * ks + 1][0], s[2 * ks + 1][1]), lm_pack(s[2 * ks + 1][2], s[2 * ks + 1][3])};
 #pragma unroll
@@ -233,119 +237,371 @@ __global__ __launch_bounds__(32 * RW * KW, 1) void latent_attention_mma_kernel(L
         }
         if (bad && lane == 0) atomicOr(a.err, AIRUN_DEV_BAD_PAGE);
 
-        if (KW > 1) {
-            // merge the warps' partial results of the same 16 rows, in warp order, through shared memory
-            float* s_m = reinterpret_cast<float*>(s_k);                 // [KW][16] maxima, [KW][16] sums, then [KW][16][LM_CW]
-            float* s_l = s_m + KW * 16;
-            float* s_o = s_l + KW * 16;
-            if (qd == 0) {
-                s_m[warp * 16 + g] = m_run[0]; s_m[warp * 16 + g + 8] = m_run[1];
-                s_l[warp * 16 + g] = l_run[0]; s_l[warp * 16 + g + 8] = l_run[1];
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+            const int r = rw * 16 + g + 8 * i, tl = r / a.hg, h = h0 + r - tl * a.hg;
+            if (tl >= n_tok || h >= a.H) continue;
+            float m = m_run[i], l = l_run[i], scale_o = 1.0f;
+            if (a.sink) {
+                const float sk = a.sink[h] * 1.4426950408889634f;
+                const float mf = fmaxf(m, sk);
+                scale_o = m == -INFINITY ? 0.0f : exp2f(m - mf);
+                l = l * scale_o + exp2f(sk - mf);
             }
+            float inv = l > 0.0f ? scale_o / l : 0.0f;
+            if (a.gate) inv /= 1.0f + __expf(-a.gate[(size_t)(tb + tl) * a.gate_stride + h]);
+            __nv_bfloat16* dst = a.out + ((size_t)(tb + tl) * a.H + h) * a.R + c0;
 #pragma unroll
             for (int nt = 0; nt < LM_NT; ++nt) {
-                float* d = s_o + ((size_t)warp * 16 + g) * LM_CW + nt * 8 + qd * 2;
-                d[0] = o[nt][0]; d[1] = o[nt][1];
-                d[8 * LM_CW] = o[nt][2]; d[8 * LM_CW + 1] = o[nt][3];
-            }
-            __syncthreads();
-            // thread t handles row t / 8 and every 8th column from t % 8
-            const int r = threadIdx.x >> 3, cs = threadIdx.x & 7;
-            const int tl = r / a.hg, h = h0 + r - tl * a.hg;
-            if (r < 16 && tl < n_tok && h < a.H) {
-                float gm = a.sink ? a.sink[h] * 1.4426950408889634f : -INFINITY;
-                const float sk = gm;
-#pragma unroll
-                for (int w = 0; w < KW; ++w) gm = fmaxf(gm, s_m[w * 16 + r]);
-                float wgt[KW], gl = a.sink ? exp2f(sk - gm) : 0.0f;
-#pragma unroll
-                for (int w = 0; w < KW; ++w) {
-                    wgt[w] = s_m[w * 16 + r] == -INFINITY ? 0.0f : exp2f(s_m[w * 16 + r] - gm);
-                    gl += s_l[w * 16 + r] * wgt[w];
-                }
-                float inv = gl > 0.0f ? 1.0f / gl : 0.0f;
-                if (a.gate) inv /= 1.0f + __expf(-a.gate[(size_t)(tb + tl) * a.gate_stride + h]);
-                __nv_bfloat16* dst = a.out + ((size_t)(tb + tl) * a.H + h) * a.R;
-                for (int c = cs; c < LM_CW && c0 + c < a.R; c += 8) {
-                    float v = 0.0f;
-#pragma unroll
-                    for (int w = 0; w < KW; ++w) v = fmaf(s_o[((size_t)w * 16 + r) * LM_CW + c], wgt[w], v);
-                    dst[c0 + c] = __float2bfloat16_rn(v * inv);
-                }
-            }
-        } else {
-#pragma unroll
-            for (int i = 0; i < 2; ++i) {
-                const int r = rw * 16 + g + 8 * i, tl = r / a.hg, h = h0 + r - tl * a.hg;
-                if (tl >= n_tok || h >= a.H) continue;
-                float m = m_run[i], l = l_run[i], scale_o = 1.0f;
-                if (a.sink) {
-                    const float sk = a.sink[h] * 1.4426950408889634f;
-                    const float mf = fmaxf(m, sk);
-                    scale_o = m == -INFINITY ? 0.0f : exp2f(m - mf);
-                    l = l * scale_o + exp2f(sk - mf);
-                }
-                float inv = l > 0.0f ? scale_o / l : 0.0f;
-                if (a.gate) inv /= 1.0f + __expf(-a.gate[(size_t)(tb + tl) * a.gate_stride + h]);
-                __nv_bfloat16* dst = a.out + ((size_t)(tb + tl) * a.H + h) * a.R + c0;
-#pragma unroll
-                for (int nt = 0; nt < LM_NT; ++nt) {
-                    const int c = nt * 8 + qd * 2;
-                    if (c0 + c < a.R) dst[c] = __float2bfloat16_rn(o[nt][2 * i] * inv);
-                    if (c0 + c + 1 < a.R) dst[c + 1] = __float2bfloat16_rn(o[nt][2 * i + 1] * inv);
-                }
+                const int c = nt * 8 + qd * 2;
+                if (c0 + c < a.R) dst[c] = __float2bfloat16_rn(o[nt][2 * i] * inv);
+                if (c0 + c + 1 < a.R) dst[c + 1] = __float2bfloat16_rn(o[nt][2 * i + 1] * inv);
             }
         }
         tb = te;
     }
 }
 
-// qlat [T][H][R + rd], out [T][H][R], pool pages of [page_size][R + rd], all bfloat16.  ``single``: the step's rows
-// are mostly single tokens of different requests (one token a CTA, the warps share the keys); otherwise prompt
-// portions (several tokens a CTA).  Needs (R + rd) % 8 == 0.
-AIRUN_EXPORT int airun_latent_attention_mma(const void* qlat, void* out, const void* pool, const int32_t* block_table,
-                                            int max_blocks, const int32_t* positions, const int32_t* req_of_token, int T,
-                                            int num_reqs, int num_pages, int page_size, int H, int R, int rd, float scale,
-                                            int window, const float* sink, const float* gate, long long gate_stride, int single,
-                                            int* err, cudaStream_t stream) {
+// ---------------------------------------------------------------------------------------------------------
+// Single decoded tokens.  One CTA (8 warps) per (slice of the keys, group of 16 * RT heads, request that brings ONE token):
+// the rows of the products are the heads, so a cached row is read once for all of them, and all R output columns stay in
+// the CTA's registers.  Tiles of 64 cached rows arrive by cp.async in two stages.  In a tile
+//   scores   warp w takes rows 16 (w % 4) .. + 15 and one half (w / 4) of the row's elements; the halves meet in shared memory
+//   softmax  warp w takes 2 RT heads, all 64 scores of a head over its lanes, with the head's running maximum and sum
+//   output   warp w takes the columns 16 (w + 8 i) .. + 15 over all 64 rows
+// With one slice the result (sink, division, gate) goes to `out`; with several each slice writes its float32 sums, maximum
+// and denominator to `partial` and latent_merge_kernel adds them up in slice order.
+#define LG_KEYS 64
+#define LG_SS (LG_KEYS + 8)       // row stride of the scores in shared memory
+#define LG_PAIRS 5                // 16-column pieces of a warp: R <= 8 * 5 * 16
+#define LG_LOG2E 1.4426950408889634f
+
+template <int RT>
+__global__ __launch_bounds__(256, 1) void latent_attention_group_kernel(LatentMmaArgs a) {
+    pdl_trigger();
+    pdl_wait();
+    constexpr int ROWS = 16 * RT, RPW = ROWS / 8;
+    extern __shared__ __align__(16) uint8_t lm_smem[];
+    const int kdp = a.kdp, KD = a.R + a.rd, chunks = KD / 8;
+    __nv_bfloat16* s_q = reinterpret_cast<__nv_bfloat16*>(lm_smem);                  // [ROWS][kdp]
+    __nv_bfloat16* s_k = s_q + (size_t)ROWS * kdp;                                   // [2][64][kdp]
+    float* s_s = reinterpret_cast<float*>(s_k + (size_t)2 * LG_KEYS * kdp);          // [2][ROWS][LG_SS]: the halves' scores
+    __nv_bfloat16* s_p = reinterpret_cast<__nv_bfloat16*>(s_s + 2 * ROWS * LG_SS);   // [ROWS][LG_SS]: the weights
+    float* s_c = reinterpret_cast<float*>(s_p + ROWS * LG_SS);                       // [ROWS] factors, then [ROWS] maxima and [ROWS] sums
+    float* s_m = s_c + ROWS;
+    float* s_l = s_m + ROWS;
+    const int slice = blockIdx.x, h0 = blockIdx.y * ROWS, r = blockIdx.z;
+    const int tok = a.cu_tokens[r];
+    if (a.cu_tokens[r + 1] - tok != 1) return;
+    const int pos = a.positions[tok];                      // the last key the token sees
+    if (pos < 0) return;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, qd = lane & 3;
+    const int first_key = a.window > 0 ? max(0, pos - a.window + 1) : 0;
+    const int tiles = (pos - first_key) / LG_KEYS + 1, per_slice = (tiles + a.splits - 1) / a.splits;
+    const int lo = first_key + slice * per_slice * LG_KEYS;
+    const int hi = min(pos, first_key + (slice + 1) * per_slice * LG_KEYS - 1);
+    const int32_t* bt = a.block_table + (size_t)r * a.max_blocks;
+    // the queries; heads beyond the last one and the padding behind the rows are zero, in the stages too
+    for (int row = warp; row < ROWS; row += 8) {
+        const bool on = h0 + row < a.H;
+        const __nv_bfloat16* src = a.qlat + ((size_t)tok * a.H + (on ? h0 + row : 0)) * KD;
+        for (int ch = lane; ch < kdp / 8; ch += 32) {
+            uint4 v = make_uint4(0, 0, 0, 0);
+            if (on && ch < chunks) v = *reinterpret_cast<const uint4*>(src + ch * 8);
+            *reinterpret_cast<uint4*>(s_q + (size_t)row * kdp + ch * 8) = v;
+        }
+    }
+    for (int e = threadIdx.x; e < 2 * LG_KEYS * (kdp / 8 - chunks); e += 256) {
+        const int row = e / (kdp / 8 - chunks), ch = chunks + e - row * (kdp / 8 - chunks);
+        *reinterpret_cast<uint4*>(s_k + (size_t)row * kdp + ch * 8) = make_uint4(0, 0, 0, 0);
+    }
+    bool bad = false;
+    auto load_tile = [&](int kbase, int buf) {             // warp w copies rows w, w + 8, ...; rows beyond the slice are zeros
+        __nv_bfloat16* dst = s_k + (size_t)buf * LG_KEYS * kdp;
+        int page[LG_KEYS / 8];
+#pragma unroll
+        for (int i = 0; i < LG_KEYS / 8; ++i) {            // the page lookups first, so that they are under way together
+            const int j = kbase + warp + 8 * i, blk = j / a.page_size;
+            page[i] = j <= hi && blk < a.max_blocks ? bt[blk] : (j <= hi ? -1 : -2);
+        }
+#pragma unroll
+        for (int i = 0; i < LG_KEYS / 8; ++i) {
+            const int row = warp + 8 * i, j = kbase + row;
+            __nv_bfloat16* d = dst + (size_t)row * kdp;
+            if (page[i] >= 0 && page[i] < a.num_pages) {
+                const __nv_bfloat16* src = a.pool + ((size_t)page[i] * a.page_size + j % a.page_size) * KD;
+                for (int ch = lane; ch < chunks; ch += 32) lm_cp16(d + ch * 8, src + ch * 8);
+            } else {
+                if (page[i] != -2) bad = true;
+                for (int ch = lane; ch < chunks; ch += 32) *reinterpret_cast<uint4*>(d + ch * 8) = make_uint4(0, 0, 0, 0);
+            }
+        }
+        asm volatile("cp.async.commit_group;" ::: "memory");
+    };
+    float o[RT][LG_PAIRS][8];
+#pragma unroll
+    for (int t = 0; t < RT; ++t)
+#pragma unroll
+        for (int i = 0; i < LG_PAIRS; ++i)
+#pragma unroll
+            for (int e = 0; e < 8; ++e) o[t][i][e] = 0.0f;
+    float m_run[RPW], l_run[RPW];                          // of this warp's heads in the softmax, the same in all lanes
+#pragma unroll
+    for (int i = 0; i < RPW; ++i) { m_run[i] = -INFINITY; l_run[i] = 0.0f; }
+    const int kg = warp & 3, kh = warp >> 2;
+    const int steps = a.kd16 / 16, half = (steps + 1) / 2;
+    const int s0 = kh ? half : 0, s1 = kh ? steps : half;  // this warp's k-steps of a row
+    const int pairs = (a.R + 15) / 16;
+
+    if (lo <= hi) load_tile(lo, 0);
+    int it = 0;
+    for (int kbase = lo; kbase <= hi; kbase += LG_KEYS, ++it) {
+        const int buf = it & 1;
+        asm volatile("cp.async.wait_group 0;" ::: "memory");
+        __syncthreads();                                   // the tile is here, and everybody is done with the one before
+        if (kbase + LG_KEYS <= hi) load_tile(kbase + LG_KEYS, buf ^ 1);
+        const __nv_bfloat16* kt = s_k + (size_t)buf * LG_KEYS * kdp;
+        {
+            float s[RT][2][4];
+#pragma unroll
+            for (int t = 0; t < RT; ++t)
+#pragma unroll
+                for (int i = 0; i < 2; ++i) s[t][i][0] = s[t][i][1] = s[t][i][2] = s[t][i][3] = 0.0f;
+            uint32_t qaddr = lm_saddr(s_q + (size_t)(lane & 15) * kdp + (lane >> 4) * 8 + s0 * 16);
+            uint32_t kaddr = lm_saddr(kt + (size_t)(16 * kg + (lane & 7) + ((lane >> 4) << 3)) * kdp + ((lane >> 3) & 1) * 8 + s0 * 16);
+            const uint32_t qstep = (uint32_t)(16 * kdp * 2);
+#pragma unroll 4
+            for (int st = s0; st < s1; ++st, qaddr += 32, kaddr += 32) {
+                uint32_t bf[4];
+                lm_ldsm4(bf, kaddr);
+#pragma unroll
+                for (int t = 0; t < RT; ++t) {
+                    uint32_t af[4];
+                    lm_ldsm4(af, qaddr + t * qstep);
+                    lm_mma(s[t][0], af, bf[0], bf[1]);
+                    lm_mma(s[t][1], af, bf[2], bf[3]);
+                }
+            }
+            float* dst = s_s + (size_t)kh * ROWS * LG_SS + 16 * kg + 2 * qd;
+#pragma unroll
+            for (int t = 0; t < RT; ++t)
+#pragma unroll
+                for (int i = 0; i < 2; ++i) {
+                    *reinterpret_cast<float2*>(dst + (size_t)(16 * t + g) * LG_SS + 8 * i) = make_float2(s[t][i][0], s[t][i][1]);
+                    *reinterpret_cast<float2*>(dst + (size_t)(16 * t + g + 8) * LG_SS + 8 * i) = make_float2(s[t][i][2], s[t][i][3]);
+                }
+        }
+        __syncthreads();
+#pragma unroll
+        for (int i = 0; i < RPW; ++i) {
+            const int row = warp * RPW + i;
+            const float2 x0 = *reinterpret_cast<const float2*>(s_s + (size_t)row * LG_SS + 2 * lane);
+            const float2 x1 = *reinterpret_cast<const float2*>(s_s + (size_t)(ROWS + row) * LG_SS + 2 * lane);
+            const int j = kbase + 2 * lane;
+            const float v0 = j <= hi ? (x0.x + x1.x) * a.scale_log2 : -INFINITY, v1 = j + 1 <= hi ? (x0.y + x1.y) * a.scale_log2 : -INFINITY;
+            const float m_new = fmaxf(m_run[i], warp_max(fmaxf(v0, v1)));
+            const float corr = m_new == -INFINITY ? 1.0f : exp2f(m_run[i] - m_new);
+            const float p0 = m_new == -INFINITY ? 0.0f : exp2f(v0 - m_new), p1 = m_new == -INFINITY ? 0.0f : exp2f(v1 - m_new);
+            m_run[i] = m_new;
+            l_run[i] = l_run[i] * corr + warp_sum(p0 + p1);
+            *reinterpret_cast<uint32_t*>(s_p + (size_t)row * LG_SS + 2 * lane) = lm_pack(p0, p1);
+            if (lane == 0) s_c[row] = corr;
+        }
+        __syncthreads();
+        const uint32_t vaddr = lm_saddr(kt + (size_t)((lane & 7) + ((lane >> 3) & 1) * 8) * kdp + (lane >> 4) * 8 + warp * 16);
+        const uint32_t paddr = lm_saddr(s_p + (size_t)(lane & 15) * LG_SS + (lane >> 4) * 8);
+        const uint32_t vstep = (uint32_t)(16 * kdp * 2);
+#pragma unroll
+        for (int t = 0; t < RT; ++t) {
+            const float c0 = s_c[16 * t + g], c1 = s_c[16 * t + g + 8];
+            if (c0 != 1.0f || c1 != 1.0f) {                // once the maxima have settled nothing is rescaled
+#pragma unroll
+                for (int i = 0; i < LG_PAIRS; ++i) {
+                    o[t][i][0] *= c0; o[t][i][1] *= c0; o[t][i][2] *= c1; o[t][i][3] *= c1;
+                    o[t][i][4] *= c0; o[t][i][5] *= c0; o[t][i][6] *= c1; o[t][i][7] *= c1;
+                }
+            }
+        }
+#pragma unroll
+        for (int ks = 0; ks < LG_KEYS / 16; ++ks) {
+            uint32_t pf[RT][4];
+#pragma unroll
+            for (int t = 0; t < RT; ++t) lm_ldsm4(pf[t], paddr + t * (uint32_t)(16 * LG_SS * 2) + ks * 32);
+#pragma unroll
+            for (int i = 0; i < LG_PAIRS; ++i) {
+                if (warp + 8 * i < pairs) {
+                    uint32_t vf[4];
+                    lm_ldsm4t(vf, vaddr + ks * vstep + i * 256);
+#pragma unroll
+                    for (int t = 0; t < RT; ++t) {
+                        lm_mma(*reinterpret_cast<float(*)[4]>(&o[t][i][0]), pf[t], vf[0], vf[1]);
+                        lm_mma(*reinterpret_cast<float(*)[4]>(&o[t][i][4]), pf[t], vf[2], vf[3]);
+                    }
+                }
+            }
+        }
+    }
+    if (bad && lane == 0) atomicOr(a.err, AIRUN_DEV_BAD_PAGE);
+#pragma unroll
+    for (int i = 0; i < RPW; ++i)
+        if (lane == 0) { s_m[warp * RPW + i] = m_run[i]; s_l[warp * RPW + i] = l_run[i]; }
+    __syncthreads();
+#pragma unroll
+    for (int t = 0; t < RT; ++t)
+#pragma unroll
+        for (int u = 0; u < 2; ++u) {
+            const int row = 16 * t + g + 8 * u, h = h0 + row;
+            if (h >= a.H) continue;
+            const float m = s_m[row], l = s_l[row];
+            if (a.splits > 1) {
+                float* base = a.partial + ((size_t)slice * a.num_reqs + r) * ((size_t)a.H * (a.R + 2));
+                float* dst = base + (size_t)h * a.R;
+#pragma unroll
+                for (int i = 0; i < LG_PAIRS; ++i)
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) {
+                        const int c = (warp + 8 * i) * 16 + (e >> 1) * 8 + 2 * qd + (e & 1);
+                        if (c < a.R) dst[c] = o[t][i][(e >> 1) * 4 + 2 * u + (e & 1)];
+                    }
+                if (warp == 0 && qd == 0) {
+                    base[(size_t)a.H * a.R + 2 * h] = m;
+                    base[(size_t)a.H * a.R + 2 * h + 1] = l;
+                }
+                continue;
+            }
+            const float sk = a.sink ? a.sink[h] * LG_LOG2E : -INFINITY, top = fmaxf(m, sk);
+            const float f = m == -INFINITY ? 0.0f : exp2f(m - top);
+            const float den = l * f + (a.sink ? exp2f(sk - top) : 0.0f);
+            float inv = den > 0.0f ? f / den : 0.0f;
+            if (a.gate) inv /= 1.0f + __expf(-a.gate[(size_t)tok * a.gate_stride + h]);
+            __nv_bfloat16* dst = a.out + ((size_t)tok * a.H + h) * a.R;
+#pragma unroll
+            for (int i = 0; i < LG_PAIRS; ++i)
+#pragma unroll
+                for (int e = 0; e < 4; ++e) {
+                    const int c = (warp + 8 * i) * 16 + (e >> 1) * 8 + 2 * qd + (e & 1);
+                    if (c < a.R) dst[c] = __float2bfloat16_rn(o[t][i][(e >> 1) * 4 + 2 * u + (e & 1)] * inv);
+                }
+        }
+}
+
+// The slices of every single token merged in slice order, with the sink and the gate.  One block per (request, head); lane
+// s of every warp holds slice s's maximum and sum (at most 32 slices).
+__global__ __launch_bounds__(128) void latent_merge_kernel(LatentMmaArgs a) {
+    pdl_trigger();
+    pdl_wait();
+    const int r = blockIdx.x, h = blockIdx.y;
+    const int tok = a.cu_tokens[r];
+    if (a.cu_tokens[r + 1] - tok != 1) return;
+    const int lane = threadIdx.x & 31;
+    const size_t width = (size_t)a.H * (a.R + 2), slice = (size_t)a.num_reqs * width;
+    const float* base = a.partial + (size_t)r * width;
+    const float* ml = base + (size_t)a.H * a.R + 2 * h;
+    const float m = lane < a.splits ? ml[lane * slice] : -INFINITY, l = lane < a.splits ? ml[lane * slice + 1] : 0.0f;
+    const float sk = a.sink ? a.sink[h] * LG_LOG2E : -INFINITY;
+    const float top = fmaxf(warp_max(m), sk);
+    const float w = m == -INFINITY ? 0.0f : exp2f(m - top);
+    const float den = warp_sum(l * w) + (a.sink ? exp2f(sk - top) : 0.0f);
+    float inv = den > 0.0f ? 1.0f / den : 0.0f;
+    if (a.gate) inv /= 1.0f + __expf(-a.gate[(size_t)tok * a.gate_stride + h]);
+    const float* col = base + (size_t)h * a.R;
+    __nv_bfloat16* dst = a.out + ((size_t)tok * a.H + h) * a.R;
+    for (int c0 = 0; c0 < a.R; c0 += 128) {                // (every lane takes part in the shuffles)
+        const int c = min(c0 + (int)threadIdx.x, a.R - 1);
+        float acc = 0.0f;
+#pragma unroll 4
+        for (int s = 0; s < a.splits; ++s) acc = fmaf(col[s * slice + c], __shfl_sync(0xffffffffu, w, s), acc);
+        if (c0 + (int)threadIdx.x < a.R) dst[c] = __float2bfloat16_rn(acc * inv);
+    }
+}
+
+static bool lm_fill(LatentMmaArgs& a, const void* qlat, void* out, const void* pool, const int32_t* block_table, int max_blocks,
+                    const int32_t* cu_tokens, const int32_t* positions, int T, int num_reqs, int num_pages, int page_size, int H, int R,
+                    int rd, float scale, int window, const float* sink, const float* gate, long long gate_stride, int* err) {
     const int KD = R + rd;
-    if (T < 0 || H <= 0 || R <= 0 || rd < 0 || KD % 8 != 0 || KD > 1024 || page_size <= 0 || num_pages <= 0 || max_blocks <= 0 ||
-        window < 0 || !err || (gate && gate_stride < H) || (((uintptr_t)qlat | (uintptr_t)pool) & 15))
-        return AIRUN_ERR_ARG;
-    if (T == 0) return AIRUN_OK;
-    LatentMmaArgs a = {};
+    if (T < 0 || num_reqs < 0 || H <= 0 || R <= 0 || rd < 0 || KD % 8 != 0 || KD > 640 || page_size <= 0 || num_pages <= 0 ||
+        max_blocks <= 0 || window < 0 || !err || !cu_tokens || !positions || (gate && gate_stride < H) ||
+        (((uintptr_t)qlat | (uintptr_t)pool) & 15))
+        return false;
     a.qlat = (const __nv_bfloat16*)qlat; a.out = (__nv_bfloat16*)out; a.pool = (const __nv_bfloat16*)pool;
-    a.block_table = block_table; a.max_blocks = max_blocks; a.positions = positions; a.req_of_token = req_of_token;
+    a.block_table = block_table; a.max_blocks = max_blocks; a.cu_tokens = cu_tokens; a.positions = positions;
     a.T = T; a.num_reqs = num_reqs; a.num_pages = num_pages; a.page_size = page_size; a.H = H; a.R = R; a.rd = rd; a.window = window;
-    a.scale_log2 = scale * 1.4426950408889634f;
+    a.scale_log2 = scale * LG_LOG2E;
     a.sink = sink; a.gate = gate; a.gate_stride = gate_stride; a.err = err;
     a.kd16 = (KD + 15) / 16 * 16;
     a.kdp = a.kd16 + 8;
-    // prompt portions: 8 row tiles (128 rows) a CTA when its queries and two key tiles fit the shared memory, else 4;
-    // single tokens: one row tile, 8 warps on the 128 cached rows of a tile, one stage
+    a.splits = 1;
+    return true;
+}
+
+// Prompt portions (and, with skip_single == 0, single tokens too).  qlat [T][H][R + rd], out [T][H][R], pool pages of
+// [page_size][R + rd], all bfloat16.  Needs (R + rd) % 8 == 0 and rows of up to 640 elements.
+AIRUN_EXPORT int airun_latent_attention_mma(const void* qlat, void* out, const void* pool, const int32_t* block_table,
+                                            int max_blocks, const int32_t* cu_tokens, const int32_t* positions,
+                                            const int32_t* req_of_token, int T, int num_reqs, int num_pages,
+                                            int page_size, int H, int R, int rd, float scale, int window, const float* sink,
+                                            const float* gate, long long gate_stride, int skip_single, int* err, cudaStream_t stream) {
+    LatentMmaArgs a = {};
+    if (!req_of_token || !lm_fill(a, qlat, out, pool, block_table, max_blocks, cu_tokens, positions, T, num_reqs, num_pages,
+                                                page_size, H, R, rd, scale, window, sink, gate, gate_stride, err))
+        return AIRUN_ERR_ARG;
+    if (T == 0) return AIRUN_OK;
+    a.req_of_token = req_of_token; a.skip_single = skip_single;
+    // 8 row tiles (128 rows) a CTA when its queries and two key tiles fit the shared memory, else 4
     const size_t limit = 227 * 1024;
-    int rw = single ? 1 : 8;
-    if (!single && ((size_t)128 + 2 * 32) * a.kdp * 2 > limit) rw = 4;
-    const int rows = 16 * rw, bn = single ? 128 : 32, stages = single ? 1 : 2;
+    const int rw = ((size_t)128 + 2 * 32) * a.kdp * 2 > limit ? 4 : 8, rows = 16 * rw;
     a.hg = H < rows ? H : rows;
     a.tok = rows / a.hg;
-    size_t kbytes = (size_t)stages * bn * a.kdp * 2;
-    if (single) { const size_t merge = (2 * 8 * 16 + (size_t)8 * 16 * LM_CW) * 4; if (kbytes < merge) kbytes = merge; }
-    const size_t smem = (size_t)rows * a.kdp * 2 + kbytes;
+    const size_t smem = ((size_t)rows + 2 * 32) * a.kdp * 2;
     if (smem > limit) return AIRUN_ERR_ARG;
     dim3 grid(ceil_div_i(T, a.tok), ceil_div_i(H, a.hg), ceil_div_i(R, LM_CW));
     if (grid.y > 65535 || grid.z > 65535) return AIRUN_ERR_ARG;
-    static unsigned long long conf1 = 0, conf4 = 0, conf8 = 0;
-#define LM_LAUNCH(RW_, KW_, ST_, CONF) do { \
-        auto kern = latent_attention_mma_kernel<RW_, KW_, ST_>; \
+    static unsigned long long conf4 = 0, conf8 = 0;
+#define LM_LAUNCH(RW_, CONF) do { \
+        auto kern = latent_attention_mma_kernel<RW_>; \
         if (first_on_device(CONF)) { \
             cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)limit); \
             if (e != cudaSuccess) return (int)e; \
         } \
-        airun_launch(kern, grid, dim3(32 * RW_ * KW_), smem, stream, a); } while (0)
-    if (single) LM_LAUNCH(1, 8, 1, conf1);
-    else if (rw == 8) LM_LAUNCH(8, 1, 2, conf8);
-    else LM_LAUNCH(4, 1, 2, conf4);
+        airun_launch(kern, grid, dim3(32 * RW_), smem, stream, a); } while (0)
+    if (rw == 8) LM_LAUNCH(8, conf8);
+    else LM_LAUNCH(4, conf4);
 #undef LM_LAUNCH
+    return airun_launch_status();
+}
+
+// The single tokens of the batch (requests that bring one).  splits > 1: the keys of a token are cut into that many slices,
+// and `partial` holds splits * num_reqs * H * (R + 2) floats.
+AIRUN_EXPORT int airun_latent_attention_group(const void* qlat, void* out, const void* pool, const int32_t* block_table, int max_blocks,
+                                              const int32_t* cu_tokens, const int32_t* positions, int T, int num_reqs, int num_pages,
+                                              int page_size, int H, int R, int rd, float scale, int window, const float* sink,
+                                              const float* gate, long long gate_stride, int splits, float* partial, int* err,
+                                              cudaStream_t stream) {
+    LatentMmaArgs a = {};
+    if (!lm_fill(a, qlat, out, pool, block_table, max_blocks, cu_tokens, positions, T, num_reqs, num_pages, page_size, H, R, rd, scale,
+                 window, sink, gate, gate_stride, err) ||
+        splits < 1 || splits > 32 || (splits > 1 && !partial) || num_reqs > 65535 || H > 65535)
+        return AIRUN_ERR_ARG;
+    if (T == 0 || num_reqs == 0) return AIRUN_OK;
+    a.splits = splits; a.partial = partial;
+    const int rt = H > 16 ? 2 : 1, rows = 16 * rt;
+    const size_t smem = ((size_t)rows + 2 * LG_KEYS) * a.kdp * 2 + (size_t)rows * LG_SS * (2 * 4 + 2) + (size_t)3 * rows * 4;
+    const size_t limit = 227 * 1024;
+    if (smem > limit) return AIRUN_ERR_ARG;
+    dim3 grid(splits, ceil_div_i(H, rows), num_reqs);
+    static unsigned long long conf1 = 0, conf2 = 0;
+#define LG_LAUNCH(RT_, CONF) do { \
+        auto kern = latent_attention_group_kernel<RT_>; \
+        if (first_on_device(CONF)) { \
+            cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)limit); \
+            if (e != cudaSuccess) return (int)e; \
+        } \
+        airun_launch(kern, grid, dim3(256), smem, stream, a); } while (0)
+    if (rt == 2) LG_LAUNCH(2, conf2);
+    else LG_LAUNCH(1, conf1);
+#undef LG_LAUNCH
+    int rc = airun_launch_status();
+    if (rc != AIRUN_OK || splits == 1) return rc;
+    airun_launch(latent_merge_kernel, dim3(num_reqs, H), dim3(128), 0, stream, a);
     return airun_launch_status();
 }

@@ -658,7 +658,7 @@ def diff_attention_bf16(ctx, q, out, cache, part) -> bool:
 
 def latent_attention_bf16(ctx, qlat, out, cache, part, gate: Optional[torch.Tensor] = None) -> bool:
     """Attention over a cached latent on the tensor cores (csrc/latent_attention_mma.cu): prompt portions with several
-    tokens a CTA, steps of single tokens with one token a CTA whose warps share the keys.  False: the caller runs the
+    tokens a CTA, single tokens with the heads as rows and their keys cut into slices.  False: the caller runs the
     plain kernel (rows that are no multiple of 8 elements, or too long for the shared memory)."""
     H, R, rd = part.nh, part.R, part.rd
     KD = R + rd
@@ -672,13 +672,43 @@ def latent_attention_bf16(ctx, qlat, out, cache, part, gate: Optional[torch.Tens
     pool, bt = cache.pool, cache.block_table
     _need(pool.is_contiguous() and pool[0].numel() == cache.page_size * KD, "the cache pages do not fit the latent rows")
     _need(qlat.data_ptr() % 16 == 0 and pool.data_ptr() % 16 == 0, "qlat and the cache pages must begin on 16-byte boundaries")
-    f = _fn("latent_attention_mma", "airun_latent_attention_mma",
-            [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
-             c_float, c_int, c_void_p, c_void_p, c_longlong, c_int, c_void_p, c_void_p])
-    _check(f(_p(qlat), _p(out), _p(pool), _p(bt), bt.stride(0), _p(ctx.positions), _p(ctx.req_of_token), T, int(ctx.num_reqs),
-             pool.shape[0], int(cache.page_size), H, R, rd, float(part.scale), int(part.window), _p(part.sink),
-             _p(gate), ops.attention_gate(gate, T, H), 1 if getattr(ctx, "decode_only", False) else 0, _p(ctx.err), _stream()), "latent_attention_mma")
+    _need(ctx.cu_tokens.numel() >= ctx.num_reqs + 1, "the batch's layout arrays are shorter than its number of requests")
+    common = [_p(qlat), _p(out), _p(pool), _p(bt), bt.stride(0), _p(ctx.cu_tokens), _p(ctx.positions)]
+    consts = [T, int(ctx.num_reqs), pool.shape[0], int(cache.page_size), H, R, rd, float(part.scale), int(part.window), _p(part.sink),
+              _p(gate), ops.attention_gate(gate, T, H)]
+    sig = [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p]
+    csig = [c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_void_p, c_void_p, c_longlong]
+    # requests that bring ONE token go to the kernel whose product rows are the heads, their keys cut into slices; it finds
+    # them on the device, and the kernel for portions then skips them
+    single = "latent_group" not in DISABLED
+    decode_only, extras = bool(getattr(ctx, "decode_only", False)), getattr(ctx, "extras", {})
+    lens = None if extras.get("device_plan") else getattr(ctx, "query_lens", None)
+    if single and (decode_only or lens is None or 1 in list(lens)):
+        # (a context that does not say how long its requests are: as long as their block tables)
+        context = extras.get("planning_context_len", getattr(ctx, "max_context_len", bt.shape[1] * int(cache.page_size)))
+        if part.window > 0:
+            context = min(context, part.window)
+        rows = 32 if H > 16 else 16
+        resident = max(1, 227 * 1024 // latent_group_smem(rows, KD))
+        splits = plan_sigmoid_slices(int(ctx.num_reqs), -(-H // rows), int(context), resident * machine(qlat.device).sms, LATENT_MIN_KEYS_PER_SLICE)
+        partial = ctx.ws.alloc((splits, int(ctx.num_reqs), H * (R + 2)), torch.float32) if splits > 1 else None
+        f = _fn("latent_attention_mma", "airun_latent_attention_group", sig + csig + [c_int, c_void_p, c_void_p, c_void_p])
+        _check(f(*common, *consts, splits, _p(partial), _p(ctx.err), _stream()), "latent_attention_group")
+    if single and decode_only:
+        return True
+    f = _fn("latent_attention_mma", "airun_latent_attention_mma", sig + [c_void_p] + csig + [c_int, c_void_p, c_void_p])
+    _check(f(*common, _p(ctx.req_of_token), *consts, 1 if single else 0, _p(ctx.err), _stream()), "latent_attention_mma")
     return True
+
+
+LATENT_MIN_KEYS_PER_SLICE = 128        # a slice of a single token's cached rows is at least this long
+
+
+def latent_group_smem(rows: int, KD: int) -> int:
+    """Shared memory of a CTA of the kernel for single tokens (csrc/latent_attention_mma.cu): ``rows`` queries and two
+    stages of 64 cached rows of KD elements, the scores and weights of a tile."""
+    kdp = (KD + 15) // 16 * 16 + 8
+    return (rows + 2 * 64) * kdp * 2 + rows * 72 * 10 + 12 * rows + 1024
 
 
 def linear_act_bf16(ctx, x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, mode: int) -> bool:
@@ -707,14 +737,14 @@ def sigmoid_group_resident(D: int, Dv: int) -> int:
     return max(1, min(227 * 1024 // smem, 4))
 
 
-def plan_sigmoid_slices(n_reqs: int, nkv: int, context_len: int, slots: int) -> int:
+def plan_sigmoid_slices(n_reqs: int, nkv: int, context_len: int, slots: int, least: int = SIGMOID_MIN_KEYS_PER_SLICE) -> int:
     """Slices the keys of a single token are cut into.  ``slots`` CTAs run at once and the CTAs (request x KV head x
     slice) come in waves of that many; a CTA's time goes with the length of its slice plus what it costs to set up
     and hand on its sums (about 32 keys' worth).  So s slices cost ceil(units * s / slots) * (context / s + 32): with
     512 units and 444 slots one slice a token is two waves (the second nearly empty) and four slices are five waves
-    of a quarter the length.  No slice is shorter than SIGMOID_MIN_KEYS_PER_SLICE keys."""
+    of a quarter the length.  No slice is shorter than ``least`` keys."""
     units = max(1, n_reqs * nkv)
-    most = max(1, min(context_len // SIGMOID_MIN_KEYS_PER_SLICE, 32))
+    most = max(1, min(context_len // least, 32))
     best, best_cost = 1, None
     for s in range(1, most + 1):
         cost = -(-units * s // max(1, slots)) * (context_len / s + 32.0)

@@ -1118,6 +1118,79 @@ def workload_losalorn(a) -> int:
     return 0
 
 
+# The Pirerax design beside the designs that have its mechanisms, at equal size (--workload pirerax)
+def pirerax_config(size: dict):
+    """A Pirerax configuration of the width, head counts and vocabulary of the other designs' workloads and six layers:
+    latent attention (Pogarax's sizes: heads x (128 + 64), values of 128, latent 512), attention with a query temperature
+    (heads of 128) and the pair of a rotated attention (heads of 128, half of each rotated) with a gated delta rule (Losalorn's
+    sizes: heads x 64 x 128, q/k heads halved, 4 taps), twice over; every layer routes a token to 4 of 16 experts (four groups
+    of which two are kept) of a quarter of the dense feed-forward size: the dense layer's FLOPs."""
+    from airun_b200.config import PireraxConfig
+    W, F, H, G = size["width"], size["ff"], size["heads"], size["kv_heads"]
+    mlp = dict(kind="moe", expert=dict(ff=F // 4, limit=7.0), router=dict(experts=16, top=4, groups=dict(count=4, keep=2)))
+    heads = dict(heads=H, kv_heads=G, dim=128, vdim=128, scale=128 ** -0.5)
+    lat = dict(type="latent_attention", mixer=dict(heads=H, dim=128, rot_dim=64, vdim=128, kv_rank=512, scale=192 ** -0.5,
+                                                   rot=dict(dims=64, base=10000.0)), mlp=mlp)
+    att = dict(type="attention", mixer=dict(heads, q_temp=dict(coef=0.3, every=512)), mlp=mlp)
+    par = dict(type="parallel", mixer=dict(left=dict(heads, rot=dict(dims=64, base=10000.0)),
+                                           right=dict(heads=H, kv_heads=H // 2, dim=64, vdim=128, conv=4)), mlp=mlp)
+    return PireraxConfig.from_dict(dict(architecture="Pirerax", vocab=VEDIZEN_VOCAB, width=W, norm=dict(eps=1e-5), layers=[lat, att, par] * 2))
+
+
+def pirerax_kinds(size: dict, ctx_len: int) -> dict:
+    """Kind -> (module, function, work at t tokens of one prompt, work at a batch of b single tokens, bound)."""
+    from airun_b200.kernels import fast, ops
+    from airun_b200.parts import latent_attention as latent_part
+    W, F, H, G = size["width"], size["ff"], size["heads"], size["kv_heads"]
+    R, rd, D, Dv, Fe, E, top = 512, 64, 128, 128, F // 4, 16, 4
+    tri = lambda t: t * (t + 1) / 2                                   # keys all tokens of a t-token prompt see together
+    return {
+        "norm + add (rms)": (ops, "rmsnorm", lambda t: 10 * t * W * 14.0, lambda b: 10 * b * W * 14.0, "hbm"),
+        "two results normed, averaged, added, normed": (ops, "sandwich_norm", lambda t: 2 * t * W * 18.0, lambda b: 2 * b * W * 18.0, "hbm"),
+        "latent: query parts, norm, rotation, cache write": (ops, "latent_query", lambda t: 2 * t * (H * (D + rd) + R + rd) * 6.0,
+                                                             lambda b: 2 * b * (H * (D + rd) + R + rd) * 6.0, "hbm"),
+        "latent attention": (fast, "latent_attention_bf16", lambda t: 2 * H * 2.0 * (2 * R + rd) * tri(t), lambda b: 2 * b * ctx_len * (R + rd) * 2.0, "mixed"),
+        "products per head (Wuk, Wuv)": (latent_part, "head_linear", lambda t: 2 * t * H * 2.0 * (D * R + R * Dv),
+                                         lambda b: 2 * H * (D * R + R * Dv) * 2.0, "tensor"),
+        "q/k norm, rotation, temperature, cache write": (ops, "qkv_prepare", lambda t: 4 * t * (H + 2 * G) * 128 * 6.0,
+                                                         lambda b: 4 * b * (H + 2 * G) * 128 * 6.0, "hbm"),
+        "softmax attention (sink, gate)": (fast, "softmax_attention_bf16", lambda t: 4 * H * 4.0 * 128 * tri(t), lambda b: 4 * b * ctx_len * G * 256 * 2.0, "mixed"),
+        "delta rule: convolution": (ops, "short_conv", lambda t: 2 * t * (H * 64 + H * 128) * 8.0, lambda b: 2 * b * (H * 64 + H * 128) * 8.0, "hbm"),
+        "delta rule: recurrence": (ops, "recurrent_state", lambda t: t * 2 * H * 64 * 128 * 9.0, lambda b: b * 2 * H * 64 * 128 * 8.0, "fp32"),
+        "norm and gate of the heads": (ops, "gla_out_gate", lambda t: 2 * t * H * 128 * 10.0, lambda b: 2 * b * H * 128 * 10.0, "hbm"),
+        "expert products (gate/up + unit, down)": (fast, "grouped_linear_bf16", lambda t: 6 * t * top * 6.0 * W * Fe,
+                                                   lambda b: 6 * min(E, b * top) * 3 * W * Fe * 2.0, "tensor"),
+        "router with groups": (ops, "moe_route_grouped", lambda t: 6 * t * (E + 3 * top) * 4.0, lambda b: 6 * b * (E + 3 * top) * 4.0, "hbm"),
+        "rows to experts and back": (ops, "moe_scatter", lambda t: 6 * t * (W * 2 + top * W * 2.0), lambda b: 6 * b * (W * 2 + top * W * 2.0), "hbm"),
+        "sum of a token's experts": (ops, "moe_combine", lambda t: 6 * t * (top + 1) * W * 4.0, lambda b: 6 * b * (top + 1) * W * 4.0, "hbm"),
+    }
+
+
+def workload_pirerax(a) -> int:
+    """Prefill (one 2,048-token prompt) and decode (batch 8 and 64 at a context of 1,024) of the Pirerax design, of the
+    Tagulix design (which has its softmax attention and its routed experts), of the Pogarax design (its latent attention) and
+    of the Losalorn design (its gated delta rule) at equal size, and each kind of kernel inside those steps
+    (``measure_design``).  One JSON line per size."""
+    import torch
+    from airun_b200 import Engine, EngineOptions
+    pk = peaks()
+    T, ctx_len, steps = 2048, 1024, max(8, min(a.steps, 32))
+    for name in (a.sizes.split(",") if a.sizes else list(VEDIZEN_SIZES)):
+        size = VEDIZEN_SIZES[name]
+        line = {"workload": "pirerax", "size": size, "layer_runs": 6, "vocab": VEDIZEN_VOCAB, "dtype": "bf16",
+                "data": "synthetic, random weights", "prompt": T, "decode_context": ctx_len, "peaks": pk["source"], "models": {}}
+        for model, cfg, kinds in (("pirerax", pirerax_config(size), pirerax_kinds), ("tagulix", tagulix_pair(size)[0], tagulix_kinds),
+                                  ("pogarax", pogarax_pair(size)[0], pogarax_kinds), ("losalorn", losalorn_config(size), losalorn_kinds)):
+            eng = Engine.from_config(cfg, seed=0, options=EngineOptions(
+                dtype="bfloat16", page_size=16, cache_tokens=64 * (ctx_len + 4 * steps + 64) + 4096, max_batch_tokens=T,
+                max_requests=64, max_context=max(T, ctx_len + 4 * steps + 64)))
+            line["models"][model] = measure_design(eng, kinds(size, ctx_len), T, ctx_len, steps, a.warmup, pk)
+            del eng
+            torch.cuda.empty_cache()
+        print(json.dumps(line), flush=True)
+    return 0
+
+
 def reference_arm(a) -> int:
     """The same metric on the reference's own CUDA kernels (compiled unmodified for sm_100), called
     through their C entry points in the order the reference's runtime calls them
@@ -1298,7 +1371,7 @@ def main() -> int:
     ap.add_argument("--decode-only", action="store_true", help="time the decode step only (for profiling runs)")
     ap.add_argument("--prefill-only", action="store_true", help="time the 2,048-token prompt only (for profiling runs)")
     ap.add_argument("--workload", default="decode", choices=("decode", "serve", "long", "ablate", "vedizen", "pogarax", "gamanex", "tagulix",
-                                                               "losalorn"),
+                                                               "losalorn", "pirerax"),
                     help="decode: the headline line; serve: 128 requests continuously batched (Qwen3-1.7B shape); "
                          "long: a 32,768-token prompt, then decoding alone and as 16 forks (Qwen3-32B shape); "
                          "ablate: the decode step timed with one kind of kernel left out at a time; "
@@ -1306,8 +1379,9 @@ def main() -> int:
                          "pogarax: the same for the Pogarax design beside the Vedizen design; "
                          "gamanex: the same for the Gamanex design beside the Qwen3 decoder; "
                          "tagulix: the same for the Tagulix design beside the Qwen3 decoder; "
-                         "losalorn: the same for the Losalorn design beside the Pogarax and the Tagulix design")
-    ap.add_argument("--sizes", default="", help="vedizen / pogarax / gamanex / tagulix / losalorn: widths to run, comma separated (default: 2048,4096)")
+                         "losalorn: the same for the Losalorn design beside the Pogarax and the Tagulix design; "
+                         "pirerax: the same for the Pirerax design beside the Tagulix, the Pogarax and the Losalorn design")
+    ap.add_argument("--sizes", default="", help="vedizen / pogarax / gamanex / tagulix / losalorn / pirerax: widths to run, comma separated (default: 2048,4096)")
     ap.add_argument("--requests", type=int, default=128, help="serve: requests")
     ap.add_argument("--new-tokens", type=int, default=None, help="serve / long: tokens decoded per request")
     ap.add_argument("--budget", type=int, default=512, help="serve: tokens per step")
@@ -1338,6 +1412,8 @@ def main() -> int:
         return workload_tagulix(a)
     if a.workload == "losalorn":
         return workload_losalorn(a)
+    if a.workload == "pirerax":
+        return workload_pirerax(a)
 
     import torch
     from airun_b200 import Engine, EngineOptions, Qwen3Config

@@ -283,3 +283,119 @@ def plain_greedy(cfg, W, prompt: List[int], n_new: int) -> List[int]:
     for _ in range(n_new):
         toks.append(int(torch.argmax(plain_forward(cfg, W, toks)[-1])))
     return toks[len(prompt):]
+
+
+# ----------------------------------------------------------------------------- configurations and weights
+def moe(ff: int, limit: float, experts: int, top: int, groups: Optional[Tuple[int, int]] = None) -> dict:
+    """``groups``: (count, keep)."""
+    router = dict(experts=experts, top=top)
+    if groups is not None:
+        router["groups"] = dict(count=groups[0], keep=groups[1])
+    return dict(kind="moe", expert=dict(ff=ff, limit=limit), router=router)
+
+
+def latent_layer(heads, dim, rot_dim, vdim, kv_rank, scale, base=10000.0, mlp=None) -> dict:
+    return dict(type="latent_attention", mixer=dict(heads=heads, dim=dim, rot_dim=rot_dim, vdim=vdim, kv_rank=kv_rank, scale=scale,
+                                                    rot=dict(dims=rot_dim, base=base)), mlp=mlp)
+
+
+def attention_layer(heads, kv_heads, dim, vdim, scale, temp=None, mlp=None) -> dict:
+    """``temp``: (coef, every)."""
+    m = dict(heads=heads, kv_heads=kv_heads, dim=dim, vdim=vdim, scale=scale)
+    if temp is not None:
+        m["q_temp"] = dict(coef=temp[0], every=temp[1])
+    return dict(type="attention", mixer=m, mlp=mlp)
+
+
+def parallel_layer(left, right, mlp=None) -> dict:
+    """``left``: (heads, kv_heads, dim, vdim, scale, rotated dims, base); ``right``: (heads, kv_heads, dim, vdim, taps)."""
+    return dict(type="parallel", mixer=dict(
+        left=dict(zip(("heads", "kv_heads", "dim", "vdim", "scale"), left[:5]), rot=dict(dims=left[5], base=left[6])),
+        right=dict(zip(("heads", "kv_heads", "dim", "vdim", "conv"), right))), mlp=mlp)
+
+
+def make_config(vocab: int, width: int, layers: List[dict], eps: float = 1e-5) -> dict:
+    return dict(architecture="Pirerax", vocab=vocab, width=width, norm=dict(eps=eps), layers=layers)
+
+
+def all_experts(cfg: dict) -> dict:
+    """The same model with routers that choose every expert."""
+    cfg = json.loads(json.dumps(cfg))
+    for l in cfg["layers"]:
+        if l.get("mlp"):
+            r = l["mlp"]["router"]
+            r["top"] = r["experts"]
+            if "groups" in r:
+                r["groups"]["keep"] = r["groups"]["count"]
+    return cfg
+
+
+def tensor_shapes(cfg: dict) -> Dict[str, tuple]:
+    Wd = cfg["width"]
+    shapes = {"embed": (cfg["vocab"], Wd), "head": (cfg["vocab"], Wd), "final.norm": (Wd,)}
+
+    def grouped(x: str, m: dict) -> None:
+        H, G, D, Dv = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+        shapes.update({x + "q": (H * D, Wd), x + "k": (G * D, Wd), x + "v": (G * Dv, Wd), x + "q.norm": (H * D,), x + "k.norm": (G * D,),
+                       x + "g": (H * Dv, Wd), x + "o": (Wd, H * Dv)})
+
+    for i, l in enumerate(cfg["layers"]):
+        m, x = l["mixer"], f"l{i}.mix."
+        shapes[f"l{i}.norm1"] = (Wd,)
+        if l["type"] == "latent_attention":
+            H, D, rd, Dv, R = m["heads"], m["dim"], m["rot_dim"], m["vdim"], m["kv_rank"]
+            shapes.update({x + "q": (H * (D + rd), Wd), x + "dkv": (R + rd, Wd), x + "dkv.norm": (R,), x + "uk": (H * D, R),
+                           x + "uv": (H * Dv, R), x + "sink": (H,), x + "g": (H, Wd), x + "o": (Wd, H * Dv)})
+        elif l["type"] == "attention":
+            grouped(x, m)
+            shapes[x + "sink"] = (m["heads"],)
+        else:
+            grouped(x + "left.", m["left"])
+            r, y = m["right"], x + "right."
+            kd, vd = r["kv_heads"] * r["dim"], r["heads"] * r["vdim"]
+            shapes.update({y + "q": (kd, Wd), y + "k": (kd, Wd), y + "v": (vd, Wd), y + "q.conv": (kd, r["conv"]), y + "k.conv": (kd, r["conv"]),
+                           y + "v.conv": (vd, r["conv"]), y + "b": (r["heads"], Wd), y + "a": (r["heads"], Wd), y + "A_log": (r["heads"],),
+                           y + "dt_bias": (r["heads"],), y + "norm": (r["vdim"],), y + "g": (vd, Wd), y + "o": (Wd, vd),
+                           x + "left.out": (Wd,), x + "right.out": (Wd,)})
+        if l.get("mlp"):
+            ff = l["mlp"]["expert"]["ff"]
+            shapes.update({f"l{i}.norm2": (Wd,), f"l{i}.mlp.router": (l["mlp"]["router"]["experts"], Wd)})
+            for e in range(l["mlp"]["router"]["experts"]):
+                shapes.update({f"l{i}.mlp.e{e}.gate": (ff, Wd), f"l{i}.mlp.e{e}.up": (ff, Wd), f"l{i}.mlp.e{e}.down": (Wd, ff)})
+    return shapes
+
+
+def random_weights(cfg: dict, seed: int, gain: float = 1.0) -> Dict[str, torch.Tensor]:
+    """Weights large enough that every mechanism moves the logits: matrices N(0, gain^2 / fan_in), gates, routers and the
+    experts' gates twice that, norm weights near 1, sinks near 1, decays spread between slow and fast; all rounded to
+    bfloat16, the file's type."""
+    g = torch.Generator().manual_seed(seed)
+    W = {}
+    for name, shape in tensor_shapes(cfg).items():
+        leaf = name.rsplit(".", 1)[-1]
+        if leaf == "conv":
+            t = 0.6 * torch.randn(shape, generator=g)
+        elif len(shape) == 2:
+            std = 1.0 if name == "embed" else gain / math.sqrt(shape[1])
+            if leaf in ("gate", "g", "router"):
+                std *= 2.0
+            t = torch.randn(shape, generator=g) * std
+        elif leaf.startswith("norm") or leaf == "out":
+            t = 1.0 + 0.2 * torch.randn(shape, generator=g)
+        elif leaf == "A_log":
+            t = torch.randn(shape, generator=g) - 1.0
+        elif leaf == "sink":
+            t = 1.0 + torch.randn(shape, generator=g)
+        else:                                               # dt_bias
+            t = 0.5 * torch.randn(shape, generator=g)
+        W[name] = t.to(torch.bfloat16)
+    return W
+
+
+def write_folder(folder: str, cfg: dict, W: Dict[str, torch.Tensor]) -> str:
+    from safetensors.torch import save_file
+    os.makedirs(folder, exist_ok=True)
+    with open(os.path.join(folder, "config.json"), "w") as f:
+        json.dump(cfg, f)
+    save_file({k: v.contiguous() for k, v in W.items()}, os.path.join(folder, "model.safetensors"))
+    return folder
