@@ -195,6 +195,8 @@ struct GemmParams {
     // memory) and segment e is multiplied by rows e * b_rows .. of the B operand (one matrix per segment, stacked)
     const int32_t* seg;
     int n_seg;
+    int batch_a;                  // batched form: columns of A from one product to the next, and elements of the output
+    long long batch_out;
 };
 
 template <int BN, int STAGES>
@@ -659,14 +661,21 @@ __global__ __launch_bounds__(GEMM_THREADS, 1) void gemm_tcgen05_kernel(
 // the row tiles of all segments in shared memory (first row, end of the segment, segment) and then walks
 // (row tile, column tile) pairs as above; a tile's rows beyond its segment's end are computed and not stored.  The
 // launch is sized for the most row tiles any cut can have, ceil(rows / 128) + segments.
+//
+// BATCHED: n_seg products of equal sizes in one launch: product e reads the columns e * batch_a .. + K - 1 of A (column
+// slices of one buffer: the heads of a per-head product), has the rows e * b_rows .. of B as its matrix and writes its
+// bfloat16 result batch_out elements further on than product e - 1.  A last K block that reaches into the next slice's
+// columns meets zeros there: beyond K the tensor map of B has nothing.
 #define PBN 256
 #define PSTAGES 4
 #define GROUP_MAX_TILES 1024
 #define GROUP_MAX_SEGS 1024
-template <int EPI, bool GROUPED>
+enum { FORM_PLAIN = 0, FORM_GROUPED = 1, FORM_BATCHED = 2 };
+template <int EPI, int FORM>
 __global__ __launch_bounds__(GEMM_THREADS, 1) void gemm_tcgen05_persistent_kernel(
     const __grid_constant__ CUtensorMap map_a, const __grid_constant__ CUtensorMap map_b, const GemmParams p,
     int m_tiles, int n_tiles) {
+    constexpr bool GROUPED = FORM == FORM_GROUPED, BATCHED = FORM == FORM_BATCHED;
     pdl_trigger();
     __shared__ int s_tab[GROUPED ? 3 * GROUP_MAX_TILES : 1], s_first[GROUPED ? GROUP_MAX_SEGS + 1 : 1];
     using L = SmemLayout<PBN, PSTAGES>;
@@ -676,7 +685,7 @@ __global__ __launch_bounds__(GEMM_THREADS, 1) void gemm_tcgen05_persistent_kerne
     __shared__ uint32_t tmem_slot_p;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int kb_total = (p.K + BK - 1) / BK;
-    int total_tiles = m_tiles * n_tiles;
+    int total_tiles = m_tiles * n_tiles * (BATCHED ? p.n_seg : 1);
     const uint32_t full0 = smem_u32(bars), empty0 = smem_u32(bars + PSTAGES);
     const uint32_t accf0 = smem_u32(bars + 2 * PSTAGES), acce0 = smem_u32(bars + 2 * PSTAGES + 2);
     if (threadIdx.x == 0) {
@@ -695,7 +704,8 @@ __global__ __launch_bounds__(GEMM_THREADS, 1) void gemm_tcgen05_persistent_kerne
     // (Not when grouped: which matrix a tile needs is not known before the segments are.)
     const int n_pre = (!GROUPED && (int)blockIdx.x < total_tiles) ? (kb_total < PSTAGES ? kb_total : PSTAGES) : 0;
     if (warp == 0 && lane == 0) {
-        const int b0 = ((int)blockIdx.x / m_tiles) * PBN;
+        const int col = (int)blockIdx.x / m_tiles;
+        const int b0 = BATCHED ? (col % n_tiles) * PBN + (col / n_tiles) * p.b_rows : col * PBN;
         for (int i = 0; i < n_pre; ++i) {
             mbar_expect_tx(full0 + 8 * i, L::STAGE_BYTES);
             tma_load_2d(smem_u32(smem + i * L::STAGE_BYTES) + L::A_BYTES, &map_b, full0 + 8 * i, i * BK, b0);
@@ -728,17 +738,19 @@ __global__ __launch_bounds__(GEMM_THREADS, 1) void gemm_tcgen05_persistent_kerne
             for (int tile = blockIdx.x; tile < total_tiles && ok; tile += gridDim.x) {
                 const int mi = tile % m_tiles;
                 const int a0 = GROUPED ? s_tab[3 * mi] : mi * BM;
-                const int b0 = (tile / m_tiles) * PBN + (GROUPED ? s_tab[3 * mi + 2] * p.b_rows : 0);
+                const int col = tile / m_tiles, batch = BATCHED ? col / n_tiles : 0;
+                const int b0 = (BATCHED ? col % n_tiles : col) * PBN + (GROUPED ? s_tab[3 * mi + 2] : batch) * p.b_rows;
+                const int ka0 = BATCHED ? batch * p.batch_a : 0;        // where this product's columns of A begin
                 for (int kb = 0; kb < kb_total; ++kb, ++it) {
                     const int s = it % PSTAGES;
                     const uint32_t sa = smem_u32(smem + s * L::STAGE_BYTES);
                     if (it < n_pre) {                // the weight half of this stage is already on its way
-                        tma_load_2d(sa, &map_a, full0 + 8 * s, kb * BK, a0);
+                        tma_load_2d(sa, &map_a, full0 + 8 * s, ka0 + kb * BK, a0);
                         continue;
                     }
                     if (!mbar_wait(empty0 + 8 * s, ((it / PSTAGES) & 1) ^ 1)) { atomicOr(p.err, AIRUN_DEV_TIMEOUT); ok = false; break; }
                     mbar_expect_tx(full0 + 8 * s, L::STAGE_BYTES);
-                    tma_load_2d(sa, &map_a, full0 + 8 * s, kb * BK, a0);
+                    tma_load_2d(sa, &map_a, full0 + 8 * s, ka0 + kb * BK, a0);
                     tma_load_2d(sa + L::A_BYTES, &map_b, full0 + 8 * s, kb * BK, b0);
                 }
             }
@@ -769,11 +781,14 @@ __global__ __launch_bounds__(GEMM_THREADS, 1) void gemm_tcgen05_persistent_kerne
         }
     } else {
         const int quad = warp & 3;
+        GemmParams q = p;                                    // BATCHED: with this product's part of the output
         int n = 0;
         for (int tile = blockIdx.x; tile < total_tiles; tile += gridDim.x, ++n) {
             const int buf = n & 1;
             const int mi = tile % m_tiles;
-            const int a0 = GROUPED ? s_tab[3 * mi] : mi * BM, b0 = (tile / m_tiles) * PBN;
+            const int col = tile / m_tiles;
+            const int a0 = GROUPED ? s_tab[3 * mi] : mi * BM, b0 = (BATCHED ? col % n_tiles : col) * PBN;
+            if (BATCHED) q.out = (__nv_bfloat16*)p.out + (size_t)(col / n_tiles) * p.batch_out;
             const int a_row = a0 + quad * 32 + lane;
             const bool row_on = !GROUPED || a_row < s_tab[3 * mi + 1];       // grouped: rows of the tile's own segment only
             const float row_scale = (AIRUN_FOLD_NORM && p.ssq_in && a_row < p.a_rows) ? token_scale(p, a_row) : 1.0f;   // while the MMAs run
@@ -801,7 +816,7 @@ __global__ __launch_bounds__(GEMM_THREADS, 1) void gemm_tcgen05_persistent_kerne
                 else if (EPI == EPI_RESID) ssq_acc += store_resid_normal(p, v, a_row, b0 + c);
                 else {
                     if (p.act) epilogue_act(v, p.act - 1);
-                    store_chunk<EPI, false>(p, v, a_row, b0, c);
+                    store_chunk<EPI, false>(BATCHED ? q : p, v, a_row, b0, c);
                 }
             }
             if (EPI == EPI_RESID && a_row < p.a_rows) p.ssq_out[(size_t)(tile / m_tiles) * p.ssq_out_ld + a_row] = ssq_acc;
@@ -910,13 +925,14 @@ int launch(const CUtensorMap& ma, const CUtensorMap& mb, const GemmParams& p, di
     return airun_launch_status();
 }
 
-template <int EPI, bool GROUPED = false>
+template <int EPI, int FORM = FORM_PLAIN>
 int launch_persistent(const CUtensorMap& ma, const CUtensorMap& mb, const GemmParams& p, cudaStream_t stream) {
+    constexpr bool GROUPED = FORM == FORM_GROUPED;
     using L = SmemLayout<PBN, PSTAGES>;
     constexpr int SMEM = L::TOTAL + 64;
     static unsigned long long configured = 0;
     static int sms_of[64];
-    auto kern = gemm_tcgen05_persistent_kernel<EPI, GROUPED>;
+    auto kern = gemm_tcgen05_persistent_kernel<EPI, FORM>;
     int dev = 0;
     cudaGetDevice(&dev);
     if (dev < 0 || dev >= 64) return AIRUN_ERR_ARG;
@@ -928,7 +944,8 @@ int launch_persistent(const CUtensorMap& ma, const CUtensorMap& mb, const GemmPa
     const int n_sm = sms_of[dev];
     const int m_tiles = (p.a_rows + BM - 1) / BM + (GROUPED ? p.n_seg : 0), n_tiles = (p.b_rows + PBN - 1) / PBN;
     if (GROUPED && (m_tiles > GROUP_MAX_TILES || p.n_seg > GROUP_MAX_SEGS)) return AIRUN_ERR_ARG;
-    const int total = m_tiles * n_tiles;
+    const long long total = (long long)m_tiles * n_tiles * (FORM == FORM_BATCHED ? p.n_seg : 1);
+    if (total > 0x3fffffff) return AIRUN_ERR_ARG;
     const int grid = total < n_sm ? total : n_sm;
     airun_launch(kern, dim3(grid), dim3(GEMM_THREADS), SMEM, stream, ma, mb, p, m_tiles, n_tiles);
     return airun_launch_status();
@@ -1145,10 +1162,38 @@ static int gemm_grouped(const void* x, const void* W, void* out, int M, int N, i
     int r;
     if ((r = make_map(&ma, x, M, K, ldx, BM)) != AIRUN_OK) return r;
     if ((r = make_map(&mb, W, (long long)n_seg * N, K, K, PBN)) != AIRUN_OK) return r;
-    if (epi == EPI_F32) return launch_persistent<EPI_F32, true>(ma, mb, p, stream);
-    if (epi == EPI_BF16) return launch_persistent<EPI_BF16, true>(ma, mb, p, stream);
-    if (epi == EPI_SWIGLU) return launch_persistent<EPI_SWIGLU, true>(ma, mb, p, stream);
+    if (epi == EPI_F32) return launch_persistent<EPI_F32, FORM_GROUPED>(ma, mb, p, stream);
+    if (epi == EPI_BF16) return launch_persistent<EPI_BF16, FORM_GROUPED>(ma, mb, p, stream);
+    if (epi == EPI_SWIGLU) return launch_persistent<EPI_SWIGLU, FORM_GROUPED>(ma, mb, p, stream);
     return AIRUN_ERR_UNSUPPORTED;
+}
+
+// The batched product: for every e < n_batch, out[:, e * so .. + N) = x[:, e * sx .. + K) * W[e]^T with x rows of ldx
+// elements, W [n_batch][N][K] contiguous, out rows of ldc elements, all bfloat16.
+AIRUN_EXPORT int airun_gemm_tcgen05_batched(const void* x, const void* W, void* out, int M, int N, int K, int n_batch, long long ldx,
+                                            long long sx, long long ldc, long long so, int* err, cudaStream_t stream) {
+    if (M <= 0 || N <= 0 || K <= 0 || n_batch <= 0 || !err) return M == 0 ? AIRUN_OK : AIRUN_ERR_ARG;
+    if (K % 8 != 0 || ldx % 8 != 0 || sx % 8 != 0 || sx < K || ldx < (n_batch - 1) * sx + K || ((uintptr_t)x & 15) || ((uintptr_t)W & 15))
+        return AIRUN_ERR_ARG;
+    if ((long long)n_batch * N > 0x7fffffffLL || (n_batch - 1) * sx + K > 0x7fffffffLL || so < N || ldc < (n_batch - 1) * so + N)
+        return AIRUN_ERR_ARG;
+    GemmParams p = {};
+    p.a_rows = M;
+    p.b_rows = N;
+    p.K = K;
+    p.k_blocks_per_split = (K + BK - 1) / BK;
+    p.ksplit = 1;
+    p.out = out;
+    p.ldc = ldc;
+    p.err = err;
+    p.n_seg = n_batch;
+    p.batch_a = (int)sx;
+    p.batch_out = so;
+    CUtensorMap ma, mb;
+    int r;
+    if ((r = make_map(&ma, x, M, (n_batch - 1) * sx + K, ldx, BM)) != AIRUN_OK) return r;
+    if ((r = make_map(&mb, W, (long long)n_batch * N, K, K, PBN)) != AIRUN_OK) return r;
+    return launch_persistent<EPI_BF16, FORM_BATCHED>(ma, mb, p, stream);
 }
 
 AIRUN_EXPORT int airun_gemm_tcgen05_ex(const void* x, const void* W, void* out, int M, int N, int K,

@@ -86,10 +86,19 @@ __global__ __launch_bounds__(32 * XA_PREP_WARPS) void qkv_prepare_kernel(
         __shared__ float s_red[33];
         const int qn = nh * D, kn = store ? nkv * D : 0;
         float sq = 0.0f, sk = 0.0f;
-        for (int c = threadIdx.x; c < qn + kn; c += blockDim.x) {
-            const float v = row[c] + (bias ? bias[c] : 0.0f);
-            if (c < qn) sq = fmaf(v, v, sq);
-            else sk = fmaf(v, v, sk);
+        if ((D & 3) == 0 && ((uintptr_t)row & 15) == 0 && !bias) {
+            for (int c = threadIdx.x; c < (qn + kn) >> 2; c += blockDim.x) {
+                const float4 v = reinterpret_cast<const float4*>(row)[c];
+                const float s4 = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, v.w * v.w)));
+                if (4 * c < qn) sq += s4;
+                else sk += s4;
+            }
+        } else {
+            for (int c = threadIdx.x; c < qn + kn; c += blockDim.x) {
+                const float v = row[c] + (bias ? bias[c] : 0.0f);
+                if (c < qn) sq = fmaf(v, v, sq);
+                else sk = fmaf(v, v, sk);
+            }
         }
         whole_q = 1.0f / sqrtf(block_sum(sq, s_red) / (float)qn + eps);
         if (kn) whole_k = 1.0f / sqrtf(block_sum(sk, s_red) / (float)kn + eps);

@@ -272,6 +272,26 @@ def grouped_linear_bf16(ctx, x: torch.Tensor, w: torch.Tensor, out: torch.Tensor
     return True
 
 
+def head_linear_bf16(ctx, x: torch.Tensor, w: torch.Tensor, out: torch.Tensor) -> bool:
+    """out[:, h] = x[:, h] @ w[h]^T for all heads in one launch on tcgen05: x [T, heads, K], w [heads, N, K] contiguous,
+    out [T, heads, N], bfloat16; x and out may be column slices of wider rows.  False when the kernel does not take the
+    sizes or the alignment (the caller then uses the plain batched product)."""
+    T, heads, K = x.shape
+    N = w.shape[1]
+    if ("gemm" in DISABLED or "head_linear" in DISABLED or x.dtype != torch.bfloat16 or w.dtype != torch.bfloat16 or out.dtype != torch.bfloat16
+            or T == 0 or K % 8 or x.stride(0) % 8 or x.stride(1) % 8 or x.data_ptr() % 16 or w.data_ptr() % 16 or not w.is_contiguous()
+            or x.stride(2) != 1 or out.stride(2) != 1):
+        return False
+    _cuda(x, w, out)
+    _need(tuple(w.shape) == (heads, N, K) and tuple(out.shape) == (T, heads, N), "per-head product shapes do not agree")
+    f = _fn("gemm_tcgen05", "airun_gemm_tcgen05_batched",
+            [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_longlong, c_longlong, c_longlong, c_longlong, c_void_p, c_void_p])
+    sx, so = (x.stride(1), out.stride(1)) if heads > 1 else (K, N)
+    _check(f(_p(x), _p(w), _p(out), T, N, K, heads, x.stride(0) if T > 1 else max(x.stride(0), heads * sx),
+             sx, out.stride(0) if T > 1 else max(out.stride(0), heads * so), so, _p(ctx.err), _stream()), "gemm_tcgen05_batched")
+    return True
+
+
 # Folding the residual add and the RMSNorm into the products around them (EPI_RESID + token scales)
 # removes two launches per layer, but as measured on the Qwen3-8B shape the heavier epilogues cost
 # what the launches saved (decode) or more (prompt portions, whose epilogue accesses are strided),

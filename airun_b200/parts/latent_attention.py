@@ -160,18 +160,13 @@ class LatentAttention(Mixer):
 
 def head_linear(ctx, x: torch.Tensor, w: torch.Tensor, out: torch.Tensor) -> None:
     """out[:, h, :] = x[:, h, :] @ w[h]^T for every head: x [T, heads, K], w [heads, N, K], out [T, heads, N]
-    (x and out may be column slices of wider rows).  Prompt portions in bfloat16 run head by head on the tensor
-    cores where the slices are aligned for them; everything else is one launch of the plain batched product."""
-    T, heads, K = x.shape
-    if (x.dtype == torch.bfloat16 and T > HEAD_LOOP_MIN_TOKENS and K % 8 == 0 and x.stride(0) % 8 == 0
-            and (x.stride(1) * 2) % 16 == 0 and x.data_ptr() % 16 == 0):
+    (x and out may be column slices of wider rows).  In bfloat16 all heads run as one launch on the tensor cores where the
+    slices are aligned for them; everything else is one launch of the plain batched product."""
+    if x.dtype == torch.bfloat16:
         from ..kernels import fast
-        if all(fast.linear_bf16(ctx, x[:, h], w[h], out[:, h]) for h in range(heads)):
+        if fast.head_linear_bf16(ctx, x, w, out):
             return
     ops.gemm_simt_batched(x, w, out)
-
-
-HEAD_LOOP_MIN_TOKENS = 128
 
 
 register_part("mixer", "latent_attention", LatentAttention)

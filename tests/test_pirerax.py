@@ -618,6 +618,25 @@ def test_one_latent_that_stands_out(key_at, new, tensor_cores):
     assert torch.allclose(got[-1, :R], c[key_at] * gate0, atol=8e-2) and float(got[-1, R:].abs().max()) < 1e-6
 
 
+@gpu
+@pytest.mark.parametrize("T", [1, 5, 64, 129, 300])
+@pytest.mark.parametrize("heads,K,N,pad_x,pad_out", [(3, 24, 40, 0, 0), (16, 128, 512, 0, 64), (5, 72, 300, 8, 3), (1, 64, 16, 0, 0), (20, 8, 264, 16, 8), (2, 520, 24, 0, 0)])
+def test_products_per_head_in_one_launch(heads, K, N, pad_x, pad_out, T):
+    """Column slices of wider rows on both sides; what lies between the slices (set to large numbers) does not show, nor is
+    anything written there."""
+    from airun_b200.kernels import fast
+    g = torch.Generator().manual_seed(K + N)
+    x = torch.full((T, heads, K + pad_x), 1e4)
+    x[:, :, :K] = P.to_bf16_and_back(torch.randn(T, heads, K, generator=g))
+    w = P.to_bf16_and_back(torch.randn(heads, N, K, generator=g) / math.sqrt(K))
+    xd, out = dev(x, torch.bfloat16), torch.full((T, heads, N + pad_out), 7.0, device="cuda", dtype=torch.bfloat16)
+    ctx = batch_ctx([(0, T)])
+    assert fast.head_linear_bf16(ctx, xd[:, :, :K], dev(w, torch.bfloat16), out[:, :, :N])
+    want = torch.einsum("thk,hnk->thn", x[:, :, :K].double(), w.double())
+    assert int(ctx.err.item()) == 0 and torch.allclose(out[:, :, :N].cpu().double(), want, atol=2e-2, rtol=1e-2)
+    assert (out[:, :, N:] == 7.0).all()
+
+
 # ---- routed experts
 @gpu
 @pytest.mark.parametrize("n_out,top,groups,keep", [(6, 3, 3, 2), (20, 4, 2, 1), (9, 3, 3, 2), (5, 5, 5, 5), (4, 1, 4, 1), (40, 6, 1, 1), (64, 8, 8, 4), (12, 2, 4, 3)])
