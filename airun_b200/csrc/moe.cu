@@ -194,47 +194,72 @@ __global__ void moe_offsets_kernel(const int32_t* __restrict__ counts, int32_t* 
     }
 }
 
+// One block per (token, choice); rows without a weight on them are copied sixteen bytes at a time (`vec`).
 template <typename TH>
 __global__ __launch_bounds__(256) void moe_scatter_kernel(
     const TH* __restrict__ h, int W, int top, const int32_t* __restrict__ ids, const float* __restrict__ wts,
     const int32_t* __restrict__ rank, const int32_t* __restrict__ seg, int scale_input, TH* __restrict__ xs,
-    int32_t* __restrict__ row_of, int num_real) {
+    int32_t* __restrict__ row_of, int num_real, int vec) {
     pdl_trigger();
     pdl_wait();
-    const int t = blockIdx.x;
-    for (int k = 0; k < top; ++k) {
-        const int e = ids[(size_t)t * top + k];
-        if (e < 0) return;
-        if (e >= num_real) {                  // an expert that hands its input on: it has no row in any segment
-            if (threadIdx.x == 0) row_of[(size_t)t * top + k] = -1;
-            continue;
-        }
-        const int row = seg[e] + rank[(size_t)t * top + k];
-        if (threadIdx.x == 0) row_of[(size_t)t * top + k] = row;
-        const float w = scale_input ? wts[(size_t)t * top + k] : 1.0f;
-        for (int c = threadIdx.x; c < W; c += blockDim.x)
-            xs[(size_t)row * W + c] = from_f32<TH>(w * to_f32<TH>(h[(size_t)t * W + c]));
+    const int t = blockIdx.x, k = blockIdx.y;
+    const size_t at = (size_t)t * top + k;
+    const int e = ids[at];
+    if (e < 0) return;
+    if (e >= num_real) {                      // an expert that hands its input on: it has no row in any segment
+        if (threadIdx.x == 0) row_of[at] = -1;
+        return;
     }
+    const int row = seg[e] + rank[at];
+    if (threadIdx.x == 0) row_of[at] = row;
+    if (vec) {
+        const uint4* src = reinterpret_cast<const uint4*>(h + (size_t)t * W);
+        uint4* dst = reinterpret_cast<uint4*>(xs + (size_t)row * W);
+        for (int c = threadIdx.x; c < W * (int)sizeof(TH) / 16; c += blockDim.x) dst[c] = src[c];
+        return;
+    }
+    const float w = scale_input ? wts[at] : 1.0f;
+    for (int c = threadIdx.x; c < W; c += blockDim.x)
+        xs[(size_t)row * W + c] = from_f32<TH>(w * to_f32<TH>(h[(size_t)t * W + c]));
 }
 
-template <typename TH>
+// VEC columns a thread (four on 16-byte boundaries), blockIdx.y picks a token's run of columns.
+template <typename TH, int VEC>
 __global__ __launch_bounds__(256) void moe_combine_kernel(
     const float* __restrict__ ys, int W, int top, const int32_t* __restrict__ ids, const float* __restrict__ wts,
     const int32_t* __restrict__ row_of, int scale_output, float* __restrict__ out, const TH* __restrict__ h) {
     pdl_trigger();
     pdl_wait();
-    const int t = blockIdx.x;
+    const int t = blockIdx.x, c = (blockIdx.y * blockDim.x + threadIdx.x) * VEC;
+    if (c >= W) return;
     const bool pad = ids[(size_t)t * top] < 0;
-    for (int c = threadIdx.x; c < W; c += blockDim.x) {
-        float acc = 0.0f;
-        if (!pad)
-            for (int k = 0; k < top; ++k) {
-                const int r = row_of[(size_t)t * top + k];
-                const float y = r >= 0 ? ys[(size_t)r * W + c] : (h ? to_f32<TH>(h[(size_t)t * W + c]) : 0.0f);
-                acc = scale_output ? fmaf(wts[(size_t)t * top + k], y, acc) : acc + y;
+    float acc[VEC];
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) acc[i] = 0.0f;
+    if (!pad)
+#pragma unroll 4
+        for (int k = 0; k < top; ++k) {
+            const int r = row_of[(size_t)t * top + k];
+            const float w = scale_output ? wts[(size_t)t * top + k] : 1.0f;
+            float y[VEC];
+            if (r >= 0) {
+                const float* src = ys + (size_t)r * W + c;
+                if (VEC == 4) {
+                    const float4 v = *reinterpret_cast<const float4*>(src);
+                    y[0] = v.x; y[1 % VEC] = v.y; y[2 % VEC] = v.z; y[3 % VEC] = v.w;
+                } else {
+                    y[0] = src[0];
+                }
+            } else {
+#pragma unroll
+                for (int i = 0; i < VEC; ++i) y[i] = h ? to_f32<TH>(h[(size_t)t * W + c + i]) : 0.0f;
             }
-        out[(size_t)t * W + c] = acc;
-    }
+#pragma unroll
+            for (int i = 0; i < VEC; ++i) acc[i] = scale_output ? fmaf(w, y[i], acc[i]) : acc[i] + y[i];
+        }
+    float* dst = out + (size_t)t * W + c;
+    if (VEC == 4) *reinterpret_cast<float4*>(dst) = make_float4(acc[0], acc[1 % VEC], acc[2 % VEC], acc[3 % VEC]);
+    else dst[0] = acc[0];
 }
 
 AIRUN_EXPORT int airun_moe_route(const float* z, long long z_stride, const float* bias, int T, int E, int top, int softmax_scores, int renorm,
@@ -270,12 +295,14 @@ AIRUN_EXPORT int airun_moe_scatter(const void* h, int dtype, int T, int W, int t
                                    int num_real, cudaStream_t stream) {
     if (T < 0 || W <= 0 || top <= 0 || !ids || !wts || !rank || !seg || !xs || !row_of || num_real <= 0) return AIRUN_ERR_ARG;
     if (T == 0) return AIRUN_OK;
+    if (top > 65535) return AIRUN_ERR_ARG;
+    const int vec = !scale_input && (W * (dtype == AIRUN_DT_F32 ? 4LL : 2LL)) % 16 == 0 && (((uintptr_t)h | (uintptr_t)xs) & 15) == 0;
     if (dtype == AIRUN_DT_F32)
-        airun_launch(moe_scatter_kernel<float>, dim3(T), dim3(256), 0, stream, (const float*)h, W, top, ids, wts, rank, seg,
-                     scale_input, (float*)xs, row_of, num_real);
+        airun_launch(moe_scatter_kernel<float>, dim3(T, top), dim3(256), 0, stream, (const float*)h, W, top, ids, wts, rank, seg,
+                     scale_input, (float*)xs, row_of, num_real, vec);
     else if (dtype == AIRUN_DT_BF16)
-        airun_launch(moe_scatter_kernel<__nv_bfloat16>, dim3(T), dim3(256), 0, stream, (const __nv_bfloat16*)h, W, top, ids, wts,
-                     rank, seg, scale_input, (__nv_bfloat16*)xs, row_of, num_real);
+        airun_launch(moe_scatter_kernel<__nv_bfloat16>, dim3(T, top), dim3(256), 0, stream, (const __nv_bfloat16*)h, W, top, ids, wts,
+                     rank, seg, scale_input, (__nv_bfloat16*)xs, row_of, num_real, vec);
     else
         return AIRUN_ERR_UNSUPPORTED;
     return airun_launch_status();
@@ -287,13 +314,15 @@ AIRUN_EXPORT int airun_moe_combine(const float* ys, int T, int W, int top, const
                                    cudaStream_t stream) {
     if (T < 0 || W <= 0 || top <= 0 || !ys || !ids || !wts || !row_of || !out) return AIRUN_ERR_ARG;
     if (T == 0) return AIRUN_OK;
-    if (h && h_dtype == AIRUN_DT_BF16)
-        airun_launch(moe_combine_kernel<__nv_bfloat16>, dim3(T), dim3(256), 0, stream, ys, W, top, ids, wts, row_of, scale_output, out,
-                     (const __nv_bfloat16*)h);
-    else if (!h || h_dtype == AIRUN_DT_F32)
-        airun_launch(moe_combine_kernel<float>, dim3(T), dim3(256), 0, stream, ys, W, top, ids, wts, row_of, scale_output, out,
-                     (const float*)h);
-    else
-        return AIRUN_ERR_UNSUPPORTED;
+    const bool vec = W % 4 == 0 && (((uintptr_t)ys | (uintptr_t)out) & 15) == 0;
+    const int threads = 128;
+    const dim3 grid(T, ceil_div_i(W, threads * (vec ? 4 : 1)));
+    if (grid.y > 65535) return AIRUN_ERR_ARG;
+#define MC_LAUNCH(TH, VEC) airun_launch(moe_combine_kernel<TH, VEC>, grid, dim3(threads), 0, stream, ys, W, top, ids, wts, row_of, \
+        scale_output, out, (const TH*)h)
+    if (h && h_dtype == AIRUN_DT_BF16) { if (vec) MC_LAUNCH(__nv_bfloat16, 4); else MC_LAUNCH(__nv_bfloat16, 1); }
+    else if (!h || h_dtype == AIRUN_DT_F32) { if (vec) MC_LAUNCH(float, 4); else MC_LAUNCH(float, 1); }
+    else return AIRUN_ERR_UNSUPPORTED;
+#undef MC_LAUNCH
     return airun_launch_status();
 }

@@ -635,6 +635,79 @@ def check_delta_rule(dev) -> Tuple[float, float]:
     return _rel(got, want), 2e-5
 
 
+def check_latent_attention(dev) -> Tuple[float, float]:
+    """Attention over a cached latent with a rotated part (pairs (i, i + r/2)), a sink and a gate per head, in float32 and on
+    the tensor cores: a prompt portion beside a single token, pages handed out from the pool's end."""
+    from types import SimpleNamespace
+    from .engine.batch import Workspace
+    from .kernels import fast, ops
+    from .parts.rope import RotaryNeox
+    H, D, R, rd, page, lens, new = 5, 16, 40, 8, 8, [60, 300], [25, 1]
+    width, scale, worst = H * (D + rd) + R + rd + H, 0.3, 0.0
+    inv = RotaryNeox(rotary_dim=rd, theta=1000.0, device=dev).inv_freq
+    wkv, sink = 1 + 0.3 * torch.randn(R), torch.randn(H)
+    rows = [torch.randn(n, width) for n in lens]
+    for dtype in (torch.float32, torch.bfloat16):
+        blocks = [(n + page - 1) // page for n in lens]
+        bt, at = torch.full((2, max(blocks)), -1, dtype=torch.int32), sum(blocks)
+        for r, nb in enumerate(blocks):
+            for b in range(nb):
+                at -= 1
+                bt[r, b] = at
+        cache = SimpleNamespace(pool=torch.zeros(sum(blocks), page * (R + rd), device=dev, dtype=dtype), block_table=bt.to(dev), page_size=page)
+        for part in (0, 1):
+            spans = [(0, n - m) if part == 0 else (n - m, n) for n, m in zip(lens, new)]
+            cu = torch.tensor([0, spans[0][1] - spans[0][0], sum(e - a for a, e in spans)], dtype=torch.int32, device=dev)
+            ctx = SimpleNamespace(cu_tokens=cu, num_reqs=2, err=torch.zeros(1, dtype=torch.int32, device=dev), ws=Workspace(dev, 8 << 20), extras={},
+                                  positions=torch.cat([torch.arange(a, e) for a, e in spans]).to(dev, torch.int32), max_context_len=max(lens),
+                                  req_of_token=torch.cat([torch.full((e - a,), r) for r, (a, e) in enumerate(spans)]).to(dev, torch.int32),
+                                  query_lens=[e - a for a, e in spans], decode_only=False)
+            x = torch.cat([rows[r][a:e] for r, (a, e) in enumerate(spans)]).to(dev)
+            qn, qlat = torch.empty(len(x), H * D, device=dev, dtype=dtype), torch.zeros(len(x), H * (R + rd), device=dev, dtype=dtype)
+            ops.latent_query(x, qn, qlat, H, D, R, rd, rd, inv, 1.0, ctx, rope_kind=ops.ROPE_NEOX, wkv=wkv.to(dev), eps=1e-5, cache=cache)
+            qlat.view(-1, H, R + rd)[:, :, :D].copy_(qn.view(-1, H, D))                # Wuk: the first D latents as they are
+        out = torch.zeros(len(x), H * R, device=dev, dtype=dtype)
+        gate = x[:, width - H:]
+        if dtype == torch.bfloat16:
+            part = SimpleNamespace(nh=H, R=R, rd=rd, scale=scale, window=0, sink=sink.to(dev))
+            if not fast.latent_attention_bf16(ctx, qlat, out, cache, part, gate):
+                raise RuntimeError("the tensor-core latent attention refused its sizes")
+        else:
+            ops.latent_attention(qlat, out, cache, ctx, H, R, rd, scale, 0, sink.to(dev), gate)
+        want = []
+        for r, (a, e) in enumerate(spans):
+            x64, pos = rows[r].double(), torch.arange(lens[r])
+            q, c, kr = x64[:, :H * (D + rd)].view(-1, H, D + rd), x64[:, H * (D + rd):H * (D + rd) + R], x64[:, H * (D + rd) + R:-H]
+            c = c / torch.sqrt((c * c).mean(-1, keepdim=True) + 1e-5) * wkv.double()
+            turn = lambda t: ref_rope_neox(t, pos.tolist(), 1000.0)
+            key, qr = torch.cat([c[:, :D], turn(kr[:, None])[:, 0]], 1), torch.cat([q[..., :D], turn(q[..., D:])], 2)
+            s = torch.einsum("ihd,jd->hij", qr, key) * scale
+            s = s.masked_fill(pos[None, None, :] > pos[None, :, None], -float("inf"))
+            p = torch.softmax(torch.cat([s, sink.double()[:, None, None].expand(H, len(pos), 1)], 2), dim=-1)[:, :, :-1]
+            o = torch.einsum("hij,jr->ihr", p, c) * torch.sigmoid(x64[:, -H:])[:, :, None]
+            want.append(o.reshape(len(pos), H * R)[a:e])
+        err = _rel(out, torch.cat(want))
+        worst = max(worst, err if dtype == torch.float32 else err * 1e-3)             # bfloat16 is held to 2e-2
+    return worst, 2e-5
+
+
+def check_group_routing(dev) -> Tuple[float, float]:
+    """Experts chosen by sigmoid scores inside the best groups (the sum of a group's two largest)."""
+    from .kernels import ops
+    T, E, top, groups, keep = 50, 12, 3, 4, 2
+    z = 2 * torch.randn(T, E)
+    ids, rank = (torch.empty(T, top, dtype=torch.int32, device=dev) for _ in range(2))
+    wts, seg = torch.empty(T, top, device=dev), torch.empty(E + 1, dtype=torch.int32, device=dev)
+    ops.moe_route_grouped(z.to(dev), E, top, groups, keep, 1.0, None, torch.zeros(T, dtype=torch.int32, device=dev), ids, wts, rank,
+                          torch.zeros(E, dtype=torch.int32, device=dev), seg, sigmoid_scores=True, group_best=2, renorm=False)
+    s = torch.sigmoid(z.double())
+    best = s.view(T, groups, E // groups).topk(2, dim=-1).values.sum(-1).topk(keep, dim=-1).indices
+    able = torch.zeros(T, groups, dtype=torch.bool).scatter_(1, best, True).repeat_interleave(E // groups, dim=1)
+    pick = s.masked_fill(~able, -1.0).topk(top, dim=-1)
+    wrong = float((ids.cpu().long() != pick.indices).sum())
+    return wrong + _rel(wts, pick.values), 2e-6
+
+
 CHECKS: List[Tuple[str, Callable]] = [
     ("embedding gather", check_embedding),
     ("rmsnorm + residual add", check_rmsnorm),
@@ -657,6 +730,8 @@ CHECKS: List[Tuple[str, Callable]] = [
     ("decayed linear attention: recurrence, norm over all heads and gate", check_decay_attention),
     ("norms on both sides of a sub-layer in one pass", check_sandwich_norm),
     ("delta rule with a decay per head: chunks and single tokens", check_delta_rule),
+    ("attention over a latent: rotation, sink, gate; float32 and mma.sync", check_latent_attention),
+    ("experts chosen in groups by sigmoid scores", check_group_routing),
     ("sampling", check_sampling),
     ("largest logits of a row", check_largest_logits),
 ]
